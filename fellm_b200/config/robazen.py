@@ -35,6 +35,8 @@ def _get(d, key, kind, where, *, default=None, required=True, positive=False):
         if isinstance(v, bool) or not isinstance(v, (int, float)):
             raise ConfigError(f"config.json: '{where}.{key}' must be a number, got {v!r}")
         return float(v)
+    if kind is bool and not isinstance(v, bool):
+        raise ConfigError(f"config.json: '{where}.{key}' must be true or false, got {v!r}")
     if kind is dict:
         if not isinstance(v, dict):
             raise ConfigError(f"config.json: '{where}.{key}' must be an object")

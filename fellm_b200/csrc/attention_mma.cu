@@ -1,6 +1,6 @@
 // Causal GQA attention over the paged cache on tensor cores (mma.sync.m16n8k16, ldmatrix,
 // cp.async), bfloat16 queries and cache, float32 softmax and sums; compiled for one head size
-// (-DHD=...).  Two kernels share one inner step ("a 16-row block of queries against a tile of
+// (-DHD=...) and one size of values (-DVD=..., HD by default).  Two kernels share one inner step ("a 16-row block of queries against a tile of
 // keys in shared memory"):
 //
 //  * prefill: portions of prompts (and any mix of item lengths).  A CTA takes one item, one kv
@@ -26,16 +26,27 @@
 #ifndef HD
 #define HD 64
 #endif
+#ifndef VD
+#define VD HD
+#endif
 static_assert(HD % 16 == 0 && HD >= 16 && HD <= 256, "head size: a multiple of 16 in 16..256");
+static_assert(VD % 16 == 0 && VD >= 16 && VD <= 256, "size of values: a multiple of 16 in 16..256");
 
 constexpr int CPR = HD / 8;                         // 16-byte chunks per row
 constexpr bool SWZ = (CPR % 8 == 0);                // rows of whole 128-byte lines: XOR swizzle
 constexpr int ROWB = HD * 2 + (SWZ ? 0 : 16);       // else 16 bytes of padding spread the banks
 constexpr int KS = HD / 16;                         // k16 steps over the head size
-constexpr int DN = HD / 8;                          // n8 tiles over the head size
+constexpr int DN = VD / 8;                          // n8 tiles over the size of values
+constexpr int CPRV = VD / 8;                        // the same of a value's row
+constexpr bool SWZV = (CPRV % 8 == 0);
+constexpr int ROWBV = VD * 2 + (SWZV ? 0 : 16);
+constexpr float LOG2E = 1.4426950408889634f;
 
 __device__ __forceinline__ int tile_off(int row, int chunk) {
   return row * ROWB + ((SWZ ? (chunk ^ (row & 7)) : chunk) << 4);
+}
+__device__ __forceinline__ int tile_off_v(int row, int chunk) {
+  return row * ROWBV + ((SWZV ? (chunk ^ (row & 7)) : chunk) << 4);
 }
 __device__ __forceinline__ void cp_async16(unsigned smem_addr, const void* gmem) {
   asm volatile("cp.async.cg.shared.global [%0], [%1], 16;\n" ::"r"(smem_addr), "l"(gmem));
@@ -65,7 +76,7 @@ __device__ __forceinline__ unsigned pack_bf16(float lo, float hi) {
 }
 
 // One 16-row block of queries (fragments qf) against NKT*8 keys staged at k_s / v_s (shared-memory
-// addresses of [keys][ROWB] tiles).  Thread (g = lane/4, c = lane%4) owns rows g and g+8; a key at
+// addresses of [keys][ROWB] and [keys][ROWBV] tiles).  Thread (g = lane/4, c = lane%4) owns rows g and g+8; a key at
 // tile index i (absolute index key0 + i) counts for row r iff lo[r] <= key0 + i <= hi[r].
 // m, l: running maximum (log2 domain) and this thread's share of the running sum per row.
 // CAPPED: scores are soft-capped, cap * tanh(s * scale / cap), with cap_log2 = cap * log2(e).
@@ -151,7 +162,7 @@ __device__ __forceinline__ void attend_tile(const unsigned (&qf)[KS][4], unsigne
       int row = j * 16 + (lane & 7) + (((lane >> 3) & 1) << 3);
       int chunk = dn * 2 + (lane >> 4);
       unsigned r[4];
-      ldsm_x4_trans(r, v_s + tile_off(row, chunk));
+      ldsm_x4_trans(r, v_s + tile_off_v(row, chunk));
       mma16816(o[2 * dn], a, r[0], r[1]);
       mma16816(o[2 * dn + 1], a, r[2], r[3]);
     }
@@ -200,7 +211,7 @@ __device__ __forceinline__ void load_q_as_b(unsigned (&qb)[KS][2], F row_ptr, in
 // thread's keys only).
 template <int NKT, bool MASKED>
 __device__ __forceinline__ void attend_tile_keys_as_rows(const unsigned (&qb)[KS][2], unsigned k_s, unsigned v_s, int key0,
-                                                         int lo, int hi, float scale_log2, float (&ot)[HD / 16][4],
+                                                         int lo, int hi, float scale_log2, float (&ot)[VD / 16][4],
                                                          float (&m)[2], float (&l)[2], int lane) {
   constexpr int KB = NKT / 2;                            // blocks of 16 keys
   const int g = lane >> 2;
@@ -244,7 +255,7 @@ __device__ __forceinline__ void attend_tile_keys_as_rows(const unsigned (&qb)[KS
     l[h] *= corr[h];
   }
 #pragma unroll
-  for (int dm = 0; dm < HD / 16; ++dm) { ot[dm][0] *= corr[0]; ot[dm][1] *= corr[1]; ot[dm][2] *= corr[0]; ot[dm][3] *= corr[1]; }
+  for (int dm = 0; dm < VD / 16; ++dm) { ot[dm][0] *= corr[0]; ot[dm][1] *= corr[1]; ot[dm][2] *= corr[0]; ot[dm][3] *= corr[1]; }
 #pragma unroll
   for (int b = 0; b < KB; ++b) {
 #pragma unroll
@@ -261,11 +272,11 @@ __device__ __forceinline__ void attend_tile_keys_as_rows(const unsigned (&qb)[KS
     const unsigned p0 = movmatrix_trans(pack_bf16(s[b][0], s[b][1]));       // keys 2c, 2c+1 of head g
     const unsigned p1 = movmatrix_trans(pack_bf16(s[b][2], s[b][3]));       // keys 2c+8, 2c+9
 #pragma unroll
-    for (int dm = 0; dm < HD / 16; ++dm) {
+    for (int dm = 0; dm < VD / 16; ++dm) {
       const int row = b * 16 + (lane & 7) + ((lane >> 4) << 3);
       const int chunk = dm * 2 + ((lane >> 3) & 1);
       unsigned r[4];
-      ldsm_x4_trans(r, v_s + tile_off(row, chunk));
+      ldsm_x4_trans(r, v_s + tile_off_v(row, chunk));
       mma16816(ot[dm], r, p0, p1);
     }
   }
@@ -286,13 +297,31 @@ struct AttnArgs {
   // slopes [H] of a bias by distance (null: none); a query temperature 1 + qt_coef ln(floor((p + 1) / qt_every) + 1)
   // (qt_every 0: none); kv_planes: 2 = keys then values in a page-layer record, 1 = the values are the keys
   const float* slopes; float qt_coef; int qt_every, kv_planes;
+  // sinks [H] (null: none): exp(sinks[h]) joins the denominator of head h's softmax once, with no key and no value
+  const float* sinks;
 };
+
+// One page of one layer: the keys [G][page_tokens][HD], then (unless they are the values too) the values [G][page_tokens][VD].
+__device__ __forceinline__ size_t record_elems(const AttnArgs& a) {
+  return (size_t)a.G * a.page_tokens * (a.kv_planes == 1 ? HD : HD + VD);
+}
+// (m, l) of a row, m in the log2 domain: the factor of its sums, with the head's sink in the denominator.
+__device__ __forceinline__ float denominator_inv(const AttnArgs& a, int h, float m, float l) {
+  if (!a.sinks) return 1.0f / l;
+  const float sk = a.sinks[h] * LOG2E, mm = fmaxf(m, sk), f = exp2f(m - mm);
+  return f / fmaf(l, f, exp2f(sk - mm));
+}
 
 __device__ __forceinline__ const bf16* key_row(const AttnArgs& a, const int* bt, int g, int key) {
   int lp = key / a.page_tokens;
   int page = max(bt[lp], 0);                 // an unmapped entry (-1) must never become an address: page 0 is read instead
-  return a.pool + ((((size_t)page * a.layers_in_group + a.layer) * a.kv_planes) * a.G + g) * ((size_t)a.page_tokens * HD)
-         + (size_t)(key - lp * a.page_tokens) * HD;
+  return a.pool + ((size_t)page * a.layers_in_group + a.layer) * record_elems(a) + ((size_t)g * a.page_tokens + (key - lp * a.page_tokens)) * HD;
+}
+__device__ __forceinline__ const bf16* value_row(const AttnArgs& a, const int* bt, int g, int key) {
+  int lp = key / a.page_tokens;
+  int page = max(bt[lp], 0);
+  return a.pool + ((size_t)page * a.layers_in_group + a.layer) * record_elems(a) + (size_t)a.G * a.page_tokens * HD
+         + ((size_t)g * a.page_tokens + (key - lp * a.page_tokens)) * VD;
 }
 
 // ------------------------------------------------------------------------------------ prefill
@@ -318,7 +347,7 @@ __global__ void __launch_bounds__(PF_WARPS * 32) attention_prefill_kernel(AttnAr
   const unsigned s_base = (unsigned)__cvta_generic_to_shared(smem);
   const bool biased = a.slopes != nullptr || a.qt_every > 0;
   const bool v_is_k = a.kv_planes == 1;
-  constexpr int TILE_B = PF_TK * ROWB;                         // bytes of one K (or V) tile
+  constexpr int TILE_B = PF_TK * ROWB, STAGE_B = PF_TK * (ROWB + ROWBV);       // bytes of a K tile, of K and V
 
   // Causal work grows with the block's position: a CTA takes block bx and then its mirror
   // n_blocks-1-bx, so that every CTA of an item has the same number of key tiles to go through.
@@ -365,7 +394,7 @@ __global__ void __launch_bounds__(PF_WARPS * 32) attention_prefill_kernel(AttnAr
     const int n_tiles = (k_last - k_first) / PF_TK + 1;
     auto issue = [&](int j) {
       if (j < n_tiles) {
-        unsigned ks = s_base + (j % PF_STAGES) * 2 * TILE_B, vs = ks + TILE_B;
+        unsigned ks = s_base + (j % PF_STAGES) * STAGE_B, vs = ks + TILE_B;
         int key0 = k_first + j * PF_TK;
         for (int i = threadIdx.x; i < PF_TK * CPR; i += PF_WARPS * 32) {
           int row = i / CPR, ch = i - row * CPR;
@@ -373,10 +402,17 @@ __global__ void __launch_bounds__(PF_WARPS * 32) attention_prefill_kernel(AttnAr
           if (key <= k_last) {
             const bf16* kp = key_row(a, bt, g, key) + ch * 8;
             cp_async16(ks + tile_off(row, ch), kp);
-            if (!v_is_k) cp_async16(vs + tile_off(row, ch), kp + (size_t)a.G * a.page_tokens * HD);
+            if (VD == HD && !v_is_k) cp_async16(vs + tile_off_v(row, ch), kp + (size_t)a.G * a.page_tokens * HD);
           } else {                       // past the last key: zeros, so that 0 * V stays 0
             st_shared_zero16(ks + tile_off(row, ch));
-            if (!v_is_k) st_shared_zero16(vs + tile_off(row, ch));
+            if (VD == HD && !v_is_k) st_shared_zero16(vs + tile_off_v(row, ch));
+          }
+        }
+        if (VD != HD) {
+          for (int i = threadIdx.x; i < PF_TK * CPRV; i += PF_WARPS * 32) {
+            int row = i / CPRV, ch = i - row * CPRV;
+            if (key0 + row <= k_last) cp_async16(vs + tile_off_v(row, ch), value_row(a, bt, g, key0 + row) + ch * 8);
+            else st_shared_zero16(vs + tile_off_v(row, ch));
           }
         }
       }
@@ -388,7 +424,7 @@ __global__ void __launch_bounds__(PF_WARPS * 32) attention_prefill_kernel(AttnAr
       issue(j + 1);
       cp_async_wait<1>();
       __syncthreads();
-      unsigned ks = s_base + (j % PF_STAGES) * 2 * TILE_B, vs = v_is_k ? ks : ks + TILE_B;
+      unsigned ks = s_base + (j % PF_STAGES) * STAGE_B, vs = v_is_k ? ks : ks + TILE_B;
       int key0 = k_first + j * PF_TK;
       // a warp whose rows all end before this tile has nothing to add (warp-uniform test)
       int warp_hi = pos0 + min(n_tok - 1, (warp * 16 + 15) / R);
@@ -410,9 +446,9 @@ __global__ void __launch_bounds__(PF_WARPS * 32) attention_prefill_kernel(AttnAr
       l[r] += __shfl_xor_sync(0xffffffffu, l[r], 1);
       l[r] += __shfl_xor_sync(0xffffffffu, l[r], 2);
       if (!valid[r]) continue;
-      float inv = 1.0f / l[r];
+      float inv = denominator_inv(a, g * R + hr[r], m[r], l[r]);
       if (a.gate) inv *= 1.0f / (1.0f + expf(-a.gate[(size_t)(row_begin + tok0 + tok[r]) * a.ldg + g * R + hr[r]]));
-      bf16* dst = a.out + ((size_t)(row_begin + tok0 + tok[r]) * a.H + g * R + hr[r]) * HD;
+      bf16* dst = a.out + ((size_t)(row_begin + tok0 + tok[r]) * a.H + g * R + hr[r]) * VD;
 #pragma unroll
       for (int d = 0; d < DN; ++d)
         *(unsigned*)(dst + d * 8 + 2 * c) = pack_bf16(o[d][2 * r] * inv, o[d][2 * r + 1] * inv);
@@ -428,7 +464,7 @@ __global__ void __launch_bounds__(PF_WARPS * 32) attention_prefill_kernel(AttnAr
 #define DC_MAX_PAGES 256
 
 // The warps of a decode CTA hold partial results (o, m, l) for the same 16-row block of heads over
-// different keys: they are combined through `merge` ([warp][16][HD + 2] floats of shared memory that
+// different keys: they are combined through `merge` ([warp][16][VD + 2] floats of shared memory that
 // no warp reads as a key tile any more) into the CTA's result, which goes to `out` when the CTA is the
 // only one of its (row, kv head), else into the CTA's record of the scratch buffer.
 __device__ __forceinline__ void decode_merge_records(const AttnArgs& a, const float* merge, int t, int g, int r0, int R,
@@ -437,7 +473,7 @@ __device__ __forceinline__ void decode_warps_to_cta(const AttnArgs& a, float (&o
                                                     float* merge, int warp, int lane, int t, int g, int r0, int R,
                                                     int split_index, int n_active, float* cta_rec = nullptr) {
   const int gq = lane >> 2, c = lane & 3;
-  const int SW = HD + 2;
+  const int SW = VD + 2;
 #pragma unroll
   for (int r = 0; r < 2; ++r) {
     l[r] += __shfl_xor_sync(0xffffffffu, l[r], 1);
@@ -445,18 +481,18 @@ __device__ __forceinline__ void decode_warps_to_cta(const AttnArgs& a, float (&o
     float* rec = merge + ((size_t)warp * 16 + gq + 8 * r) * SW;
 #pragma unroll
     for (int d = 0; d < DN; ++d) { rec[d * 8 + 2 * c] = o[d][2 * r]; rec[d * 8 + 2 * c + 1] = o[d][2 * r + 1]; }
-    if (c == 0) { rec[HD] = m[r]; rec[HD + 1] = l[r]; }
+    if (c == 0) { rec[VD] = m[r]; rec[VD + 1] = l[r]; }
   }
   decode_merge_records(a, merge, t, g, r0, R, split_index, n_active, cta_rec);
 }
 // The same from the keys-as-rows layout (heads 0..7 only: rows 8..15 of the records are not written and, with R <= 8,
 // not read).
-__device__ __forceinline__ void decode_warps_to_cta_keys_as_rows(const AttnArgs& a, float (&ot)[HD / 16][4], float (&m)[2],
+__device__ __forceinline__ void decode_warps_to_cta_keys_as_rows(const AttnArgs& a, float (&ot)[VD / 16][4], float (&m)[2],
                                                                  float (&l)[2], float* merge, int warp, int lane, int t,
                                                                  int g, int R, int split_index, int n_active,
                                                                  float* cta_rec = nullptr) {
   const int gq = lane >> 2, c = lane & 3;
-  const int SW = HD + 2;
+  const int SW = VD + 2;
 #pragma unroll
   for (int e = 0; e < 2; ++e) {
     l[e] += __shfl_xor_sync(0xffffffffu, l[e], 4);
@@ -464,39 +500,39 @@ __device__ __forceinline__ void decode_warps_to_cta_keys_as_rows(const AttnArgs&
     l[e] += __shfl_xor_sync(0xffffffffu, l[e], 16);
     float* rec = merge + ((size_t)warp * 16 + 2 * c + e) * SW;
 #pragma unroll
-    for (int dm = 0; dm < HD / 16; ++dm) { rec[dm * 16 + gq] = ot[dm][e]; rec[dm * 16 + gq + 8] = ot[dm][2 + e]; }
-    if (gq == 0) { rec[HD] = m[e]; rec[HD + 1] = l[e]; }
+    for (int dm = 0; dm < VD / 16; ++dm) { rec[dm * 16 + gq] = ot[dm][e]; rec[dm * 16 + gq + 8] = ot[dm][2 + e]; }
+    if (gq == 0) { rec[VD] = m[e]; rec[VD + 1] = l[e]; }
   }
   decode_merge_records(a, merge, t, g, 0, R, split_index, n_active, cta_rec);
 }
-// cta_rec: the CTA's record stays in its shared memory ([row][HD + 2] floats) for the cluster's first active CTA to
+// cta_rec: the CTA's record stays in its shared memory ([row][VD + 2] floats) for the cluster's first active CTA to
 // read, instead of going to the scratch buffer.
 __device__ __forceinline__ void decode_merge_records(const AttnArgs& a, const float* merge, int t, int g, int r0, int R,
                                                      int split_index, int n_active, float* cta_rec) {
-  const int SW = HD + 2;
+  const int SW = VD + 2;
   __syncthreads();
   const int rows_here = min(16, R - r0);
-  for (int i = threadIdx.x; i < rows_here * HD; i += DC_WARPS * 32) {
-    int row = i / HD, d = i - row * HD;
+  for (int i = threadIdx.x; i < rows_here * VD; i += DC_WARPS * 32) {
+    int row = i / VD, d = i - row * VD;
     float mx = -INFINITY;
 #pragma unroll
-    for (int w = 0; w < DC_WARPS; ++w) mx = fmaxf(mx, merge[((size_t)w * 16 + row) * SW + HD]);
+    for (int w = 0; w < DC_WARPS; ++w) mx = fmaxf(mx, merge[((size_t)w * 16 + row) * SW + VD]);
     float lt = 0.f, at = 0.f;
 #pragma unroll
     for (int w = 0; w < DC_WARPS; ++w) {
       const float* rec = merge + ((size_t)w * 16 + row) * SW;
-      float cw = rec[HD] == -INFINITY ? 0.f : exp2f(rec[HD] - mx);
-      lt += rec[HD + 1] * cw;
+      float cw = rec[VD] == -INFINITY ? 0.f : exp2f(rec[VD] - mx);
+      lt += rec[VD + 1] * cw;
       at += rec[d] * cw;
     }
     int h = g * R + r0 + row;
     if (n_active == 1) {
-      a.out[((size_t)t * a.H + h) * HD + d] = __float2bfloat16_rn(at / lt);
+      a.out[((size_t)t * a.H + h) * VD + d] = __float2bfloat16_rn(a.sinks ? at * denominator_inv(a, h, mx, lt) : at / lt);
     } else {
       float* rec = cta_rec ? cta_rec + (size_t)(r0 + row) * SW
                            : a.scratch + (((size_t)t * a.H + h) * a.max_splits + split_index) * SW;
       rec[d] = at;
-      if (d == 0) { rec[HD] = mx; rec[HD + 1] = lt; }
+      if (d == 0) { rec[VD] = mx; rec[VD + 1] = lt; }
     }
   }
   __syncthreads();
@@ -505,7 +541,7 @@ __device__ __forceinline__ void decode_merge_records(const AttnArgs& a, const fl
 // The last CTA of a (row, kv head) to get here merges the ranges' records in order.
 __device__ __forceinline__ void decode_last_cta_merges(const AttnArgs& a, int* sm_last, int t, int g, int R, int n_active) {
   if (n_active == 1) return;
-  const int SW = HD + 2;
+  const int SW = VD + 2;
   __threadfence();                                      // every writer publishes its records ...
   __syncthreads();                                      // ... before thread 0 counts this CTA in
   if (threadIdx.x == 0) {
@@ -516,19 +552,19 @@ __device__ __forceinline__ void decode_last_cta_merges(const AttnArgs& a, int* s
   __syncthreads();
   if (!*sm_last) return;
   __threadfence();
-  for (int i = threadIdx.x; i < R * HD; i += DC_WARPS * 32) {
-    int r = i / HD, d = i - r * HD;
+  for (int i = threadIdx.x; i < R * VD; i += DC_WARPS * 32) {
+    int r = i / VD, d = i - r * VD;
     int h = g * R + r;
     const float* rec = a.scratch + ((size_t)t * a.H + h) * a.max_splits * SW;
     float mx = -INFINITY;
-    for (int j = 0; j < n_active; ++j) mx = fmaxf(mx, rec[(size_t)j * SW + HD]);
+    for (int j = 0; j < n_active; ++j) mx = fmaxf(mx, rec[(size_t)j * SW + VD]);
     float lt = 0.f, at = 0.f;
     for (int j = 0; j < n_active; ++j) {
-      float cj = exp2f(rec[(size_t)j * SW + HD] - mx);
-      lt += rec[(size_t)j * SW + HD + 1] * cj;
+      float cj = exp2f(rec[(size_t)j * SW + VD] - mx);
+      lt += rec[(size_t)j * SW + VD + 1] * cj;
       at += rec[(size_t)j * SW + d] * cj;
     }
-    a.out[((size_t)t * a.H + h) * HD + d] = __float2bfloat16_rn(at / lt);
+    a.out[((size_t)t * a.H + h) * VD + d] = __float2bfloat16_rn(a.sinks ? at * denominator_inv(a, h, mx, lt) : at / lt);
   }
 }
 
@@ -559,29 +595,31 @@ __global__ void __launch_bounds__(DC_WARPS * 32) attention_decode_kernel(AttnArg
     for (int i = threadIdx.x; i < n_pg; i += DC_WARPS * 32) sm_pages[i] = bt[pg0 + i];
   pdl_wait(); FELLM_TRACE_WAITED();
   __syncthreads();
-  constexpr int TILE_B = DC_TK * ROWB;
-  const unsigned ring = (unsigned)__cvta_generic_to_shared(smem) + warp * DC_STAGES * 2 * TILE_B;
-  float* merge = (float*)smem;       // [warp][16][HD + 2], over the rings once every warp is done with them
+  constexpr int TILE_B = DC_TK * ROWB, STAGE_B = DC_TK * (ROWB + ROWBV);
+  const unsigned ring = (unsigned)__cvta_generic_to_shared(smem) + warp * DC_STAGES * STAGE_B;
+  float* merge = (float*)smem;       // [warp][16][VD + 2], over the rings once every warp is done with them
   const int cta_step = DC_WARPS * DC_TK;
   const int n_tiles = (k1 - k0 - warp * DC_TK + cta_step - 1) / cta_step;          // may be <= 0
-  const size_t page_elems = (size_t)a.page_tokens * HD;
+  const size_t record = record_elems(a), k_off = (size_t)g * a.page_tokens * HD;
+  const size_t v_off = (size_t)a.G * a.page_tokens * HD + (size_t)g * a.page_tokens * VD;
   auto issue = [&](int j) {
     if (j < n_tiles) {
-      unsigned ks = ring + (j % DC_STAGES) * 2 * TILE_B, vs = ks + TILE_B;
+      unsigned ks = ring + (j % DC_STAGES) * STAGE_B, vs = ks + TILE_B;
       int key0 = k0 + (j * DC_WARPS + warp) * DC_TK;
-      for (int i = lane; i < DC_TK * CPR; i += 32) {
-        int row = i / CPR, ch = i - row * CPR;
-        int key = key0 + row;
+      // a row's chunks of K, then of V: consecutive lanes read consecutive 16-byte pieces
+      for (int i = lane; i < DC_TK * (CPR + CPRV); i += 32) {
+        const bool is_v = i >= DC_TK * CPR;
+        const int u = is_v ? i - DC_TK * CPR : i, row = is_v ? u / CPRV : u / CPR, ch = u - row * (is_v ? CPRV : CPR);
+        const int key = key0 + row;
+        const unsigned dst = is_v ? vs + tile_off_v(row, ch) : ks + tile_off(row, ch);
         if (key < k1) {
           int lp = key / a.page_tokens;
           int page = max(pages_in_smem ? sm_pages[lp - pg0] : bt[lp], 0);      // never an address below the pool
-          const bf16* kp = a.pool + ((((size_t)page * a.layers_in_group + a.layer) * 2) * a.G + g) * page_elems
-                           + (size_t)(key - lp * a.page_tokens) * HD + ch * 8;
-          cp_async16(ks + tile_off(row, ch), kp);
-          cp_async16(vs + tile_off(row, ch), kp + (size_t)a.G * page_elems);
+          const bf16* rec = a.pool + ((size_t)page * a.layers_in_group + a.layer) * record;
+          const size_t tok = (size_t)(key - lp * a.page_tokens);
+          cp_async16(dst, rec + (is_v ? v_off + tok * VD : k_off + tok * HD) + ch * 8);
         } else {                       // past the range: zeros, so that 0 * V stays 0
-          st_shared_zero16(ks + tile_off(row, ch));
-          st_shared_zero16(vs + tile_off(row, ch));
+          st_shared_zero16(dst);
         }
       }
     }
@@ -593,7 +631,7 @@ __global__ void __launch_bounds__(DC_WARPS * 32) attention_decode_kernel(AttnArg
     for (int j = 0; j < DC_STAGES - 1; ++j) issue(j);
     unsigned qf[KS][4];
     load_q(qf, [&](int i) -> const bf16* {
-      return r0 + i < R ? a.q + ((size_t)t * a.H + g * R + r0 + i) * HD : nullptr;
+      return r0 + i < R ? a.q + (size_t)t * a.ldq + (size_t)(g * R + r0 + i) * HD : nullptr;
     }, lane);
     float o[DN][4], m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
 #pragma unroll
@@ -603,7 +641,7 @@ __global__ void __launch_bounds__(DC_WARPS * 32) attention_decode_kernel(AttnArg
       issue(j + DC_STAGES - 1);
       cp_async_wait<DC_STAGES - 1>();
       __syncwarp();
-      unsigned ks = ring + (j % DC_STAGES) * 2 * TILE_B, vs = ks + TILE_B;
+      unsigned ks = ring + (j % DC_STAGES) * STAGE_B, vs = ks + TILE_B;
       attend_tile<DC_TK / 8>(qf, ks, vs, k0 + (j * DC_WARPS + warp) * DC_TK, lo, hi, a.scale_log2, o, m, l, lane);
       __syncwarp();
     }
@@ -625,7 +663,7 @@ __global__ void __launch_bounds__(DC_WARPS * 32) attention_decode_kernel(AttnArg
 // a third of the instructions of the cp.async kernel, which stays for other head and page sizes.
 // Waits are bounded (a second): a warp that gives up sets *status = 301 and the CTA finishes with
 // what it has.
-#if HD == 64
+#if HD == 64 && VD == 64
 #define DT_PT 64
 #define DT_HALF 32                     // keys per tile: half a page, so that a warp has two tiles in flight
 #define DT_TILE_B (DT_HALF * 128)
@@ -889,7 +927,7 @@ attention_decode_tma_kernel(const __grid_constant__ CUtensorMap pool_map, AttnAr
   if constexpr (CL) {
     cluster_barrier();                                     // the records of all ranges are written
     if (active && n_active > 1 && s == s_lo) {
-      const int SW = HD + 2;
+      const int SW = VD + 2;
       const unsigned mine = (unsigned)__cvta_generic_to_shared(cta_rec);
       for (int i = threadIdx.x; i < R * HD; i += DC_WARPS * 32) {
         const int r = i / HD, d = i - r * HD;
@@ -915,7 +953,7 @@ attention_decode_tma_kernel(const __grid_constant__ CUtensorMap pool_map, AttnAr
           lt += lj[j] * cj;
           at += aj[j] * cj;
         }
-        a.out[((size_t)t * a.H + g * R + r) * HD + d] = __float2bfloat16_rn(at / lt);
+        a.out[((size_t)t * a.H + g * R + r) * HD + d] = __float2bfloat16_rn(a.sinks ? at * denominator_inv(a, g * R + r, mx, lt) : at / lt);
       }
     }
     cluster_barrier();                                     // nobody leaves while its record may be read
@@ -1032,9 +1070,9 @@ attention_prefill_tma_kernel(const __grid_constant__ CUtensorMap pool_map, AttnA
       l[r] += __shfl_xor_sync(0xffffffffu, l[r], 1);
       l[r] += __shfl_xor_sync(0xffffffffu, l[r], 2);
       if (!valid[r]) continue;
-      float inv = 1.0f / l[r];
+      float inv = denominator_inv(a, g * R + hr[r], m[r], l[r]);
       if (a.gate) inv *= 1.0f / (1.0f + expf(-a.gate[(size_t)(row_begin + tok0 + tok[r]) * a.ldg + g * R + hr[r]]));
-      bf16* dst = a.out + ((size_t)(row_begin + tok0 + tok[r]) * a.H + g * R + hr[r]) * HD;
+      bf16* dst = a.out + ((size_t)(row_begin + tok0 + tok[r]) * a.H + g * R + hr[r]) * VD;
 #pragma unroll
       for (int d = 0; d < DN; ++d)
         *(unsigned*)(dst + d * 8 + 2 * c) = pack_bf16(o[d][2 * r] * inv, o[d][2 * r + 1] * inv);
@@ -1090,11 +1128,12 @@ static int fill_args(AttnArgs& a, const void* q, const void* pool, const int* bl
   a.scale_log2 = scale * 1.4426950408889634f;
   a.item_start = nullptr; a.scratch = nullptr; a.counters = nullptr; a.split_len = 1; a.max_splits = 1; a.n_items = 0;
   a.ldq = H * HD; a.chunk = 0; a.ldg = 0; a.cap_log2 = 0.f; a.gate = nullptr;
-  a.slopes = nullptr; a.qt_coef = 0.f; a.qt_every = 0; a.kv_planes = 2;
+  a.slopes = nullptr; a.qt_coef = 0.f; a.qt_every = 0; a.kv_planes = 2; a.sinks = nullptr;
   return 0;
 }
 
 FELLM_API int fellm_attn_head_dim() { return HD; }
+FELLM_API int fellm_attn_value_dim() { return VD; }
 
 // q [T, H, hd], out [T, H*hd]; rows of item i are item_start[i]..item_start[i+1], its positions are
 // consecutive from positions[item_start[i]]; max_item_rows: the longest item of the step.
@@ -1115,13 +1154,13 @@ FELLM_API int fellm_attn_prefill_mma(const void* q, const void* pool, const int*
 }
 
 // The same with a bias by distance (slopes float32 [H], null: none), a query temperature (qt_every 0: none) and values
-// that are the keys (v_is_k: a page-layer record is the keys [G][page_tokens][hd] alone).
+// that are the keys (v_is_k: a page-layer record is the keys [G][page_tokens][hd] alone); sinks: float32 [H] or null.
 FELLM_API int fellm_attn_prefill_mma_biased(const void* q, int ldq, const void* pool, const int* block_table, int max_pages,
                                             const int* positions, const int* row_slot, const int* item_start, int n_items,
                                             int max_item_rows, void* out, int T, int H, int G, int hd, int page_tokens,
                                             int layer, int layers_in_group, float scale, int window, int chunk,
                                             float softcap, const float* gate, int ldg, const float* slopes, float qt_coef,
-                                            int qt_every, int v_is_k, cudaStream_t stream);
+                                            int qt_every, int v_is_k, const float* sinks, cudaStream_t stream);
 
 FELLM_API int fellm_attn_prefill_mma_general(const void* q, int ldq, const void* pool, const int* block_table, int max_pages,
                                              const int* positions, const int* row_slot, const int* item_start, int n_items,
@@ -1130,7 +1169,7 @@ FELLM_API int fellm_attn_prefill_mma_general(const void* q, int ldq, const void*
                                              float softcap, const float* gate, int ldg, cudaStream_t stream) {
   return fellm_attn_prefill_mma_biased(q, ldq, pool, block_table, max_pages, positions, row_slot, item_start, n_items,
                                        max_item_rows, out, T, H, G, hd, page_tokens, layer, layers_in_group, scale, window,
-                                       chunk, softcap, gate, ldg, nullptr, 0.f, 0, 0, stream);
+                                       chunk, softcap, gate, ldg, nullptr, 0.f, 0, 0, nullptr, stream);
 }
 
 FELLM_API int fellm_attn_prefill_mma_biased(const void* q, int ldq, const void* pool, const int* block_table, int max_pages,
@@ -1138,7 +1177,7 @@ FELLM_API int fellm_attn_prefill_mma_biased(const void* q, int ldq, const void* 
                                             int max_item_rows, void* out, int T, int H, int G, int hd, int page_tokens,
                                             int layer, int layers_in_group, float scale, int window, int chunk,
                                             float softcap, const float* gate, int ldg, const float* slopes, float qt_coef,
-                                            int qt_every, int v_is_k, cudaStream_t stream) {
+                                            int qt_every, int v_is_k, const float* sinks, cudaStream_t stream) {
   if (T <= 0 || n_items <= 0) return 0;
   AttnArgs a;
   int e = fill_args(a, q, pool, block_table, max_pages, positions, row_slot, out, T, H, G, hd, page_tokens, layer,
@@ -1147,13 +1186,14 @@ FELLM_API int fellm_attn_prefill_mma_biased(const void* q, int ldq, const void* 
   if (!item_start) return FELLM_ERR_ARG;
   if (ldq < H * hd || (ldq & 1) || chunk < 0 || softcap < 0.f) return FELLM_ERR_ARG;
   a.ldq = ldq; a.chunk = chunk; a.cap_log2 = softcap * 1.4426950408889634f; a.gate = gate; a.ldg = ldg;
-  if (qt_every < 0) return FELLM_ERR_ARG;
+  if (qt_every < 0 || (v_is_k && VD != HD)) return FELLM_ERR_ARG;
+  a.sinks = sinks;
   a.slopes = slopes; a.qt_coef = qt_coef; a.qt_every = qt_every; a.kv_planes = v_is_k ? 1 : 2;
   int R = H / G;
   if (R > PF_WARPS * 16) return FELLM_ERR_SIZE;
   a.item_start = item_start; a.n_items = n_items;
   int tokb = (PF_WARPS * 16) / R; if (tokb < 1) tokb = 1;
-  size_t smem = (size_t)PF_STAGES * 2 * PF_TK * ROWB;
+  size_t smem = (size_t)PF_STAGES * PF_TK * (ROWB + ROWBV);
   auto kern = attention_prefill_kernel;
   if (smem > 32 * 1024) {        // static shared memory counts against the 48 KB default too
     cudaError_t ce = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
@@ -1162,21 +1202,24 @@ FELLM_API int fellm_attn_prefill_mma_biased(const void* q, int ldq, const void* 
   return launch_k_class(launch_class_for_rows(T, 0), kern, dim3((ceil_div(max_item_rows, tokb) + 1) / 2, G, n_items), dim3(PF_WARPS * 32), smem, stream, 1, a);
 }
 
-// One query row per item.  scratch: float32 [T*H*max_splits*(hd+2)]; counters: int32 [T*G], zero
-// before the first launch (the kernel leaves them zero).  max_splits >= ceil(longest context / split_len).
-FELLM_API int fellm_attn_decode_mma(const void* q, const void* pool, const int* block_table, int max_pages,
+// One query row per item (head h of row t at q + t ldq + h hd).  scratch: float32 [T*H*max_splits*(VD+2)]; counters: int32 [T*G], zero
+// before the first launch (the kernel leaves them zero).  max_splits >= ceil(longest context / split_len).  sinks: float32
+// [H] or null.
+FELLM_API int fellm_attn_decode_mma(const void* q, int ldq, const void* pool, const int* block_table, int max_pages,
                                     const int* positions, const int* row_slot, void* out, float* scratch,
                                     int* counters, int T, int H, int G, int hd, int page_tokens, int layer,
                                     int layers_in_group, float scale, int window, int split_len, int max_splits,
-                                    cudaStream_t stream) {
+                                    const float* sinks, cudaStream_t stream) {
   if (T <= 0) return 0;
   AttnArgs a;
   int e = fill_args(a, q, pool, block_table, max_pages, positions, row_slot, out, T, H, G, hd, page_tokens, layer,
                     layers_in_group, scale, window);
   if (e) return e;
+  if (ldq < H * hd || (ldq & 1)) return FELLM_ERR_ARG;
+  a.ldq = ldq; a.sinks = sinks;
   if (!scratch || !counters || split_len < 1 || max_splits < 1) return FELLM_ERR_ARG;
   a.scratch = scratch; a.counters = counters; a.split_len = split_len; a.max_splits = max_splits;
-  size_t ring = (size_t)DC_WARPS * DC_STAGES * 2 * DC_TK * ROWB, mrg = (size_t)DC_WARPS * 16 * (HD + 2) * sizeof(float);
+  size_t ring = (size_t)DC_WARPS * DC_STAGES * DC_TK * (ROWB + ROWBV), mrg = (size_t)DC_WARPS * 16 * (VD + 2) * sizeof(float);
   size_t smem = ring > mrg ? ring : mrg;
   auto kern = attention_decode_kernel;
   if (smem > 32 * 1024) {        // static shared memory counts against the 48 KB default too
@@ -1199,7 +1242,7 @@ FELLM_API int fellm_attn_decode_tma(const void* q, const void* pool, long long n
                                     int layer, int layers_in_group, float scale, int window, int split_len,
                                     int max_splits, int* status, const void* qkv, const float* q_w, const float* k_w,
                                     float eps, const float* inv_freq, int pairing, int stages, cudaStream_t stream) {
-#if HD == 64
+#if HD == 64 && VD == 64
   if (T <= 0) return 0;
   AttnArgs a;
   if (!q) q = qkv;
@@ -1268,7 +1311,7 @@ FELLM_API int fellm_attn_prefill_tma(const void* q, const void* pool, long long 
                                      int n_items, int max_item_rows, void* out, int T, int H, int G, int hd,
                                      int page_tokens, int layer, int layers_in_group, float scale, int window,
                                      int* status, cudaStream_t stream) {
-#if HD == 64
+#if HD == 64 && VD == 64
   if (T <= 0 || n_items <= 0) return 0;
   AttnArgs a;
   int e = fill_args(a, q, pool, block_table, max_pages, positions, row_slot, out, T, H, G, hd, page_tokens, layer,

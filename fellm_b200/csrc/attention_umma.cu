@@ -1,11 +1,15 @@
-// Causal attention of prompt portions over the paged cache on the Blackwell tensor path: head size
-// 64, pages of 64 tokens, no window.  A CTA takes 128 rows (token, head of one kv head's group) and
+// Causal attention of prompt portions over the paged cache on the Blackwell tensor path: pages of 64
+// tokens, no window, compiled for one size of keys and one of values (-DAU_KD, -DAU_VD: multiples of
+// 16, 64 by default; what fits shared and tensor memory, AU_FITS below).  A CTA takes 128 rows (token, head of one kv head's group) and
 // walks over the pages of keys up to its last token:
 //   S = Q K^T      tcgen05.mma 128x64x16 (kind::f16), Q and the K page K-major in shared memory
-//                  (128-byte swizzle; the page comes by one bulk tensor copy), S in tensor memory;
+//                  (128-byte swizzle, 64 elements of a row an atom; a bulk tensor copy an atom; what
+//                  an atom has beyond the key's size comes as zeros), S in tensor memory;
 //   softmax        a row a thread: tcgen05.ld of the row's 64 scores, maximum and sum in registers
 //                  with no shuffles, P rounded to bfloat16 into shared memory;
 //   O += P V       tcgen05.mma with the V page as the MN-major operand, accumulated in tensor memory.
+// A sink per head (a.sinks): exp(sink) joins the softmax's denominator once, with no key and no value.
+// A page-layer record of the pool is the keys [G][64][AU_KD], then the values [G][64][AU_VD].
 // The accumulator is scaled by 2^-m with m a row's REFERENCE maximum, which moves only when a tile's
 // maximum exceeds it by 2^8: only then is the accumulator read, scaled and written back.
 // Two groups of four softmax warps take the even and the odd pages, each with its own reference,
@@ -29,22 +33,39 @@
 
 #include "common.cuh"
 
-#define AU_HD 64
+#ifndef AU_KD
+#define AU_KD 64
+#endif
+#ifndef AU_VD
+#define AU_VD 64
+#endif
 #define AU_PT 64                       // keys per tile: a page
 #define AU_ROWS 128
-#define AU_STAGES 6                    // pages in flight: the scores run two tiles a group ahead of the softmax
 #ifndef AU_GROUPS
 #define AU_GROUPS 2                    // softmax groups of four warps; group g takes pages g, g + AU_GROUPS, ...
 #endif
 #define AU_THREADS (64 + 128 * AU_GROUPS)
-#define AU_TILE_B (AU_PT * 128)        // bytes of one K (or V) page tile
+#define AU_ATOM_B (AU_PT * 128)        // bytes of 64 elements of a page's keys (or values)
+#define AU_KA ((AU_KD + 63) / 64)      // atoms of a key, of a value
+#define AU_VA ((AU_VD + 63) / 64)
+#define AU_QATOM_B (AU_ROWS * 128)     // bytes of 64 elements of the CTA's query rows
+#define AU_STAGE_B ((AU_KA + AU_VA) * AU_ATOM_B)
+#define AU_VC ((AU_VD + 31) / 32)      // 32-column pieces of the accumulator
+#define AU_FIXED_B (AU_KA * AU_QATOM_B + 2 * AU_GROUPS * AU_ROWS * 128)       // Q and the P tiles
+#define AU_ROOM_B (225 * 1024)
+// pages in flight: the scores run two tiles a group ahead of the softmax, so at least 2 * AU_GROUPS
+#define AU_FIT_STAGES ((AU_ROOM_B - AU_FIXED_B) / AU_STAGE_B)
+#define AU_STAGES (AU_FIT_STAGES > 6 ? 6 : AU_FIT_STAGES)
+#define AU_FITS (AU_KD % 16 == 0 && AU_VD % 16 == 0 && AU_KD >= 16 && AU_VD >= 16 && AU_FIT_STAGES >= 2 * AU_GROUPS && 2 * AU_GROUPS * AU_PT + AU_GROUPS * AU_VC * 32 <= 512)
+static_assert(AU_FITS, "key and value sizes the tcgen05 prefill attention takes");
 #define AU_WAIT_NS 1000000000ull
 #define AU_SPIN_LIMIT (1u << 26)
 
 struct AuArgs {
   const bf16* q; const int* block_table; const int* positions; const int* row_slot; const int* item_start;
   bf16* out; int* status;
-  int max_pages, H, G, layer, layers_in_group;
+  const float* sinks;                  // [H] or null
+  int max_pages, H, G, layer, layers_in_group, ldq;
   float scale_log2;
 };
 
@@ -85,9 +106,9 @@ __device__ __forceinline__ bool au_wait(unsigned bar, unsigned parity, volatile 
   if (status) atomicExch(status, code);
   return false;
 }
-__device__ __forceinline__ void au_tma_load_2d(unsigned dst, const CUtensorMap* map, int c0, int c1, unsigned bar) {
-  asm volatile("cp.async.bulk.tensor.2d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%3, %4}], [%2];\n"
-               ::"r"(dst), "l"(map), "r"(bar), "r"(c0), "r"(c1) : "memory");
+__device__ __forceinline__ void au_tma_load_3d(unsigned dst, const CUtensorMap* map, int c0, int c1, int c2, unsigned bar) {
+  asm volatile("cp.async.bulk.tensor.3d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%3, %4, %5}], [%2];\n"
+               ::"r"(dst), "l"(map), "r"(bar), "r"(c0), "r"(c1), "r"(c2) : "memory");
 }
 // Operand tile with rows of 128 bytes under the 128-byte swizzle, groups of 8 rows 1024 bytes apart:
 // K-major (the rows are M or N, the 128 bytes run along K) or MN-major (the rows are K, the 128
@@ -95,7 +116,7 @@ __device__ __forceinline__ void au_tma_load_2d(unsigned dst, const CUtensorMap* 
 __device__ __forceinline__ unsigned long long au_desc(unsigned smem_addr, bool mn_major = false) {
   unsigned long long d = 0;
   d |= (unsigned long long)((smem_addr & 0x3FFFF) >> 4);          // start address
-  if (mn_major) d |= (unsigned long long)(8192 >> 4) << 16;       // leading byte offset: the next 64 elements of MN (there are none here)
+  if (mn_major) d |= (unsigned long long)(AU_ATOM_B >> 4) << 16;       // leading byte offset: the next 64 elements of MN (the next atom)
   d |= (unsigned long long)(1024 >> 4) << 32;                     // stride byte offset: the next group of 8 rows
   d |= 1ull << 46;                                                // descriptor version (sm_100)
   d |= 2ull << 61;                                                // SWIZZLE_128B
@@ -158,12 +179,11 @@ __device__ __forceinline__ float au_ex2(float x) {
 #define AU_COL_S 0
 #define AU_COL_O (2 * AU_GROUPS * AU_PT)
 #define AU_TMEM_COLS 512
-static_assert(3 * AU_GROUPS * 64 <= AU_TMEM_COLS, "tensor memory: 192 columns a group");
-#define AU_MERGE_STRIDE (AU_HD + 2)    // floats of a row's record in the merge buffer: o, m, l
+#define AU_MERGE_STRIDE (AU_VD + 2)    // floats of a row's record in the merge buffer: o, m, l
 #define AU_RESCALE_AT 8.0f             // a row's reference maximum moves when a tile's maximum is 2^8 above it
 
 __global__ void __launch_bounds__(AU_THREADS, 1)
-attention_prefill_umma_kernel(const __grid_constant__ CUtensorMap pool_map, AuArgs a) {
+attention_prefill_umma_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_constant__ CUtensorMap v_map, AuArgs a) {
   FELLM_TRACE_SCOPE(TRACE_ATTENTION_PREFILL);
   extern __shared__ unsigned char smem_raw[];
   // full[STAGES], empty[STAGES], q_ready, s_full[GROUPS][2], p_full[GROUPS][2], o_full[GROUPS][2]: a barrier
@@ -189,8 +209,8 @@ attention_prefill_umma_kernel(const __grid_constant__ CUtensorMap pool_map, AuAr
 
   const unsigned base = (au_smem(smem_raw) + 1023u) & ~1023u;  // the swizzle is by address
   unsigned char* base_ptr = smem_raw + (base - au_smem(smem_raw));
-  const unsigned q_s = base, p_s0 = base + AU_ROWS * 128, stage0 = base + (1 + 2 * AU_GROUPS) * AU_ROWS * 128;
-  float* merge = (float*)(base_ptr + AU_ROWS * 128);           // over the P tiles and the stages, once every MMA is done
+  const unsigned q_s = base, p_s0 = base + AU_KA * AU_QATOM_B, stage0 = base + AU_FIXED_B;
+  float* merge = (float*)(base_ptr + AU_KA * AU_QATOM_B);           // over the P tiles and the stages, once every MMA is done
   const unsigned full0 = au_smem(&bars[0]), empty0 = au_smem(&bars[AU_STAGES]);
   const unsigned q_ready = au_smem(&bars[2 * AU_STAGES]), s_full0 = q_ready + 8, p_full0 = s_full0 + 16 * AU_GROUPS,
                  o_full0 = p_full0 + 16 * AU_GROUPS;
@@ -221,26 +241,29 @@ attention_prefill_umma_kernel(const __grid_constant__ CUtensorMap pool_map, AuAr
         const int s = j % AU_STAGES;
         if (j >= AU_STAGES && !au_wait(empty0 + 8 * s, (j / AU_STAGES - 1) & 1, fail, a.status, 311)) break;
         const int page = max(bt[j], 0);                        // an unmapped entry (-1) must never become an address
-        const int row = (((page * a.layers_in_group + a.layer) * 2) * a.G + g) * AU_PT;      // < 2^31: the launcher checks
-        const unsigned dst = stage0 + s * 2 * AU_TILE_B;
-        au_mbar_expect_tx(full0 + 8 * s, 2 * AU_TILE_B);
-        au_tma_load_2d(dst, &pool_map, 0, row, full0 + 8 * s);
-        au_tma_load_2d(dst + AU_TILE_B, &pool_map, 0, row + a.G * AU_PT, full0 + 8 * s);
+        const int rec = page * a.layers_in_group + a.layer;
+        const unsigned dst = stage0 + s * AU_STAGE_B;
+        au_mbar_expect_tx(full0 + 8 * s, AU_STAGE_B);
+#pragma unroll
+        for (int i = 0; i < AU_KA; ++i) au_tma_load_3d(dst + i * AU_ATOM_B, &k_map, 64 * i, g * AU_PT, rec, full0 + 8 * s);
+#pragma unroll
+        for (int i = 0; i < AU_VA; ++i) au_tma_load_3d(dst + (AU_KA + i) * AU_ATOM_B, &v_map, 64 * i, g * AU_PT, rec, full0 + 8 * s);
       }
     }
   } else if (warp == 1) {
     if (lane == 0) {
       // tile j belongs to softmax group j % GROUPS: its score tile, P tile, accumulator and barriers
-      const unsigned idesc_s = au_idesc(AU_ROWS, AU_PT, false), idesc_o = au_idesc(AU_ROWS, AU_HD, true);
+      const unsigned idesc_s = au_idesc(AU_ROWS, AU_PT, false), idesc_o = au_idesc(AU_ROWS, AU_VD, true);
       const unsigned long long dq = au_desc(q_s);
       auto scores = [&](int j) -> bool {                       // S_j = Q K_j^T into the group's score tile (j / GROUPS) & 1
         const int s = j % AU_STAGES, grp = j % AU_GROUPS, sb = (j / AU_GROUPS) & 1;
         if (!au_wait(full0 + 8 * s, (j / AU_STAGES) & 1, fail, a.status, 312)) return false;
         asm volatile("tcgen05.fence::after_thread_sync;\n" ::: "memory");
-        const unsigned long long dk = au_desc(stage0 + s * 2 * AU_TILE_B);
+        const unsigned long long dk = au_desc(stage0 + s * AU_STAGE_B);
 #pragma unroll
-        for (int k = 0; k < AU_HD / 16; ++k)                   // 32 bytes further along the head inside the swizzle atom
-          au_mma(tmem_base + AU_COL_S + (2 * grp + sb) * AU_PT, dq + (unsigned long long)(k * 2), dk + (unsigned long long)(k * 2), idesc_s, k ? 1u : 0u);
+        for (int k = 0; k < AU_KD / 16; ++k)                   // 32 bytes further along the head inside the swizzle atom; four steps an atom
+          au_mma(tmem_base + AU_COL_S + (2 * grp + sb) * AU_PT, dq + (unsigned long long)((k >> 2) * (AU_QATOM_B >> 4) + (k & 3) * 2),
+                 dk + (unsigned long long)((k >> 2) * (AU_ATOM_B >> 4) + (k & 3) * 2), idesc_s, k ? 1u : 0u);
         au_commit(s_full0 + 16 * grp + 8 * sb);
         return true;
       };
@@ -254,10 +277,10 @@ attention_prefill_umma_kernel(const __grid_constant__ CUtensorMap pool_map, AuAr
         if (!ok) break;
         asm volatile("tcgen05.fence::after_thread_sync;\n" ::: "memory");
         const unsigned long long dp = au_desc(p_s0 + (2 * grp + (i & 1)) * AU_ROWS * 128);
-        const unsigned long long dv = au_desc(stage0 + s * 2 * AU_TILE_B + AU_TILE_B, true);
+        const unsigned long long dv = au_desc(stage0 + s * AU_STAGE_B + AU_KA * AU_ATOM_B, true);
 #pragma unroll
         for (int k = 0; k < AU_PT / 16; ++k)                   // 16 keys further: 32 bytes along P's rows, 16 rows (2048 bytes) down V
-          au_mma(tmem_base + AU_COL_O + grp * AU_HD, dp + (unsigned long long)(k * 2), dv + (unsigned long long)(k * 128), idesc_o,
+          au_mma(tmem_base + AU_COL_O + grp * AU_VC * 32, dp + (unsigned long long)(k * 2), dv + (unsigned long long)(k * 128), idesc_o,
                  (i | k) ? 1u : 0u);                           // the group's first tile starts its accumulator
         au_commit(o_full0 + 16 * grp + 8 * (i & 1));
         au_commit(empty0 + 8 * s);                             // the page's stage is free once these MMAs have read it
@@ -270,17 +293,18 @@ attention_prefill_umma_kernel(const __grid_constant__ CUtensorMap pool_map, AuAr
     const int tok = row / R, head = row - tok * R;
     const bool valid = tok < n_tok;
     const int pos = pos0 + tok;
-    const size_t out_row = ((size_t)(row_begin + tok0 + tok) * a.H + g * R + head) * AU_HD;
+    const size_t out_row = ((size_t)(row_begin + tok0 + tok) * a.H + g * R + head) * AU_VD;
     if (grp == 0) {
-      const uint4* src = (const uint4*)(a.q + out_row);
+      const uint4* src = (const uint4*)(a.q + (size_t)(row_begin + tok0 + tok) * a.ldq + (size_t)(g * R + head) * AU_KD);
 #pragma unroll
-      for (int ch = 0; ch < 8; ++ch) au_st_shared16(q_s + au_off(row, ch), valid ? src[ch] : make_uint4(0, 0, 0, 0));
+      for (int ch = 0; ch < AU_KD / 8; ++ch)
+        au_st_shared16(q_s + (ch >> 3) * AU_QATOM_B + au_off(row, ch & 7), valid ? src[ch] : make_uint4(0, 0, 0, 0));
       asm volatile("fence.proxy.async.shared::cta;\n" ::: "memory");    // these writes before the MMA's reads
       __syncwarp();
       if (lane == 0) au_mbar_arrive(q_ready);
     }
     const unsigned t_row = tmem_base + ((unsigned)(qd * 32) << 16);
-    const unsigned t_acc = t_row + AU_COL_O + grp * AU_HD;
+    const unsigned t_acc = t_row + AU_COL_O + grp * AU_VC * 32;
     const unsigned s_full = s_full0 + 16 * grp, p_full = p_full0 + 16 * grp, o_full = o_full0 + 16 * grp;
     const float scale = a.scale_log2;
     // The accumulator of P V stays in tensor memory, scaled by 2^-m where m is the row's REFERENCE
@@ -295,9 +319,11 @@ attention_prefill_umma_kernel(const __grid_constant__ CUtensorMap pool_map, AuAr
         // rows past the last key hold whatever the page held before: zero the V rows, so that 0 * V is 0
         ok = au_wait(full0 + 8 * s, (j / AU_STAGES) & 1, fail, a.status, 315);
         if (!ok) break;
-        const unsigned v_s = stage0 + s * 2 * AU_TILE_B + AU_TILE_B;
-        for (int e = (k_last + 1 - key0) * 8 + row; e < AU_PT * 8; e += AU_ROWS)
-          au_st_shared16(v_s + au_off(e >> 3, e & 7), make_uint4(0, 0, 0, 0));
+        const unsigned v_s = stage0 + s * AU_STAGE_B + AU_KA * AU_ATOM_B;
+        for (int e = (k_last + 1 - key0) * 8 + row; e < AU_PT * 8; e += AU_ROWS) {
+#pragma unroll
+          for (int i = 0; i < AU_VA; ++i) au_st_shared16(v_s + i * AU_ATOM_B + au_off(e >> 3, e & 7), make_uint4(0, 0, 0, 0));
+        }
       }
       ok = au_wait(s_full + 8 * (i & 1), (i >> 1) & 1, fail, a.status, 316);
       if (!ok) break;
@@ -350,7 +376,7 @@ attention_prefill_umma_kernel(const __grid_constant__ CUtensorMap pool_map, AuAr
         if (!ok) break;
         asm volatile("tcgen05.fence::after_thread_sync;\n" ::: "memory");
 #pragma unroll
-        for (int hlf = 0; hlf < 2; ++hlf) {
+        for (int hlf = 0; hlf < AU_VC; ++hlf) {
           float ot[32];
           au_tmem_ld32(t_acc + 32 * hlf, ot);
 #pragma unroll
@@ -368,19 +394,19 @@ attention_prefill_umma_kernel(const __grid_constant__ CUtensorMap pool_map, AuAr
       __syncwarp();
       if (lane == 0) au_mbar_arrive(p_full + 8 * (i & 1));
     }
-    float o[AU_HD];
+    float o[AU_VC * 32];
     if (ok && n_mine > 0) {
       ok = au_wait(o_full + 8 * ((n_mine - 1) & 1), ((n_mine - 1) >> 1) & 1, fail, a.status, 317);
       if (ok) {
         asm volatile("tcgen05.fence::after_thread_sync;\n" ::: "memory");
-        au_tmem_ld32_issue(t_acc, o);
-        au_tmem_ld32_issue(t_acc + 32, o + 32);
+#pragma unroll
+        for (int i = 0; i < AU_VC; ++i) au_tmem_ld32_issue(t_acc + 32 * i, o + 32 * i);
         au_tmem_ld_wait();
       }
     }
     if (n_mine == 0 || !ok) {
 #pragma unroll
-      for (int d = 0; d < AU_HD; ++d) o[d] = 0.f;
+      for (int d = 0; d < AU_VD; ++d) o[d] = 0.f;
     }
     // Every group is through its last tile: every MMA and every copy of this CTA is done, and the P
     // tiles and stages are free for the later groups' records.  (A group that gave up still comes to
@@ -389,30 +415,33 @@ attention_prefill_umma_kernel(const __grid_constant__ CUtensorMap pool_map, AuAr
     if (grp > 0) {
       float* rec = merge + ((size_t)(grp - 1) * AU_ROWS + row) * AU_MERGE_STRIDE;
 #pragma unroll
-      for (int d = 0; d < AU_HD; ++d) rec[d] = o[d];
-      rec[AU_HD] = m; rec[AU_HD + 1] = l;
+      for (int d = 0; d < AU_VD; ++d) rec[d] = o[d];
+      rec[AU_VD] = m; rec[AU_VD + 1] = l;
     }
     asm volatile("bar.sync 1, %0;\n" ::"n"(128 * AU_GROUPS) : "memory");
     if (grp == 0 && ok && !*fail && valid) {
       float mm = m;                                            // group 0 has page 0: m is finite
 #pragma unroll
-      for (int q = 0; q < AU_GROUPS - 1; ++q) mm = fmaxf(mm, merge[((size_t)q * AU_ROWS + row) * AU_MERGE_STRIDE + AU_HD]);
+      for (int q = 0; q < AU_GROUPS - 1; ++q) mm = fmaxf(mm, merge[((size_t)q * AU_ROWS + row) * AU_MERGE_STRIDE + AU_VD]);
+      const float sk = a.sinks ? a.sinks[g * R + head] * 1.4426950408889634f : -INFINITY;
+      mm = fmaxf(mm, sk);
       const float c0 = au_ex2(m - mm);
       float lt = l * c0;
+      if (a.sinks) lt += au_ex2(sk - mm);                      // one more term of the denominator
 #pragma unroll
-      for (int d = 0; d < AU_HD; ++d) o[d] *= c0;
+      for (int d = 0; d < AU_VD; ++d) o[d] *= c0;
 #pragma unroll
       for (int q = 0; q < AU_GROUPS - 1; ++q) {
         const float* rec = merge + ((size_t)q * AU_ROWS + row) * AU_MERGE_STRIDE;
-        const float mq = rec[AU_HD], cq = (mq == -INFINITY) ? 0.f : au_ex2(mq - mm);
-        lt = fmaf(rec[AU_HD + 1], cq, lt);
+        const float mq = rec[AU_VD], cq = (mq == -INFINITY) ? 0.f : au_ex2(mq - mm);
+        lt = fmaf(rec[AU_VD + 1], cq, lt);
 #pragma unroll
-        for (int d = 0; d < AU_HD; ++d) o[d] = fmaf(rec[d], cq, o[d]);
+        for (int d = 0; d < AU_VD; ++d) o[d] = fmaf(rec[d], cq, o[d]);
       }
       const float inv = 1.0f / lt;
       uint4* dst = (uint4*)(a.out + out_row);
 #pragma unroll
-      for (int ch = 0; ch < 8; ++ch) {
+      for (int ch = 0; ch < AU_VD / 8; ++ch) {
         __nv_bfloat162 q0 = __floats2bfloat162_rn(o[8 * ch] * inv, o[8 * ch + 1] * inv), q1 = __floats2bfloat162_rn(o[8 * ch + 2] * inv, o[8 * ch + 3] * inv);
         __nv_bfloat162 q2 = __floats2bfloat162_rn(o[8 * ch + 4] * inv, o[8 * ch + 5] * inv), q3 = __floats2bfloat162_rn(o[8 * ch + 6] * inv, o[8 * ch + 7] * inv);
         dst[ch] = make_uint4(*(unsigned*)&q0, *(unsigned*)&q1, *(unsigned*)&q2, *(unsigned*)&q3);
@@ -428,18 +457,18 @@ attention_prefill_umma_kernel(const __grid_constant__ CUtensorMap pool_map, AuAr
   }
 }
 
-// The cache pool as a 2-D tensor [rows of 64 dims], a page of one kv head (64 rows) a box: the map is
-// kept per (pool, rows).
+// A page-layer record's keys (or values) as a 3-D tensor [elements of a head, rows of all heads, records]: a box is
+// 64 elements of the 64 rows of one kv head.  Kept per (base, records, G).
 typedef CUresult (*AuEncodeTiledFn)(CUtensorMap*, CUtensorMapDataType, cuuint32_t, void*, const cuuint64_t*, const cuuint64_t*,
                                     const cuuint32_t*, const cuuint32_t*, CUtensorMapInterleave, CUtensorMapSwizzle,
                                     CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
-static int au_pool_map(const void* pool, long long rows, CUtensorMap* out) {
+static int au_pool_map(const bf16* base, int size, long long records, int G, CUtensorMap* out) {
   static std::mutex mu;
-  static struct { const void* pool; long long rows; CUtensorMap map; } cache[8];
+  static struct { const void* base; long long records; int G, size; CUtensorMap map; } cache[16];
   static int n_cached = 0, next = 0;
   std::lock_guard<std::mutex> lock(mu);
   for (int i = 0; i < n_cached; ++i)
-    if (cache[i].pool == pool && cache[i].rows == rows) { *out = cache[i].map; return 0; }
+    if (cache[i].base == base && cache[i].records == records && cache[i].G == G && cache[i].size == size) { *out = cache[i].map; return 0; }
   static AuEncodeTiledFn fn = nullptr;
   if (!fn) {
     void* p = nullptr;
@@ -448,54 +477,58 @@ static int au_pool_map(const void* pool, long long rows, CUtensorMap* out) {
       return FELLM_ERR_ARG;
     fn = (AuEncodeTiledFn)p;
   }
-  cuuint64_t dims[2] = {(cuuint64_t)AU_HD, (cuuint64_t)rows};
-  cuuint64_t strides[1] = {(cuuint64_t)AU_HD * 2};
-  cuuint32_t box[2] = {AU_HD, AU_PT};
-  cuuint32_t estr[2] = {1, 1};
+  cuuint64_t dims[3] = {(cuuint64_t)size, (cuuint64_t)G * AU_PT, (cuuint64_t)records};
+  cuuint64_t strides[2] = {(cuuint64_t)size * 2, (cuuint64_t)G * AU_PT * (AU_KD + AU_VD) * 2};
+  cuuint32_t box[3] = {64, AU_PT, 1};
+  cuuint32_t estr[3] = {1, 1, 1};
   CUtensorMap m;
-  CUresult r = fn(&m, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void*>(pool), dims, strides, box, estr,
+  CUresult r = fn(&m, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, const_cast<bf16*>(base), dims, strides, box, estr,
                   CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_128B,
                   CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
   if (r != CUDA_SUCCESS) return 1000 + (int)r;
-  cache[next].pool = pool; cache[next].rows = rows; cache[next].map = m;
-  next = (next + 1) % 8;
-  if (n_cached < 8) ++n_cached;
+  cache[next].base = base; cache[next].records = records; cache[next].G = G; cache[next].size = size; cache[next].map = m;
+  next = (next + 1) % 16;
+  if (n_cached < 16) ++n_cached;
   *out = m;
   return 0;
 }
 
 // Whether fellm_attn_prefill_umma takes these sizes (1) or not (0).
-FELLM_API int fellm_attn_prefill_umma_takes(int H, int G, int hd, int page_tokens, int window) {
+FELLM_API int fellm_attn_prefill_umma_takes(int H, int G, int hd, int vd, int page_tokens, int window) {
   if (G < 1 || H % G) return 0;
   const int R = H / G;
-  return (hd == AU_HD && page_tokens == AU_PT && window <= 0 && R <= AU_ROWS && AU_ROWS % R == 0) ? 1 : 0;
+  return (hd == AU_KD && vd == AU_VD && page_tokens == AU_PT && window <= 0 && R <= AU_ROWS && AU_ROWS % R == 0) ? 1 : 0;
 }
 
-// q [T, H, 64] bfloat16 (normed, rotated), out [T, H*64]; pool [n_pages, layers_in_group, 2, G, 64, 64];
-// rows of item i are item_start[i]..item_start[i+1], its positions are consecutive from
-// positions[item_start[i]]; max_item_rows: the longest item of the step.  status: device int32 that a
-// role sets (311..317) if a wait ran out.  FELLM_ERR_SIZE for sizes it does not take.
-FELLM_API int fellm_attn_prefill_umma(const void* q, const void* pool, long long n_pages, const int* block_table,
+// q [T, ldq] bfloat16, head h at column h hd (rotated; normed where the layer norms), out [T, H*vd]; pool [n_pages,
+// layers_in_group, record], a record being the keys [G][64][hd] and then the values [G][64][vd]; rows of item i are
+// item_start[i]..item_start[i+1], its positions are consecutive from positions[item_start[i]]; max_item_rows: the longest
+// item of the step.  sinks: float32 [H] or null.  status: device int32 that a role sets (311..317) if a wait ran out.
+// FELLM_ERR_SIZE for sizes it does not take.
+FELLM_API int fellm_attn_prefill_umma(const void* q, int ldq, const void* pool, long long n_pages, const int* block_table,
                                       int max_pages, const int* positions, const int* row_slot, const int* item_start,
-                                      int n_items, int max_item_rows, void* out, int T, int H, int G, int hd,
+                                      int n_items, int max_item_rows, void* out, int T, int H, int G, int hd, int vd,
                                       int page_tokens, int layer, int layers_in_group, float scale, int window,
-                                      int* status, cudaStream_t stream) {
+                                      const float* sinks, int* status, cudaStream_t stream) {
   if (T <= 0 || n_items <= 0) return 0;
   if (!q || !pool || !block_table || !positions || !row_slot || !item_start || !out) return FELLM_ERR_ARG;
-  if (!fellm_attn_prefill_umma_takes(H, G, hd, page_tokens, window)) return FELLM_ERR_SIZE;
-  const long long rows = n_pages * layers_in_group * 2 * G * page_tokens;
-  if (rows >= (1ll << 31) || ((uintptr_t)pool & 15) || ((uintptr_t)q & 15) || ((uintptr_t)out & 15)) return FELLM_ERR_SIZE;
+  if (!fellm_attn_prefill_umma_takes(H, G, hd, vd, page_tokens, window)) return FELLM_ERR_SIZE;
+  if (!(scale > 0.f)) return FELLM_ERR_ARG;                    // a row's maximum is taken of the unscaled scores
+  const long long records = n_pages * layers_in_group;
+  if (records >= (1ll << 31) || ldq < H * hd || (ldq % 8) || ((uintptr_t)pool & 15) || ((uintptr_t)q & 15) || ((uintptr_t)out & 15))
+    return FELLM_ERR_SIZE;
   AuArgs a;
-  a.q = (const bf16*)q; a.block_table = block_table; a.positions = positions; a.row_slot = row_slot; a.item_start = item_start;
-  a.out = (bf16*)out; a.status = status; a.max_pages = max_pages; a.H = H; a.G = G; a.layer = layer;
+  a.q = (const bf16*)q; a.ldq = ldq; a.block_table = block_table; a.positions = positions; a.row_slot = row_slot; a.item_start = item_start;
+  a.out = (bf16*)out; a.status = status; a.sinks = sinks; a.max_pages = max_pages; a.H = H; a.G = G; a.layer = layer;
   a.layers_in_group = layers_in_group; a.scale_log2 = scale * 1.4426950408889634f;
-  CUtensorMap map;
-  int e = au_pool_map(pool, rows, &map);
+  CUtensorMap k_map, v_map;
+  int e = au_pool_map((const bf16*)pool, AU_KD, records, G, &k_map);
+  if (!e) e = au_pool_map((const bf16*)pool + (size_t)G * AU_PT * AU_KD, AU_VD, records, G, &v_map);
   if (e) return e;
   const int tokb = AU_ROWS / (H / G);
-  size_t smem = (size_t)(1 + 2 * AU_GROUPS) * AU_ROWS * 128 + (size_t)AU_STAGES * 2 * AU_TILE_B + 1024;     // Q, the P tiles, the stages
+  size_t smem = (size_t)AU_FIXED_B + (size_t)AU_STAGES * AU_STAGE_B + 1024;     // Q, the P tiles, the stages
   auto kern = attention_prefill_umma_kernel;
   cudaError_t ce = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
   if (ce != cudaSuccess) return (int)ce;
-  return launch_k_class(launch_class_for_rows(T, 0), kern, dim3(ceil_div(max_item_rows, tokb) * G, 1, n_items), dim3(AU_THREADS), smem, stream, 1, map, a);
+  return launch_k_class(launch_class_for_rows(T, 0), kern, dim3(ceil_div(max_item_rows, tokb) * G, 1, n_items), dim3(AU_THREADS), smem, stream, 1, k_map, v_map, a);
 }

@@ -12,7 +12,7 @@
 #define BN 64
 #define BK 16
 
-// EPI 0: C = acc (+bias);  EPI 1: C(float) = C + acc (+bias)   (residual accumulate)
+// EPI 0: C = acc (+bias);  EPI 2: C = max(acc (+bias), 0)^2;  EPI 1: C(float) = C + acc (+bias)   (residual accumulate)
 template <typename TA, typename TW, typename TO, int EPI>
 __global__ void __launch_bounds__(256)
 gemm_tn_simt_kernel(const TA* __restrict__ A, const TW* __restrict__ W, const float* __restrict__ bias,
@@ -67,6 +67,7 @@ gemm_tn_simt_kernel(const TA* __restrict__ A, const TW* __restrict__ W, const fl
       if (gn >= N) continue;
       float v = acc[i][j];
       if (bias) v += bias[gn];
+      if (EPI == 2) { v = fmaxf(v, 0.f); v *= v; }
       size_t o = (size_t)gm * ldc + gn;
       if (EPI == 1) C[o] = from_f<TO>(to_f(C[o]) + v);
       else C[o] = from_f<TO>(v);
@@ -76,30 +77,32 @@ gemm_tn_simt_kernel(const TA* __restrict__ A, const TW* __restrict__ W, const fl
 
 template <typename TA, typename TW, typename TO>
 static int launch_epi(const void* A, const void* W, const float* bias, void* C, int M, int N, int K,
-                      int lda, int ldw, int ldc, int accumulate, cudaStream_t s) {
+                      int lda, int ldw, int ldc, int epi, cudaStream_t s) {
   dim3 grid(ceil_div(N, BN), ceil_div(M, BM));
-  if (accumulate)
+  if (epi == 2)
+    gemm_tn_simt_kernel<TA, TW, TO, 2><<<grid, 256, 0, s>>>((const TA*)A, (const TW*)W, bias, (TO*)C, M, N, K, lda, ldw, ldc);
+  else if (epi)
     gemm_tn_simt_kernel<TA, TW, TO, 1><<<grid, 256, 0, s>>>((const TA*)A, (const TW*)W, bias, (TO*)C, M, N, K, lda, ldw, ldc);
   else
     gemm_tn_simt_kernel<TA, TW, TO, 0><<<grid, 256, 0, s>>>((const TA*)A, (const TW*)W, bias, (TO*)C, M, N, K, lda, ldw, ldc);
   return launch_status();
 }
 
-// dtype codes: 0 = float32, 1 = bfloat16.  accumulate needs a float32 C.
+// dtype codes: 0 = float32, 1 = bfloat16.  epi: 0 store, 1 add into C (float32), 2 store max(v, 0)^2.
 FELLM_API int fellm_gemm_simt(const void* A, int a_dt, const void* W, int w_dt, const float* bias,
                               void* C, int c_dt, int M, int N, int K, int lda, int ldw, int ldc,
-                              int accumulate, cudaStream_t s) {
+                              int epi, cudaStream_t s) {
   if (M <= 0 || N <= 0) return 0;
   if (!A || !W || !C || K <= 0) return FELLM_ERR_ARG;
-  if (accumulate && c_dt != 0) return FELLM_ERR_ARG;
+  if (epi < 0 || epi > 2 || (epi == 1 && c_dt != 0)) return FELLM_ERR_ARG;
   int key = a_dt * 4 + w_dt * 2 + c_dt;
   switch (key) {
-    case 0: return launch_epi<float, float, float>(A, W, bias, C, M, N, K, lda, ldw, ldc, accumulate, s);
-    case 2: return launch_epi<float, bf16, float>(A, W, bias, C, M, N, K, lda, ldw, ldc, accumulate, s);
-    case 4: return launch_epi<bf16, float, float>(A, W, bias, C, M, N, K, lda, ldw, ldc, accumulate, s);
-    case 5: return launch_epi<bf16, float, bf16>(A, W, bias, C, M, N, K, lda, ldw, ldc, accumulate, s);
-    case 6: return launch_epi<bf16, bf16, float>(A, W, bias, C, M, N, K, lda, ldw, ldc, accumulate, s);
-    case 7: return launch_epi<bf16, bf16, bf16>(A, W, bias, C, M, N, K, lda, ldw, ldc, accumulate, s);
+    case 0: return launch_epi<float, float, float>(A, W, bias, C, M, N, K, lda, ldw, ldc, epi, s);
+    case 2: return launch_epi<float, bf16, float>(A, W, bias, C, M, N, K, lda, ldw, ldc, epi, s);
+    case 4: return launch_epi<bf16, float, float>(A, W, bias, C, M, N, K, lda, ldw, ldc, epi, s);
+    case 5: return launch_epi<bf16, float, bf16>(A, W, bias, C, M, N, K, lda, ldw, ldc, epi, s);
+    case 6: return launch_epi<bf16, bf16, float>(A, W, bias, C, M, N, K, lda, ldw, ldc, epi, s);
+    case 7: return launch_epi<bf16, bf16, bf16>(A, W, bias, C, M, N, K, lda, ldw, ldc, epi, s);
     default: return FELLM_ERR_ARG;   // float32 activations never round down to a bfloat16 result
   }
 }

@@ -38,7 +38,9 @@ namespace cg = cooperative_groups;
 #define SK_XF 2048                   // floats of a row that a warp's float32 buffer takes at a time
 #define SK_GAMMA_MAX 2048            // norm weights of up to this many columns are parked in shared memory
 
-enum { EPI_STORE = 0, EPI_ACC = 1, EPI_SWIGLU = 2, EPI_F32 = 3, EPI_CONV = 4, EPI_ARGMAX = 5 };
+enum { EPI_STORE = 0, EPI_ACC = 1, EPI_SWIGLU = 2, EPI_F32 = 3, EPI_CONV = 4, EPI_ARGMAX = 5, EPI_RELU2 = 6 };
+template <int EPI> __host__ __device__ constexpr bool epi_bf16() { return EPI == EPI_STORE || EPI == EPI_RELU2; }
+__device__ __forceinline__ float relu2_f(float v) { v = fmaxf(v, 0.f); return v * v; }
 #define SK_MAX_LC 8
 
 __device__ __forceinline__ void mma16816(float* d, const unsigned* a, unsigned b0, unsigned b1) {
@@ -127,8 +129,9 @@ __device__ __forceinline__ void epilogue_direct(const SkinnyArgs& a, float (*acc
           if (n >= a.N) continue;
           float v = acc[t][2 * h + e];
           if (a.bias) v += a.bias[n];
+          if (EPI == EPI_RELU2) v = relu2_f(v);
           size_t o = (size_t)m * a.ldo + n;
-          if (EPI == EPI_STORE) ((bf16*)a.out)[o] = __float2bfloat16_rn(v);
+          if (epi_bf16<EPI>()) ((bf16*)a.out)[o] = __float2bfloat16_rn(v);
           else if (EPI == EPI_ACC) ((float*)a.out)[o] += v;
           else ((float*)a.out)[o] = v;
         }
@@ -162,7 +165,7 @@ __device__ __forceinline__ void norm_row_fast(const float4* piece, const float4*
 // MT: token tiles of 8 (M <= 8*MT).
 template <int MT, int EPI>
 __global__ void __launch_bounds__(SK_THREADS, MT <= 2 ? 2 : 1) gemm_skinny_kernel(SkinnyArgs a) {
-  FELLM_TRACE_SCOPE(TRACE_GEMM_SKINNY + 32 * EPI);
+  FELLM_TRACE_SCOPE(TRACE_GEMM_SKINNY + 32 * (EPI == EPI_RELU2 ? EPI_STORE : EPI));
   extern __shared__ __align__(16) unsigned char smem[];
   constexpr int MP = MT * 8;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -422,7 +425,8 @@ __global__ void __launch_bounds__(SK_THREADS, MT <= 2 ? 2 : 1) gemm_skinny_kerne
         ((bf16*)a.out)[(size_t)m * a.ldo + (n0 >> 1) + j] = __float2bfloat16_rn((v0 / (1.0f + expf(-v0))) * v1);
       } else {
         if (a.bias) v0 += a.bias[n];
-        if (EPI == EPI_STORE) ((bf16*)a.out)[o] = __float2bfloat16_rn(v0);
+        if (EPI == EPI_RELU2) v0 = relu2_f(v0);
+        if (epi_bf16<EPI>()) ((bf16*)a.out)[o] = __float2bfloat16_rn(v0);
         else if (EPI == EPI_ACC) ((float*)a.out)[o] = old + v0;
         else ((float*)a.out)[o] = v0;
       }
@@ -465,7 +469,7 @@ struct LeanLoad<N, N> {
 
 template <int MT, int EPI, bool NORM, int WARPS>
 __global__ void __launch_bounds__(WARPS * 32, WARPS == 8 ? 2 : 1) gemm_lean_kernel(SkinnyArgs a) {
-  FELLM_TRACE_SCOPE(TRACE_GEMM_SKINNY + 32 * (EPI == EPI_CONV ? EPI_STORE : (EPI == EPI_ARGMAX ? EPI_F32 : EPI)));
+  FELLM_TRACE_SCOPE(TRACE_GEMM_SKINNY + 32 * (EPI == EPI_CONV || EPI == EPI_RELU2 ? EPI_STORE : (EPI == EPI_ARGMAX ? EPI_F32 : EPI)));
   extern __shared__ __align__(16) unsigned char smem[];
   constexpr int MP = MT * 8;
   __shared__ unsigned long long arg_best[EPI == EPI_ARGMAX ? MT * 8 : 1];     // the CTA's best key of each row
@@ -777,7 +781,8 @@ __global__ void __launch_bounds__(WARPS * 32, WARPS == 8 ? 2 : 1) gemm_lean_kern
         if (live && (lane & 15) == 0) atomicMax(&arg_best[m], key);
       } else {
         if (a.bias) v0 += a.bias[n];
-        if (EPI == EPI_STORE) ((bf16*)a.out)[o] = __float2bfloat16_rn(v0);
+        if (EPI == EPI_RELU2) v0 = relu2_f(v0);
+        if (epi_bf16<EPI>()) ((bf16*)a.out)[o] = __float2bfloat16_rn(v0);
         else if (EPI == EPI_ACC) {
           const float v = old + v0;
           if (live) ((float*)a.out)[o] = v;
@@ -845,7 +850,7 @@ static inline size_t smem_bytes(int mt, int k_per_cta, bool direct, int tiles_pe
 // own.  FELLM_B200_PDL_EPIS overrides the mask (bit = epilogue kind) for experiments.
 static int pdl_class_of(int epi) {
   static int mask = -1;
-  if (mask < 0) { const char* e = getenv("FELLM_B200_PDL_EPIS"); mask = e ? atoi(e) : 47; }
+  if (mask < 0) { const char* e = getenv("FELLM_B200_PDL_EPIS"); mask = e ? atoi(e) : 111; }
   return ((mask >> epi) & 1) ? 1 : 0;
 }
 
@@ -992,7 +997,7 @@ static int dispatch_mt(const SkinnyArgs& a, int ctas_y, cudaStream_t s) {
 }
 
 // epi: 0 store bf16 [M,N]; 1 add into float32 [M,N]; 2 SiLU(gate)*up -> bf16 [M,N/2], W rows
-// interleaved in blocks of 8 gate / 8 up; 3 store float32 [M,N].
+// interleaved in blocks of 8 gate / 8 up; 3 store float32 [M,N]; 6 max(v, 0)^2 -> bf16 [M,N].
 // x: bfloat16 [M,K]; or x = null and xf/norm_w/eps given: float32 [M,K] normed on the way in.
 FELLM_API int fellm_gemm_skinny(const void* x, const float* xf, const float* norm_w, float eps, const void* W,
                                 const float* bias, void* out, int epi, int M, int N, int K, int lda, int ldw,
@@ -1072,6 +1077,7 @@ FELLM_API int fellm_gemm_skinny(const void* x, const float* xf, const float* nor
       case EPI_ACC: return dispatch_lean<EPI_ACC>(a, lp.ctas_y, lp.warps, stream);
       case EPI_SWIGLU: return dispatch_lean<EPI_SWIGLU>(a, lp.ctas_y, lp.warps, stream);
       case EPI_F32: return dispatch_lean<EPI_F32>(a, lp.ctas_y, lp.warps, stream);
+      case EPI_RELU2: return dispatch_lean<EPI_RELU2>(a, lp.ctas_y, lp.warps, stream);
       default: return FELLM_ERR_ARG;
     }
   }
@@ -1081,6 +1087,7 @@ FELLM_API int fellm_gemm_skinny(const void* x, const float* xf, const float* nor
     case EPI_ACC: return dispatch_mt<EPI_ACC>(a, ctas_y, stream);
     case EPI_SWIGLU: return dispatch_mt<EPI_SWIGLU>(a, ctas_y, stream);
     case EPI_F32: return dispatch_mt<EPI_F32>(a, ctas_y, stream);
+    case EPI_RELU2: return dispatch_mt<EPI_RELU2>(a, ctas_y, stream);
     default: return FELLM_ERR_ARG;
   }
 }

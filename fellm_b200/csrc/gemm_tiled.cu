@@ -13,7 +13,7 @@
 #define TSTAGES 3
 #define TTHREADS 256
 
-enum { EPI_STORE = 0, EPI_ACC = 1, EPI_SWIGLU = 2, EPI_F32 = 3 };
+enum { EPI_STORE = 0, EPI_ACC = 1, EPI_SWIGLU = 2, EPI_F32 = 3, EPI_RELU2 = 6 };      // 6: max(v, 0)^2 -> bfloat16
 
 __device__ __forceinline__ void cp_async16(void* smem, const void* gmem, bool pred) {
   unsigned s = (unsigned)__cvta_generic_to_shared(smem);
@@ -145,8 +145,9 @@ gemm_tiled_kernel(const bf16* __restrict__ A, const bf16* __restrict__ W, const 
             if (n + e >= N) continue;
             float v = e ? v1 : v0;
             if (bias) v += bias[n + e];
+            if (EPI == EPI_RELU2) { v = fmaxf(v, 0.f); v *= v; }
             size_t o = (size_t)m * ldo + n + e;
-            if (EPI == EPI_STORE) ((bf16*)out)[o] = __float2bfloat16_rn(v);
+            if (EPI == EPI_STORE || EPI == EPI_RELU2) ((bf16*)out)[o] = __float2bfloat16_rn(v);
             else if (EPI == EPI_ACC) ((float*)out)[o] += v;
             else ((float*)out)[o] = v;
           }
@@ -197,6 +198,7 @@ FELLM_API int fellm_gemm_tiled(const void* A, const void* W, const float* bias, 
     case EPI_ACC: return launch<EPI_ACC>(a, w, bias, out, M, N, K, lda, ldw, ldo, stream);
     case EPI_SWIGLU: return launch<EPI_SWIGLU>(a, w, bias, out, M, N, K, lda, ldw, ldo, stream);
     case EPI_F32: return launch<EPI_F32>(a, w, bias, out, M, N, K, lda, ldw, ldo, stream);
+    case EPI_RELU2: return launch<EPI_RELU2>(a, w, bias, out, M, N, K, lda, ldw, ldo, stream);
     default: return FELLM_ERR_ARG;
   }
 }

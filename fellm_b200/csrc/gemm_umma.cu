@@ -27,7 +27,9 @@ namespace cgx = cooperative_groups;
 #define UM_SPIN_LIMIT (1u << 26)
 #define UM_WAIT_NS 1000000000ull       // one second: far beyond any healthy wait, short enough to stay responsive
 
-enum { EPI_STORE = 0, EPI_ACC = 1, EPI_SWIGLU = 2, EPI_F32 = 3, EPI_CONV = 4 };      // 4: only the product of few rows
+enum { EPI_STORE = 0, EPI_ACC = 1, EPI_SWIGLU = 2, EPI_F32 = 3, EPI_CONV = 4, EPI_RELU2 = 6 };      // 4: only the product of few rows; 6: max(v, 0)^2 -> bfloat16
+template <int EPI> __host__ __device__ constexpr bool epi_bf16() { return EPI == EPI_STORE || EPI == EPI_RELU2; }
+__device__ __forceinline__ float relu2_f(float v) { v = fmaxf(v, 0.f); return v * v; }
 
 __device__ __forceinline__ unsigned smem_u32(const void* p) { return (unsigned)__cvta_generic_to_shared(p); }
 
@@ -133,7 +135,11 @@ __device__ __forceinline__ void store_chunk(const UmmaArgs& a, float* v, int m, 
 #pragma unroll
     for (int j = 0; j < 32; ++j) if (n + j < a.N) v[j] += a.bias[n + j];
   }
-  if (EPI == EPI_STORE && whole && (a.ldo % 8) == 0) {
+  if (EPI == EPI_RELU2) {
+#pragma unroll
+    for (int j = 0; j < 32; ++j) v[j] = relu2_f(v[j]);
+  }
+  if (epi_bf16<EPI>() && whole && (a.ldo % 8) == 0) {
     uint4* dst = (uint4*)((bf16*)a.out + (size_t)m * a.ldo + n);         // 64 contiguous bytes of this row
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
@@ -141,7 +147,7 @@ __device__ __forceinline__ void store_chunk(const UmmaArgs& a, float* v, int m, 
       __nv_bfloat162 p2 = __floats2bfloat162_rn(v[8 * j + 4], v[8 * j + 5]), p3 = __floats2bfloat162_rn(v[8 * j + 6], v[8 * j + 7]);
       dst[j] = make_uint4(*(unsigned*)&p0, *(unsigned*)&p1, *(unsigned*)&p2, *(unsigned*)&p3);
     }
-  } else if (EPI != EPI_STORE && whole && (a.ldo % 4) == 0) {
+  } else if (!epi_bf16<EPI>() && whole && (a.ldo % 4) == 0) {
     float4* dst = (float4*)((float*)a.out + (size_t)m * a.ldo + n);       // 128 contiguous bytes of this row
 #pragma unroll
     for (int j = 0; j < 8; ++j) {
@@ -154,7 +160,7 @@ __device__ __forceinline__ void store_chunk(const UmmaArgs& a, float* v, int m, 
     for (int j = 0; j < 32; ++j) {
       if (n + j >= a.N) break;
       size_t o = (size_t)m * a.ldo + n + j;
-      if (EPI == EPI_STORE) ((bf16*)a.out)[o] = __float2bfloat16_rn(v[j]);
+      if (epi_bf16<EPI>()) ((bf16*)a.out)[o] = __float2bfloat16_rn(v[j]);
       else if (EPI == EPI_ACC) ((float*)a.out)[o] += v[j];
       else ((float*)a.out)[o] = v[j];
     }
@@ -755,6 +761,7 @@ FELLM_API int fellm_gemm_umma(const void* A, const void* W, const float* bias, v
       case EPI_ACC: return launch_ksplit<EPI_ACC>(ma, mw, a, stream);
       case EPI_SWIGLU: return launch_ksplit<EPI_SWIGLU>(ma, mw, a, stream);
       case EPI_F32: return launch_ksplit<EPI_F32>(ma, mw, a, stream);
+      case EPI_RELU2: return launch_ksplit<EPI_RELU2>(ma, mw, a, stream);
       default: return FELLM_ERR_ARG;
     }
   }
@@ -767,6 +774,7 @@ FELLM_API int fellm_gemm_umma(const void* A, const void* W, const float* bias, v
       case EPI_ACC: return bn256 ? launch_pair<EPI_ACC, 256>(ma, mw, a, stream) : launch_pair<EPI_ACC, 128>(ma, mw, a, stream);
       case EPI_SWIGLU: return bn256 ? launch_pair<EPI_SWIGLU, 256>(ma, mw, a, stream) : launch_pair<EPI_SWIGLU, 128>(ma, mw, a, stream);
       case EPI_F32: return bn256 ? launch_pair<EPI_F32, 256>(ma, mw, a, stream) : launch_pair<EPI_F32, 128>(ma, mw, a, stream);
+      case EPI_RELU2: return bn256 ? launch_pair<EPI_RELU2, 256>(ma, mw, a, stream) : launch_pair<EPI_RELU2, 128>(ma, mw, a, stream);
       default: return FELLM_ERR_ARG;
     }
   }
@@ -778,6 +786,7 @@ FELLM_API int fellm_gemm_umma(const void* A, const void* W, const float* bias, v
     case EPI_ACC: return wide ? launch<EPI_ACC, 256>(ma, mw, a, stream) : launch<EPI_ACC, 128>(ma, mw, a, stream);
     case EPI_SWIGLU: return wide ? launch<EPI_SWIGLU, 256>(ma, mw, a, stream) : launch<EPI_SWIGLU, 128>(ma, mw, a, stream);
     case EPI_F32: return wide ? launch<EPI_F32, 256>(ma, mw, a, stream) : launch<EPI_F32, 128>(ma, mw, a, stream);
+    case EPI_RELU2: return wide ? launch<EPI_RELU2, 256>(ma, mw, a, stream) : launch<EPI_RELU2, 128>(ma, mw, a, stream);
     default: return FELLM_ERR_ARG;
   }
 }
@@ -1046,6 +1055,7 @@ gemm_umma_swap_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_co
       if (n + 2 < a.N) v.z += a.bias[n + 2];
       if (n + 3 < a.N) v.w += a.bias[n + 3];
     }
+    if (EPI == EPI_RELU2) { v.x = relu2_f(v.x); v.y = relu2_f(v.y); v.z = relu2_f(v.z); v.w = relu2_f(v.w); }
     if (EPI == EPI_CONV) {
       // B, C and X as the stored product would round them; bx = B*X; conv = bx*w[Lc-1] + sum_t state[t]*w[t]
       // (oldest first); y = C*(conv + bias); the state moves on by one (crates/backend-cpu/src/kernels/shortconv.rs:61-106)
@@ -1099,7 +1109,7 @@ gemm_umma_swap_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_co
       }
     } else if (n + 4 <= a.N && (a.ldo % 4) == 0) {
       const size_t o = (size_t)t * a.ldo + n;
-      if (EPI == EPI_STORE) {
+      if (epi_bf16<EPI>()) {
         __nv_bfloat162 p0 = __floats2bfloat162_rn(v.x, v.y), p1 = __floats2bfloat162_rn(v.z, v.w);
         *(uint2*)((bf16*)a.out + o) = make_uint2(*(unsigned*)&p0, *(unsigned*)&p1);
       } else {
@@ -1122,7 +1132,7 @@ gemm_umma_swap_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_co
       for (int c = 0; c < 4; ++c) {
         if (n + c >= a.N) break;
         const size_t o = (size_t)t * a.ldo + n + c;
-        if (EPI == EPI_STORE) ((bf16*)a.out)[o] = __float2bfloat16_rn(e[c]);
+        if (epi_bf16<EPI>()) ((bf16*)a.out)[o] = __float2bfloat16_rn(e[c]);
         else if (EPI == EPI_ACC) ((float*)a.out)[o] += e[c];
         else ((float*)a.out)[o] = e[c];
       }
@@ -1287,6 +1297,7 @@ FELLM_API int fellm_gemm_umma_swap(const void* x, const void* W, const float* bi
     case EPI_ACC: return launch_swap<EPI_ACC>(mw, mx, a, p.smem, n_tiles, stream);
     case EPI_SWIGLU: return launch_swap<EPI_SWIGLU>(mw, mx, a, p.smem, n_tiles, stream);
     case EPI_F32: return launch_swap<EPI_F32>(mw, mx, a, p.smem, n_tiles, stream);
+    case EPI_RELU2: return launch_swap<EPI_RELU2>(mw, mx, a, p.smem, n_tiles, stream);
     default: return FELLM_ERR_ARG;
   }
 }

@@ -386,3 +386,152 @@ FELLM_API int fellm_qk_rotate_norm(void* qkv, int is_bf16, int ld, int T, int n_
   return launch_k_class(cls, qk_rotate_norm_kernel<float>, grid, dim3(128), 0, stream, 1, (float*)qkv, ld, T, n_q, n_k, k_off, hd,
                         rot_dim, inv_freq, pairing, positions, eps, unit_norm);
 }
+
+// ---------------------------------------------------------------- rotation, value mixing and the cache write in one
+// For layers whose keys and values differ in size, whose cos and sin carry a magnitude, or whose values are mixed with
+// an earlier layer's: the rows of the input product are [q (H hd) | k (G hd) | v (G vd)], ld elements apart.  q is
+// rotated where it lies; k, rotated, and v, or (1 - lam) v + lam v0 (v0: the same rows' values of the layer mixed with,
+// ldv0 elements apart; lam: one float on the device), go into the row's page.  A page-layer record is the keys
+// [G][page_tokens][hd], then the values [G][page_tokens][vd].  Rotation: the first rot_dim elements of a head, angle =
+// float(position) * inv_freq[i], cos and sin times mag; float32 throughout, rounded once.  A block a row: the row's
+// sines and cosines once for all heads, and its page's number, before the wait for the product.
+#define RWM_HALF 256      // pairs of a head in shared memory: rot_dim <= 512
+
+struct RotateWriteArgs {
+  int ld, H, G, hd, vd, rot_dim, pairing, ldv0, max_pages, page_tokens, layer, layers_in_group;
+  float mag;
+  const float* inv_freq; const float* lam;
+  const int* positions; const int* row_slot; const int* block_table;
+  int* status;
+};
+
+template <typename T>
+__global__ void __launch_bounds__(128)
+qkv_rotate_write_kernel(T* __restrict__ qkv, const T* __restrict__ v0, T* __restrict__ pool, RotateWriteArgs a) {
+  __shared__ float sn_s[RWM_HALF], cs_s[RWM_HALF];
+  pdl_launch_dependents();
+  const int row = blockIdx.x, pos = a.positions[row], half = a.rot_dim >> 1;
+  const int page = a.block_table[(size_t)a.row_slot[row] * a.max_pages + pos / a.page_tokens];
+  for (int i = threadIdx.x; i < half; i += blockDim.x) {
+    float sn, cs;
+    sincosf((float)pos * a.inv_freq[i], &sn, &cs);
+    sn_s[i] = sn * a.mag; cs_s[i] = cs * a.mag;
+  }
+  __syncthreads();
+  pdl_wait();
+  T* p = qkv + (size_t)row * a.ld;
+  for (int u = threadIdx.x; u < a.H * half; u += blockDim.x) {
+    const int h = u / half, i = u - h * half;
+    T* q = p + (size_t)h * a.hd;
+    const int ia = a.pairing ? i : 2 * i, ib = a.pairing ? i + half : 2 * i + 1;
+    const float x = to_f(q[ia]), y = to_f(q[ib]);
+    q[ia] = from_f<T>(x * cs_s[i] - y * sn_s[i]); q[ib] = from_f<T>(y * cs_s[i] + x * sn_s[i]);
+  }
+  if (page < 0) {                        // never write outside the pool: record and skip
+    if (threadIdx.x == 0 && a.status) atomicExch(a.status, 2);
+    return;
+  }
+  const int in_page = pos % a.page_tokens;
+  T* rec = pool + ((size_t)page * a.layers_in_group + a.layer) * ((size_t)a.G * a.page_tokens * (a.hd + a.vd));
+  const T* kp = p + (size_t)a.H * a.hd;
+  const int per_k = a.hd - half;         // a pair, or one element behind the rotated part
+  for (int u = threadIdx.x; u < a.G * per_k; u += blockDim.x) {
+    const int g = u / per_k, i = u - g * per_k;
+    const T* k = kp + (size_t)g * a.hd;
+    T* dst = rec + ((size_t)g * a.page_tokens + in_page) * a.hd;
+    if (i < half) {
+      const int ia = a.pairing ? i : 2 * i, ib = a.pairing ? i + half : 2 * i + 1;
+      const float x = to_f(k[ia]), y = to_f(k[ib]);
+      dst[ia] = from_f<T>(x * cs_s[i] - y * sn_s[i]); dst[ib] = from_f<T>(y * cs_s[i] + x * sn_s[i]);
+    } else {
+      dst[i + half] = k[i + half];
+    }
+  }
+  const T* vp = kp + (size_t)a.G * a.hd;
+  T* vrec = rec + (size_t)a.G * a.page_tokens * a.hd;
+  const float lam = v0 ? *a.lam : 0.f;
+  for (int u = threadIdx.x; u < a.G * a.vd; u += blockDim.x) {
+    const int g = u / a.vd, c = u - g * a.vd;
+    T* dst = vrec + ((size_t)g * a.page_tokens + in_page) * a.vd + c;
+    if (v0) *dst = from_f<T>((1.0f - lam) * to_f(vp[u]) + lam * to_f(v0[(size_t)row * a.ldv0 + u]));
+    else *dst = vp[u];
+  }
+}
+
+// bfloat16, pairs (i, i + rot_dim/2), hd and vd multiples of 8, rot_dim of 16, rows on 16-byte boundaries: a thread eight
+// elements (and the eight they are paired with) by 16-byte loads and stores.
+__global__ void __launch_bounds__(128)
+qkv_rotate_write_vec_kernel(bf16* __restrict__ qkv, const bf16* __restrict__ v0, bf16* __restrict__ pool, RotateWriteArgs a) {
+  __shared__ float sn_s[RWM_HALF], cs_s[RWM_HALF];
+  pdl_launch_dependents();
+  const int row = blockIdx.x, pos = a.positions[row], half = a.rot_dim >> 1;
+  const int page = a.block_table[(size_t)a.row_slot[row] * a.max_pages + pos / a.page_tokens];
+  for (int i = threadIdx.x; i < half; i += blockDim.x) {
+    float sn, cs;
+    sincosf((float)pos * a.inv_freq[i], &sn, &cs);
+    sn_s[i] = sn * a.mag; cs_s[i] = cs * a.mag;
+  }
+  __syncthreads();
+  pdl_wait();
+  bf16* p = qkv + (size_t)row * a.ld;
+  const int hc = half >> 3, kc = (a.hd >> 3) - hc, vc = a.vd >> 3;      // units of a query head, a key head, a value
+  const int n_q = a.H * hc, n_k = a.G * kc, n_v = a.G * vc;
+  const int in_page = pos % a.page_tokens;
+  if (page < 0 && threadIdx.x == 0 && a.status) atomicExch(a.status, 2);          // never write outside the pool: record and skip
+  bf16* rec = pool + ((size_t)max(page, 0) * a.layers_in_group + a.layer) * ((size_t)a.G * a.page_tokens * (a.hd + a.vd));
+  const int n_units = page < 0 ? n_q : n_q + n_k + n_v;
+  const float lam = v0 ? *a.lam : 0.f;
+  for (int u = threadIdx.x; u < n_units; u += blockDim.x) {
+    if (u < n_q + n_k) {
+      const bool is_q = u < n_q;
+      const int w = is_q ? u : u - n_q, per = is_q ? hc : kc, head = w / per, c = w - head * per;
+      const bf16* src = p + (is_q ? (size_t)head * a.hd : (size_t)(a.H + head) * a.hd);
+      bf16* dst = is_q ? const_cast<bf16*>(src) : rec + ((size_t)head * a.page_tokens + in_page) * a.hd;
+      if (c < hc) {
+        float x[8], y[8];
+        rw_unpack8(*(const uint4*)(src + 8 * c), x); rw_unpack8(*(const uint4*)(src + half + 8 * c), y);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) {
+          const float sn = sn_s[8 * c + e], cs = cs_s[8 * c + e], xe = x[e];
+          x[e] = xe * cs - y[e] * sn; y[e] = y[e] * cs + xe * sn;
+        }
+        *(uint4*)(dst + 8 * c) = rw_pack8(x); *(uint4*)(dst + half + 8 * c) = rw_pack8(y);
+      } else {
+        *(uint4*)(dst + half + 8 * c) = *(const uint4*)(src + half + 8 * c);
+      }
+    } else {
+      const int w = u - n_q - n_k, g = w / vc, c = w - g * vc;
+      uint4 val = *(const uint4*)(p + (size_t)(a.H + a.G) * a.hd + 8 * w);
+      if (v0) {
+        float x[8], y[8];
+        rw_unpack8(val, x); rw_unpack8(*(const uint4*)(v0 + (size_t)row * a.ldv0 + 8 * w), y);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) x[e] = (1.0f - lam) * x[e] + lam * y[e];
+        val = rw_pack8(x);
+      }
+      *(uint4*)(rec + (size_t)a.G * a.page_tokens * a.hd + ((size_t)g * a.page_tokens + in_page) * a.vd + 8 * c) = val;
+    }
+  }
+}
+
+FELLM_API int fellm_qkv_rotate_write(void* qkv, int is_bf16, int ld, int T, int H, int G, int hd, int vd, int rot_dim,
+                                     const float* inv_freq, int pairing, float mag, const void* v0, int ldv0, const float* lam,
+                                     const int* positions, const int* row_slot, const int* block_table, int max_pages,
+                                     void* pool, int cache_bf16, int page_tokens, int layer, int layers_in_group, int* status,
+                                     cudaStream_t stream) {
+  if (T <= 0) return 0;
+  if (!inv_freq) rot_dim = 0;
+  if (H < 1 || G < 1 || hd < 1 || vd < 1 || rot_dim < 0 || rot_dim > hd || (rot_dim & 1) || rot_dim > 2 * RWM_HALF || page_tokens < 1) return FELLM_ERR_SIZE;
+  if (ld < H * hd + G * (hd + vd) || (v0 && ldv0 < G * vd)) return FELLM_ERR_SIZE;
+  if (!qkv || !positions || !row_slot || !block_table || !pool || (v0 && !lam) || is_bf16 != cache_bf16) return FELLM_ERR_ARG;
+  RotateWriteArgs a;
+  a.ld = ld; a.H = H; a.G = G; a.hd = hd; a.vd = vd; a.rot_dim = rot_dim; a.pairing = pairing; a.ldv0 = ldv0; a.max_pages = max_pages;
+  a.page_tokens = page_tokens; a.layer = layer; a.layers_in_group = layers_in_group; a.mag = mag; a.inv_freq = inv_freq; a.lam = lam;
+  a.positions = positions; a.row_slot = row_slot; a.block_table = block_table; a.status = status;
+  const int cls = launch_class_for_rows(T, 2);
+  const bool vec = is_bf16 && (pairing == 1 || rot_dim == 0) && hd % 8 == 0 && vd % 8 == 0 && rot_dim % 16 == 0 && ld % 8 == 0 &&
+                   (!v0 || (ldv0 % 8 == 0 && ((uintptr_t)v0 & 15) == 0)) && (((uintptr_t)qkv | (uintptr_t)pool) & 15) == 0;
+  if (vec) return launch_k_class(cls, qkv_rotate_write_vec_kernel, dim3(T), dim3(128), 0, stream, 1, (bf16*)qkv, (const bf16*)v0, (bf16*)pool, a);
+  if (is_bf16) return launch_k_class(cls, qkv_rotate_write_kernel<bf16>, dim3(T), dim3(128), 0, stream, 1, (bf16*)qkv, (const bf16*)v0, (bf16*)pool, a);
+  return launch_k_class(cls, qkv_rotate_write_kernel<float>, dim3(T), dim3(128), 0, stream, 1, (float*)qkv, (const float*)v0, (float*)pool, a);
+}

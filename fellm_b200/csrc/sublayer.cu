@@ -7,6 +7,7 @@
 //   act_mul          [gate | up] rows -> act(gate) * up, act = SiLU or the tanh form of GELU
 //   gate_mul         a *= sigmoid(g), element by element (an output gate on concatenated heads)
 //   relu2            max(z, 0)^2, float32 in, activation dtype out (a plain expert's activation)
+//   add_rmsnorm      x += RMSNorm(y) in place (float32), and the RMSNorm of the new rows for what reads the stream next
 //
 // Every row is reduced by one warp in an order that depends on the row's length alone: a token's result does not
 // depend on the batch it is in.  Means, variances and the sums into the stream are float32.
@@ -318,4 +319,115 @@ FELLM_API int fellm_relu2(const float* z, void* out, int out_is_bf16, long long 
   const int cls = launch_class_for_rows(n / 256, 0);
   if (out_is_bf16) return launch_k_class(cls, relu2_kernel<bf16>, dim3(ew_blocks(n)), dim3(256), 0, stream, 1, z, (bf16*)out, n);
   return launch_k_class(cls, relu2_kernel<float>, dim3(ew_blocks(n)), dim3(256), 0, stream, 1, z, (float*)out, n);
+}
+
+// ---------------------------------------------------------------- x += RMSNorm(y), and the norm that reads x next
+// x[t, :] += y[t, :] / rms(y[t, :]) * w; then (wn not null) h[t, :] = x[t, :] / rms(x[t, :]) * wn for the sublayer (or
+// the head) that reads the stream next, in TO.  A block a row; the row's numbers stay in registers between the two sums
+// (VPT 16-byte vectors a thread); the number of threads depends on the row's length alone, and so does every sum's order.
+template <int VPT, typename TO>
+__global__ void __launch_bounds__(1024)
+add_rmsnorm_vec_kernel(float* __restrict__ x, const float* __restrict__ y, const float* __restrict__ w, float eps,
+                       const float* __restrict__ wn, float eps_n, TO* __restrict__ h, int d) {
+  __shared__ float part[2][32];
+  pdl_launch_dependents();
+  const int nv = d >> 2, tid = threadIdx.x, nw = (blockDim.x + 31) >> 5;
+  float4 w4[VPT], n4[VPT];
+#pragma unroll
+  for (int j = 0; j < VPT; ++j) {          // (the weights do not wait for the kernel in front)
+    const int i = tid + j * blockDim.x;
+    w4[j] = i < nv ? ((const float4*)w)[i] : make_float4(0.f, 0.f, 0.f, 0.f);
+    n4[j] = (wn && i < nv) ? ((const float4*)wn)[i] : make_float4(0.f, 0.f, 0.f, 0.f);
+  }
+  pdl_wait();
+  const float4* yr = (const float4*)(y + (size_t)blockIdx.x * d);
+  float4* xr = (float4*)(x + (size_t)blockIdx.x * d);
+  float4 v[VPT], r[VPT];
+  float s = 0.f;
+#pragma unroll
+  for (int j = 0; j < VPT; ++j) {
+    const int i = tid + j * blockDim.x;
+    v[j] = i < nv ? yr[i] : make_float4(0.f, 0.f, 0.f, 0.f);
+    r[j] = i < nv ? xr[i] : make_float4(0.f, 0.f, 0.f, 0.f);
+  }
+#pragma unroll
+  for (int j = 0; j < VPT; ++j) s = fmaf(v[j].x, v[j].x, fmaf(v[j].y, v[j].y, fmaf(v[j].z, v[j].z, fmaf(v[j].w, v[j].w, s))));
+  s = warp_sum(s);
+  if ((tid & 31) == 0) part[0][tid >> 5] = s;
+  __syncthreads();
+  s = 0.f;
+  for (int i = 0; i < nw; ++i) s += part[0][i];
+  const float sc = 1.0f / sqrtf(s / (float)d + eps);
+  float q = 0.f;
+#pragma unroll
+  for (int j = 0; j < VPT; ++j) {
+    const int i = tid + j * blockDim.x;
+    r[j].x = fmaf(v[j].x * sc, w4[j].x, r[j].x); r[j].y = fmaf(v[j].y * sc, w4[j].y, r[j].y);
+    r[j].z = fmaf(v[j].z * sc, w4[j].z, r[j].z); r[j].w = fmaf(v[j].w * sc, w4[j].w, r[j].w);
+    if (i < nv) xr[i] = r[j];
+    q = fmaf(r[j].x, r[j].x, fmaf(r[j].y, r[j].y, fmaf(r[j].z, r[j].z, fmaf(r[j].w, r[j].w, q))));
+  }
+  if (!wn) return;
+  q = warp_sum(q);
+  if ((tid & 31) == 0) part[1][tid >> 5] = q;
+  __syncthreads();
+  q = 0.f;
+  for (int i = 0; i < nw; ++i) q += part[1][i];
+  const float sn = 1.0f / sqrtf(q / (float)d + eps_n);
+  TO* o = h + (size_t)blockIdx.x * d;
+#pragma unroll
+  for (int j = 0; j < VPT; ++j) {
+    const int i = tid + j * blockDim.x;
+    if (i < nv) put4(o + 4 * i, make_float4((r[j].x * sn) * n4[j].x, (r[j].y * sn) * n4[j].y, (r[j].z * sn) * n4[j].z, (r[j].w * sn) * n4[j].w));
+  }
+}
+
+// Any width and alignment: the rows are read again instead of kept.
+template <typename TO>
+__global__ void __launch_bounds__(256)
+add_rmsnorm_kernel(float* __restrict__ x, const float* __restrict__ y, const float* __restrict__ w, float eps,
+                   const float* __restrict__ wn, float eps_n, TO* __restrict__ h, int d) {
+  __shared__ float part[2][8];
+  pdl_launch_dependents();
+  pdl_wait();
+  const float* yr = y + (size_t)blockIdx.x * d;
+  float* xr = x + (size_t)blockIdx.x * d;
+  const int tid = threadIdx.x;
+  float s = 0.f;
+  for (int i = tid; i < d; i += 256) s = fmaf(yr[i], yr[i], s);
+  s = warp_sum(s);
+  if ((tid & 31) == 0) part[0][tid >> 5] = s;
+  __syncthreads();
+  s = 0.f;
+  for (int i = 0; i < 8; ++i) s += part[0][i];
+  const float sc = 1.0f / sqrtf(s / (float)d + eps);
+  float q = 0.f;
+  for (int i = tid; i < d; i += 256) { const float v = fmaf(yr[i] * sc, w[i], xr[i]); xr[i] = v; q = fmaf(v, v, q); }
+  if (!wn) return;
+  q = warp_sum(q);
+  if ((tid & 31) == 0) part[1][tid >> 5] = q;
+  __syncthreads();
+  q = 0.f;
+  for (int i = 0; i < 8; ++i) q += part[1][i];
+  const float sn = 1.0f / sqrtf(q / (float)d + eps_n);
+  TO* o = h + (size_t)blockIdx.x * d;
+  for (int i = tid; i < d; i += 256) o[i] = from_f<TO>((xr[i] * sn) * wn[i]);      // (a thread reads back what it wrote itself)
+}
+
+FELLM_API int fellm_add_rmsnorm(float* x, const float* y, const float* w, float eps, const float* wn, float eps_n, void* h,
+                                int h_is_bf16, int n_rows, int d, cudaStream_t stream) {
+  if (n_rows <= 0) return 0;
+  if (!x || !y || !w || d < 1 || (wn && !h)) return FELLM_ERR_ARG;
+  const int cls = launch_class_for_rows(n_rows, 0);
+  const bool vec = d % 4 == 0 && d <= 16384 && ((((uintptr_t)x | (uintptr_t)y | (uintptr_t)w | (uintptr_t)wn | (uintptr_t)h) & 15) == 0);
+  if (vec) {
+    const int nv = d / 4, vpt = nv <= 2048 ? 2 : 4;
+    int threads = (((nv + vpt - 1) / vpt) + 31) & ~31;
+#define AR_VEC(V_, T_) launch_k_class(cls, add_rmsnorm_vec_kernel<V_, T_>, dim3(n_rows), dim3(threads), 0, stream, 1, x, y, w, eps, wn, eps_n, (T_*)h, d)
+    if (h_is_bf16) return vpt == 2 ? AR_VEC(2, bf16) : AR_VEC(4, bf16);
+    return vpt == 2 ? AR_VEC(2, float) : AR_VEC(4, float);
+#undef AR_VEC
+  }
+  if (h_is_bf16) return launch_k_class(cls, add_rmsnorm_kernel<bf16>, dim3(n_rows), dim3(256), 0, stream, 1, x, y, w, eps, wn, eps_n, (bf16*)h, d);
+  return launch_k_class(cls, add_rmsnorm_kernel<float>, dim3(n_rows), dim3(256), 0, stream, 1, x, y, w, eps, wn, eps_n, (float*)h, d);
 }

@@ -37,10 +37,12 @@ class StepContext:
     tokens[T], positions[T] (absolute), row_item[T] (index of the row's item), row_slot[T] (its
     request's slot: the row of block tables and state arrays), item_start[n_items+1] (row offsets),
     item_slot[n_items], item_len[n_items] (request length after this step), logit_rows[W].
+    carried: what a part leaves for a later part of the same step (rows of this step's tokens, by name); a model's
+    forward() starts and ends with it empty.
     """
     __slots__ = ("tokens", "positions", "row_item", "row_slot", "item_start", "item_slot", "item_len",
                  "logit_rows", "n_rows", "n_items", "n_logit_rows", "all_single", "max_item_rows",
-                 "max_len", "status", "host", "logits_all", "fixed_addresses")
+                 "max_len", "status", "host", "logits_all", "fixed_addresses", "carried")
 
 
 class StepBuffers:

@@ -132,6 +132,44 @@ def _outnorm(block, x, ctx, cache, act_dtype, reads_only):
     block.norm2.add_normed(x, y)
 
 
+@register_arrangement("sandwich")
+def _sandwich(block, x, ctx, cache, act_dtype, reads_only):
+    """x += norm1b(mixer(norm1(x))); x += norm2b(ffn(norm2(x))).  A sublayer leaves float32 rows of its own (written where
+    it says `can_store`, else added into zeros); the norm on them takes them into the stream and, in the same kernel, norms
+    the new rows for what reads the stream next: norm2 for the feed-forward, else the next block's first norm (or the
+    final one), whose block finds the rows in ctx.carried."""
+    if block.norm1b is None or (block.ffn is not None and block.norm2b is None):
+        raise ConfigError("the 'sandwich' arrangement needs norms on the sublayers' outputs (norm1b, norm2b)")
+
+    def run(part, *args, **kw):
+        if getattr(part, "can_store", False):
+            return part.forward(*args, torch.empty_like(x), store=True, **kw)
+        return part.forward(*args, torch.zeros_like(x), **kw)
+
+    after = None if block.side is not None else block.norm_after        # (a side input changes the rows once more)
+    h = take_normed(ctx, block.norm1, x, act_dtype)
+    y = run(block.mixer, h, ctx, cache, reads_only=reads_only)
+    if block.ffn is None:
+        leave_normed(ctx, after, block.norm1b.add_normed_then(x, y, after, act_dtype))
+        return
+    h = block.norm1b.add_normed_then(x, y, block.norm2, act_dtype)
+    if h is None:
+        h = block.norm2.forward(x, act_dtype)
+    y = run(block.ffn, h, ctx)
+    leave_normed(ctx, after, block.norm2b.add_normed_then(x, y, after, act_dtype))
+
+
+def leave_normed(ctx, norm, h):
+    """The rows of the stream normed by `norm` already (or None), for the block (or the head) behind this one."""
+    ctx.carried["normed"] = (norm, h)
+
+
+def take_normed(ctx, norm, x, act_dtype):
+    """The rows of x normed by `norm`: as an earlier block left them, or normed now."""
+    left, h = ctx.carried.pop("normed", (None, None))
+    return h if left is norm and h is not None else norm.forward(x, act_dtype)
+
+
 def _with_children(part):
     return [part] + [q for c in part.children() for q in _with_children(c)]
 
@@ -151,6 +189,8 @@ class Block:
         self.ffn = build_part("feed_forward", spec.ffn, dtype) if spec.ffn is not None else None
         self.gate = build_part("gate", spec.gate, dtype) if spec.gate is not None else None
         self.side = build_part("side", spec.side, dtype) if spec.side is not None else None
+        self.norm1b = build_part("norm", spec.norm1b, dtype) if spec.norm1b is not None else None
+        self.norm2b = build_part("norm", spec.norm2b, dtype) if spec.norm2b is not None else None
         self.norm_after = None
         self.joint = None           # (weight [N, d], bias float32 [N], {"gate" | "mixer" | "ffn": (first column, end)}) after join_inputs()
 
@@ -181,7 +221,7 @@ class Block:
         self.joint = (joint, bias, cols)
 
     def parts(self):
-        return [q for p in (self.norm1, self.mixer, self.norm2, self.ffn, self.gate, self.side) if p is not None
+        return [q for p in (self.norm1, self.mixer, self.norm1b, self.norm2, self.ffn, self.norm2b, self.gate, self.side) if p is not None
                 for q in _with_children(p)]
 
     def forward(self, x, ctx, cache, act_dtype, reads_only=False, norm_after=None):
@@ -288,6 +328,7 @@ class Model:
         greedy_tokens (int32, device): the caller only wants the greedy token of every wanted row; where the
         head can give them without the logits it writes greedy_tokens[:wanted] and None is returned."""
         ops.forget_norm_handoff()
+        ctx.carried = {}
         x = self.embedding.forward(ctx.tokens, ctx.status)
         # a connector reads the embedding's output again later; the blocks update x in place
         x0 = x.clone() if any(c.needs_embedding for c in self.connectors) else None
@@ -295,6 +336,7 @@ class Model:
             src = n if run.cache_of is None else run.cache_of
             if run.before is not None:
                 x = self.connectors[run.before[0]].forward(x, x0, run.before[1], self.act_dtype)
+                ctx.carried.pop("normed", None)             # (the rows have changed)
             if n + 1 < len(self.schedule):
                 norm_after = self.blocks[self.schedule[n + 1].layer].norm1
             else:
@@ -308,10 +350,13 @@ class Model:
                 self.after_run(n, x)
         if ctx.n_logit_rows == 0:
             return torch.empty((0, self.spec.vocab_size), dtype=torch.float32, device=x.device)
-        if ctx.logits_all and getattr(self.head, "takes_lazy_norm", False):
+        if ctx.logits_all and ctx.carried.get("normed", (None, None))[0] is self.final_norm:
+            xf = take_normed(ctx, self.final_norm, x, self.act_dtype)
+        elif ctx.logits_all and getattr(self.head, "takes_lazy_norm", False):
             xf = LazyNorm(x, self.final_norm, self.act_dtype)
         else:
             xf = self.final_norm.forward(x, self.act_dtype, rows=ctx.logit_rows)
+        ctx.carried = {}
         if greedy_tokens is not None and self.head.forward_greedy(xf, greedy_tokens):
             return None
         return self.head.forward(xf)

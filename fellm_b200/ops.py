@@ -177,6 +177,24 @@ def add_layernorm(x, y, w, b, eps: float, cast=None):
     return x
 
 
+def add_rmsnorm(x, y, w, eps: float, next_w=None, next_eps: float = 0.0, out_dtype=None, out=None):
+    """x float32 [T, d] += y / sqrt(mean(y^2) + eps) * w, in place; with next_w, the RMSNorm of the new rows,
+    x / sqrt(mean(x^2) + next_eps) * next_w, in out_dtype (returned; None without next_w)."""
+    _dev(x, y, w, next_w, out)
+    assert x.dtype == torch.float32 and y.dtype == torch.float32 and w.dtype == torch.float32
+    assert x.is_contiguous() and y.is_contiguous() and x.shape == y.shape and w.numel() == x.shape[1] and w.is_contiguous()
+    if next_w is not None:
+        assert next_w.dtype == torch.float32 and next_w.numel() == x.shape[1] and next_w.is_contiguous()
+        if out is None:
+            out = torch.empty(x.shape, dtype=out_dtype, device=x.device)
+        assert out.is_contiguous() and out.shape == x.shape
+    residual_written(x)
+    f = _fn("sublayer", "fellm_add_rmsnorm", [_c_p, _c_p, _c_p, _c_f, _c_p, _c_f, _c_p, _c_int, _c_int, _c_int, _c_p])
+    _check(f(_p(x), _p(y), _p(w), float(eps), _p(next_w), float(next_eps), _p(out) if next_w is not None else None,
+             _is_bf16(out) if next_w is not None else 0, x.shape[0], x.shape[1], _stream()), "add_rmsnorm")
+    return out
+
+
 def cast_rows(x, out_dtype, out=None):
     """float32 rows in the activation dtype (the tensor itself where that is float32)."""
     if out_dtype == torch.float32:
@@ -366,15 +384,15 @@ def add_rows(x, y):
 
 # ------------------------------------------------------------------------------ matrix products
 
-def gemm_simt(a, w, bias=None, out=None, out_dtype=None, accumulate=False):
+def gemm_simt(a, w, bias=None, out=None, out_dtype=None, accumulate=False, act=None):
     """out[M, N] = a[M, K] @ w[N, K]^T (+ bias[N]) with float32 FMA on CUDA cores; with
-    accumulate=True, out (float32) += that.  Any mix of bfloat16/float32 a and w."""
+    accumulate=True, out (float32) += that; act="relu2": out = max(that, 0)^2.  Any mix of bfloat16/float32 a and w."""
     _dev(a, w, bias, out)
     M, K = a.shape
     N = w.shape[0]
     if w.shape[1] != K:
         raise KernelError(f"gemm: a is [{M},{K}] but w is {list(w.shape)}")
-    assert a.stride(1) == 1 and w.stride(1) == 1
+    assert a.stride(1) == 1 and w.stride(1) == 1 and act in (None, "relu2") and not (act and accumulate)
     if out is None:
         assert not accumulate
         out = torch.empty((M, N), dtype=out_dtype or a.dtype, device=a.device)
@@ -389,7 +407,7 @@ def gemm_simt(a, w, bias=None, out=None, out_dtype=None, accumulate=False):
             [_c_p, _c_int, _c_p, _c_int, _c_p, _c_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int,
              _c_int, _c_p])
     _check(f(_p(a), _is_bf16(a), _p(w), _is_bf16(w), _p(bias), _p(out), _is_bf16(out), M, N, K,
-             a.stride(0), w.stride(0), out.stride(0), int(accumulate), _stream()), "gemm_simt")
+             a.stride(0), w.stride(0), out.stride(0), 2 if act else int(accumulate), _stream()), "gemm_simt")
     return out
 
 
@@ -1036,6 +1054,36 @@ def qk_rotate_norm(qkv, n_q, n_k, k_off, hd, rot_dim, inv_freq, pairing, positio
     return qkv
 
 
+def qkv_rotate_write(qkv, H, G, hd, vd, rot_dim, inv_freq, pairing, mag, positions, row_slot, cache, *, v_first=None, lam=None,
+                     status=None):
+    """The rows of a layer's input product, [q (H hd) | k (G hd) | v (G vd)]: q is rotated where it lies (the first rot_dim
+    elements of a head, angle = position * inv_freq[i], cos and sin times mag; inv_freq None: no rotation), k, rotated, and v
+    go into the rows' pages.  v_first [T, G vd] with lam (float32, one element on the device): what goes into the page is
+    (1 - lam) v + lam v_first.  cache: a PagedView whose page-layer record is the keys [G][page_tokens][hd], then the values
+    [G][page_tokens][vd]."""
+    pool, bt = cache.pool, cache.block_table
+    _dev(qkv, inv_freq, positions, row_slot, pool, bt, v_first, lam)
+    T = qkv.shape[0]
+    assert qkv.stride(1) == 1 and qkv.shape[1] >= H * hd + G * (hd + vd) and pool.is_contiguous() and pool.dtype == qkv.dtype
+    assert pool[0, 0].numel() == G * cache.page_tokens * (hd + vd)
+    rot_dim = 0 if inv_freq is None else int(rot_dim)
+    if rot_dim % 2 or not 0 <= rot_dim <= min(hd, 512):
+        raise KernelError(f"qkv_rotate_write: rotated part {rot_dim} must be even, within the head ({hd}) and at most 512")
+    if inv_freq is not None:
+        assert inv_freq.dtype == torch.float32 and inv_freq.numel() == rot_dim // 2 and inv_freq.is_contiguous()
+    if v_first is not None:
+        assert v_first.shape == (T, G * vd) and v_first.dtype == qkv.dtype and v_first.stride(1) == 1
+        assert lam is not None and lam.dtype == torch.float32 and lam.numel() == 1
+    _i32(positions, "positions"), _i32(row_slot, "row_slot"), _i32(bt, "block_table")
+    f = _fn("qk_rope_write", "fellm_qkv_rotate_write",
+            [_c_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_p, _c_int, _c_f, _c_p, _c_int, _c_p, _c_p, _c_p,
+             _c_p, _c_int, _c_p, _c_int, _c_int, _c_int, _c_int, _c_p, _c_p])
+    _check(f(_p(qkv), _is_bf16(qkv), qkv.stride(0), T, H, G, hd, vd, rot_dim, _p(inv_freq), PAIRINGS[pairing], float(mag),
+             _p(v_first), v_first.stride(0) if v_first is not None else 0, _p(lam), _p(positions), _p(row_slot), _p(bt),
+             bt.shape[1], _p(pool), _is_bf16(pool), cache.page_tokens, cache.layer, pool.shape[1], _p(status), _stream()),
+           "qkv_rotate_write")
+
+
 def paged_attention_simt(q, pool, block_table, positions, row_slot, layer, scale, window=None, out=None):
     """q [T, H, hd]; pool [pages, layers, 2, G, page_tokens, hd].  Row t attends to the cache
     positions 0..positions[t] (or the last `window` of them) of its item.  Returns [T, H*hd]."""
@@ -1237,7 +1285,7 @@ def latent_attention(q_abs, H, rk, dr, pool, block_table, positions, row_slot, i
 
 # ------------------------------------------------------------------------------ tensor-core products
 
-_EPI_STORE, _EPI_ACC, _EPI_SWIGLU, _EPI_F32 = 0, 1, 2, 3
+_EPI_STORE, _EPI_ACC, _EPI_SWIGLU, _EPI_F32, _EPI_RELU2 = 0, 1, 2, 3, 6
 SKINNY_MAX_ROWS = 32      # measured on B200 (350M shapes): above 32 rows the tcgen05 product wins on every shape
 _GEMM_ARGS = [_c_p, _c_p, _c_p, _c_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_p]
 _SKINNY_ARGS = [_c_p, _c_p, _c_p, _c_f, _c_p, _c_p, _c_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_p]
@@ -1477,10 +1525,11 @@ def _announce_row_scale(row_scale, M: int, N: int, K: int, own_plan: bool = Fals
     _fn(module, f"fellm_{module}_row_scale", [_c_p, _c_int, _c_f])(_p(ssq), int(parts), float(eps))
 
 
-def gemm_bf16(x, w, bias=None, *, out=None, out_dtype=None, accumulate=False, swiglu=False, norm=None, row_scale=None):
+def gemm_bf16(x, w, bias=None, *, out=None, out_dtype=None, accumulate=False, swiglu=False, norm=None, row_scale=None, act=None):
     """out = x[M,K] @ w[N,K]^T (+bias) on tensor cores, bfloat16 in, float32 sums.
     accumulate: out (float32 [M,N]) += ; swiglu: w's rows are interleaved in blocks of 8 gate / 8 up
-    and out is bfloat16 [M, N/2] = silu(gate)*up; out_dtype float32: float32 store.
+    and out is bfloat16 [M, N/2] = silu(gate)*up; out_dtype float32: float32 store; act="relu2": out is bfloat16
+    [M, N] = max(x w^T (+bias), 0)^2.
     norm=(weight float32 [K], eps): x is the float32 residual stream and is RMS-normed on its way
     into the product (see norm_fusable).
     row_scale=(ssq, parts, eps): x is the pre-weighted input of a handed-on norm (norm_handoff)."""
@@ -1507,6 +1556,13 @@ def gemm_bf16(x, w, bias=None, *, out=None, out_dtype=None, accumulate=False, sw
         if out is None:
             out = torch.empty((M, N // 2), dtype=torch.bfloat16, device=x.device)
         assert out.dtype == torch.bfloat16 and out.shape == (M, N // 2)
+    elif act is not None:
+        if act != "relu2":
+            raise KernelError(f"gemm_bf16: unknown activation {act!r}")
+        epi = _EPI_RELU2
+        if out is None:
+            out = torch.empty((M, N), dtype=torch.bfloat16, device=x.device)
+        assert out.dtype == torch.bfloat16 and out.shape == (M, N)
     elif (out_dtype or (out.dtype if out is not None else torch.bfloat16)) == torch.float32:
         epi = _EPI_F32
         if out is None:
@@ -1617,7 +1673,7 @@ def gemm_bf16_argmax(x, w, bias, keys, out_tokens, *, norm=None, row_scale=None)
 
 def gemm_umma_swap(x, w, bias=None, *, out, epi: int, written: bool = False):
     """The tcgen05 product for up to 128 rows (weights as the MMA's rows, K split over a cluster),
-    callable by itself.  epi: 0 store bfloat16, 1 add into float32, 2 SiLU(gate)*up, 3 store float32."""
+    callable by itself.  epi: 0 store bfloat16, 1 add into float32, 2 SiLU(gate)*up, 3 store float32, 6 max(v, 0)^2 -> bfloat16."""
     M, K = x.shape
     if epi == _EPI_ACC and not written:
         residual_written(out)
@@ -1807,11 +1863,11 @@ def attention_decode(q, pool, block_table, positions, row_slot, layer, scale, wi
                  _stream()), "attention_decode (TMA)")
         return out
     f = _fn("attention_mma", "fellm_attn_decode_mma",
-            [_c_p, _c_p, _c_p, _c_int, _c_p, _c_p, _c_p, _c_p, _c_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int,
-             _c_int, _c_f, _c_int, _c_int, _c_int, _c_p], defines={"HD": hd})
-    _check(f(_p(q), _p(pool), _p(block_table), block_table.shape[1], _p(positions), _p(row_slot), _p(out),
+            [_c_p, _c_int, _c_p, _c_p, _c_int, _c_p, _c_p, _c_p, _c_p, _c_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int,
+             _c_int, _c_f, _c_int, _c_int, _c_int, _c_p, _c_p], defines={"HD": hd})
+    _check(f(_p(q), H * hd, _p(pool), _p(block_table), block_table.shape[1], _p(positions), _p(row_slot), _p(out),
              _p(scratch), _p(counters), T, H, G, hd, page_tokens, layer, pool.shape[1], float(scale),
-             int(window or 0), split_len, max_splits, _stream()), "attention_decode")
+             int(window or 0), split_len, max_splits, None, _stream()), "attention_decode")
     return out
 
 
@@ -1826,16 +1882,11 @@ def attention_prefill(q, pool, block_table, positions, row_slot, item_start, n_i
     _i32(item_start, "item_start")
     if out is None:
         out = torch.empty((T, H * hd), dtype=q.dtype, device=q.device)
-    if (USE_UMMA_PREFILL and hd == 64 and page_tokens == 64 and not window and pool.numel() // hd < 2 ** 31
-            and 128 % (H // G) == 0 and max_item_rows * (H // G) >= UMMA_PREFILL_MIN_ROWS):
+    if (hd == 64 and umma_prefill_takes(H, G, hd, hd, page_tokens, window, scale)
+            and max_item_rows * (H // G) >= UMMA_PREFILL_MIN_ROWS):
         # tcgen05: 128 (token, head) rows a CTA, S and P V in tensor memory
-        f = _fn("attention_umma", "fellm_attn_prefill_umma",
-                [_c_p, _c_p, ctypes.c_longlong, _c_p, _c_int, _c_p, _c_p, _c_p, _c_int, _c_int, _c_p, _c_int, _c_int, _c_int,
-                 _c_int, _c_int, _c_int, _c_int, _c_f, _c_int, _c_p, _c_p])
-        _check(f(_p(q), _p(pool), pool.shape[0], _p(block_table), block_table.shape[1], _p(positions), _p(row_slot),
-                 _p(item_start), n_items, max_item_rows, _p(out), T, H, G, hd, page_tokens, layer, pool.shape[1],
-                 float(scale), 0, _p(umma_status(q.device)), _stream()), "attention_prefill (tcgen05)")
-        return out
+        return _prefill_umma(q, H * hd, H, G, hd, hd, pool, block_table, positions, row_slot, item_start, n_items,
+                             max_item_rows, layer, page_tokens, scale, None, out)
     if USE_TMA_PREFILL and hd == 64 and page_tokens == 64 and not window and pool.numel() // hd < 2 ** 31:
         # a key tile is a page: K and V by bulk tensor copies
         f = _fn("attention_mma", "fellm_attn_prefill_tma",
@@ -1852,6 +1903,107 @@ def attention_prefill(q, pool, block_table, positions, row_slot, item_start, n_i
              n_items, max_item_rows, _p(out), T, H, G, hd, page_tokens, layer, pool.shape[1], float(scale),
              int(window or 0), _stream()), "attention_prefill")
     return out
+
+
+def _umma_defines(hd: int, vd: int):
+    return None if hd == vd == 64 else {"AU_KD": hd, "AU_VD": vd}
+
+
+def umma_prefill_takes(H: int, G: int, hd: int, vd: int, page_tokens: int, window, scale: float) -> bool:
+    """Whether the tcgen05 attention of prompt portions takes a layer of these sizes: pages of 64 tokens, no window, a
+    positive scale, 128 rows a whole number of tokens' heads, key and value sizes of a multiple of 16 whose query, score
+    weight and page tiles (two atoms of 64 elements at most each, so four pages fit) and accumulators fit an SM."""
+    if not USE_UMMA_PREFILL or page_tokens != 64 or window or not scale > 0 or G < 1 or H % G or 128 % (H // G):
+        return False
+    if hd % 16 or vd % 16 or min(hd, vd) < 16:
+        return False
+    ka, va = -(-hd // 64), -(-vd // 64)
+    stages = (225 * 1024 - ka * 16384 - 4 * 16384) // ((ka + va) * 8192)
+    return stages >= 4 and 256 + 2 * 32 * -(-vd // 32) <= 512
+
+
+def _prefill_umma(q, ldq, H, G, hd, vd, pool, block_table, positions, row_slot, item_start, n_items, max_item_rows, layer,
+                  page_tokens, scale, sinks, out):
+    T = q.shape[0]
+    f = _fn("attention_umma", "fellm_attn_prefill_umma",
+            [_c_p, _c_int, _c_p, ctypes.c_longlong, _c_p, _c_int, _c_p, _c_p, _c_p, _c_int, _c_int, _c_p, _c_int, _c_int, _c_int,
+             _c_int, _c_int, _c_int, _c_int, _c_int, _c_f, _c_int, _c_p, _c_p, _c_p], defines=_umma_defines(hd, vd))
+    _check(f(_p(q), int(ldq), _p(pool), pool.shape[0], _p(block_table), block_table.shape[1], _p(positions), _p(row_slot),
+             _p(item_start), n_items, max_item_rows, _p(out), T, H, G, hd, vd, page_tokens, layer, pool.shape[1],
+             float(scale), 0, _p(sinks), _p(umma_status(q.device)), _stream()), "attention_prefill (tcgen05)")
+    return out
+
+
+def _mma_defines(hd: int, vd: int):
+    return {"HD": hd} if hd == vd else {"HD": hd, "VD": vd}
+
+
+def written_attention_modules(dtype: str, H: int, G: int, hd: int, vd: int, page_tokens: int, window, scale: float):
+    """The modules attention_written launches for a layer of these sizes."""
+    mods = [("attention_simt", None)]
+    if dtype == "bfloat16" and _mma_takes(H, G, hd, vd):
+        mods.append(("attention_mma", _mma_defines(hd, vd)))
+        if umma_prefill_takes(H, G, hd, vd, page_tokens, window, scale):
+            mods.append(("attention_umma", _umma_defines(hd, vd)))
+    return mods
+
+
+def _mma_takes(H: int, G: int, hd: int, vd: int) -> bool:
+    return (GENERAL_ATTENTION_MMA and hd % 16 == 0 and vd % 16 == 0 and 16 <= hd <= 256 and 16 <= vd <= 256
+            and H // G <= 64)
+
+
+def attention_written(qkv, H, G, hd, vd, cache, ctx, scale, *, window=None, sinks=None, warps=8, out=None):
+    """Attention of a step's rows over pages that already hold the rows' own keys and values (qkv_rotate_write): query head
+    h of row t is qkv[t, h hd : (h + 1) hd] as it lies; keys of hd, values of vd; sinks float32 [H]: exp(sinks[h]) joins
+    head h's softmax denominator.  bfloat16 on tensor cores (portions: tcgen05 where the sizes allow, else mma.sync; single
+    tokens: the key walk split over CTAs), everything else on CUDA cores.  Returns [T, H * vd] in qkv's dtype."""
+    pool, bt, positions, row_slot = cache.pool, cache.block_table, ctx.positions, ctx.row_slot
+    if qkv.dtype != torch.bfloat16 or not _mma_takes(H, G, hd, vd) or qkv.stride(0) % 8 or qkv.data_ptr() % 16 or pool.data_ptr() % 16:
+        return paged_attention_general(qkv, H, hd, vd, pool, bt, positions, row_slot, cache.layer, cache.page_tokens, G, scale,
+                                       window=window, warps=warps, sinks=sinks, out=out)
+    _dev(qkv, pool, bt, positions, row_slot, sinks)
+    T, pt = qkv.shape[0], cache.page_tokens
+    if H % G:
+        raise KernelError(f"attention: {H} heads are not a multiple of {G} kv heads")
+    assert qkv.stride(1) == 1 and qkv.shape[1] >= H * hd and pool.dtype == torch.bfloat16 and pool.is_contiguous()
+    assert pool[0, 0].numel() == G * pt * (hd + vd)
+    if sinks is not None:
+        assert sinks.dtype == torch.float32 and sinks.numel() == H and sinks.is_contiguous()
+    _i32(bt, "block_table"), _i32(positions, "positions"), _i32(row_slot, "row_slot")
+    if out is None:
+        out = torch.empty((T, H * vd), dtype=torch.bfloat16, device=qkv.device)
+    if ctx.all_single:
+        split_len, max_splits = decode_split(ctx.max_len, T, G)
+        scratch, counters = reserve_decode_scratch(pool.device, T, H, G, vd, max_splits)
+        f = _fn("attention_mma", "fellm_attn_decode_mma",
+                [_c_p, _c_int, _c_p, _c_p, _c_int, _c_p, _c_p, _c_p, _c_p, _c_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int,
+                 _c_int, _c_f, _c_int, _c_int, _c_int, _c_p, _c_p], defines=_mma_defines(hd, vd))
+        _check(f(_p(qkv), qkv.stride(0), _p(pool), _p(bt), bt.shape[1], _p(positions), _p(row_slot), _p(out), _p(scratch),
+                 _p(counters), T, H, G, hd, pt, cache.layer, pool.shape[1], float(scale), int(window or 0), split_len,
+                 max_splits, _p(sinks), _stream()), "attention_decode")
+        return out
+    _i32(ctx.item_start, "item_start")
+    if umma_prefill_takes(H, G, hd, vd, pt, window, scale):
+        return _prefill_umma(qkv, qkv.stride(0), H, G, hd, vd, pool, bt, positions, row_slot, ctx.item_start, ctx.n_items,
+                             ctx.max_item_rows, cache.layer, pt, scale, sinks, out)
+    _prefill_biased(qkv, pool, bt, positions, row_slot, ctx.item_start, ctx.n_items, ctx.max_item_rows, out, T, H, G, hd, vd, pt,
+                    cache.layer, scale, window, sinks=sinks)
+    return out
+
+
+def _prefill_biased(qkv, pool, block_table, positions, row_slot, item_start, n_items, max_item_rows, out, T, H, G, hd, vd,
+                    page_tokens, layer, scale, window, *, chunk=None, softcap=None, gate=None, slopes=None, q_temp=None,
+                    values_are_keys=False, sinks=None):
+    qt_coef, qt_every = q_temp if q_temp else (0.0, 0)
+    f = _fn("attention_mma", "fellm_attn_prefill_mma_biased",
+            [_c_p, _c_int, _c_p, _c_p, _c_int, _c_p, _c_p, _c_p, _c_int, _c_int, _c_p, _c_int, _c_int, _c_int, _c_int, _c_int,
+             _c_int, _c_int, _c_f, _c_int, _c_int, _c_f, _c_p, _c_int, _c_p, _c_f, _c_int, _c_int, _c_p, _c_p],
+            defines=_mma_defines(hd, vd))
+    _check(f(_p(qkv), qkv.stride(0), _p(pool), _p(block_table), block_table.shape[1], _p(positions), _p(row_slot),
+             _p(item_start), n_items, max_item_rows, _p(out), T, H, G, hd, page_tokens, layer, pool.shape[1], float(scale),
+             int(window or 0), int(chunk or 0), float(softcap or 0.0), _p(gate), gate.stride(0) if gate is not None else 0,
+             _p(slopes), float(qt_coef), int(qt_every), int(bool(values_are_keys)), _p(sinks), _stream()), "attention_prefill_general")
 
 
 def attention_prefill_general(qkv, H, pool, block_table, positions, row_slot, item_start, n_items, max_item_rows, layer,
@@ -1871,7 +2023,6 @@ def attention_prefill_general(qkv, H, pool, block_table, positions, row_slot, it
         G, page_tokens, hd = pool.shape[3], pool.shape[4], pool.shape[5]
     if slopes is not None:
         assert slopes.dtype == torch.float32 and slopes.numel() == H and slopes.is_contiguous()
-    qt_coef, qt_every = q_temp if q_temp else (0.0, 0)
     if qkv.dtype != torch.bfloat16 or pool.dtype != torch.bfloat16 or hd % 16 or not 16 <= hd <= 256 or H % G or H // G > 64:
         raise KernelError("attention_prefill_general takes bfloat16, head sizes of a multiple of 16 in 16..256, up to 64 heads a kv head")
     assert qkv.stride(1) == 1 and qkv.stride(0) % 2 == 0 and pool.is_contiguous()
@@ -1880,13 +2031,9 @@ def attention_prefill_general(qkv, H, pool, block_table, positions, row_slot, it
         assert gate.dtype == torch.float32 and gate.stride(1) == 1
     if out is None:
         out = torch.empty((T, H * hd), dtype=torch.bfloat16, device=qkv.device)
-    f = _fn("attention_mma", "fellm_attn_prefill_mma_biased",
-            [_c_p, _c_int, _c_p, _c_p, _c_int, _c_p, _c_p, _c_p, _c_int, _c_int, _c_p, _c_int, _c_int, _c_int, _c_int, _c_int,
-             _c_int, _c_int, _c_f, _c_int, _c_int, _c_f, _c_p, _c_int, _c_p, _c_f, _c_int, _c_int, _c_p], defines={"HD": hd})
-    _check(f(_p(qkv), qkv.stride(0), _p(pool), _p(block_table), block_table.shape[1], _p(positions), _p(row_slot),
-             _p(item_start), n_items, max_item_rows, _p(out), T, H, G, hd, page_tokens, layer, pool.shape[1], float(scale),
-             int(window or 0), int(chunk or 0), float(softcap or 0.0), _p(gate), gate.stride(0) if gate is not None else 0,
-             _p(slopes), float(qt_coef), int(qt_every), int(bool(values_are_keys)), _stream()), "attention_prefill_general")
+    _prefill_biased(qkv, pool, block_table, positions, row_slot, item_start, n_items, max_item_rows, out, T, H, G, hd, hd,
+                    page_tokens, layer, scale, window, chunk=chunk, softcap=softcap, gate=gate, slopes=slopes, q_temp=q_temp,
+                    values_are_keys=values_are_keys)
     return out
 
 

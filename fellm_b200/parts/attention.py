@@ -18,7 +18,14 @@ weight) BEHIND the rotation, and `out_gate`, the heads' outputs side by side tim
 (W_g [H v_dim, size], part of the input product) before W_o.  With them the general kernels also take a rotation
 (the rows of the input product are rotated and normed where they lie, ops.qk_rotate_norm, and the cache write and
 the attention read them from there) and a layer that reads another layer's pages; `cache_window` is then the
-window the PAGES are kept for, where other layers with wider windows read them too."""
+window the PAGES are kept for, where other layers with wider windows read them too.
+
+Two more again, `sink` (a learned number per head: exp(sink_h) joins the softmax's denominator once, with no key and no
+value) and `v_mix` (values mixed with those of an earlier layer of the same token, (1 - l) v + l v_first, l the layer's own
+number: 'first' is the layer whose values the others, 'mix', mix with; the mixed value is what the cache keeps).  With
+either of them, or with a rotation whose cos and sin carry a magnitude, one kernel behind the input product rotates q
+where it lies and writes the rotated k and the (mixed) v into the pages (ops.qkv_rotate_write), and attention reads the
+pages: on tensor cores in the bfloat16 engine, keys and values of different sizes included (ops.attention_written)."""
 from __future__ import annotations
 
 import math
@@ -36,7 +43,8 @@ class Attention(Mixer):
     def __init__(self, *, dtype: str, size: int, heads: int, kv_heads: int, head_dim: int, qk_norm: bool,
                  norm_eps: float, position, window=None, shares_cache: bool = False, scale=None, softcap=None,
                  v_dim=None, chunk=None, head_gate: bool = False, bias: bool = False, values_are_keys: bool = False,
-                 slope_exp=None, q_temp=None, unit_qk_norm: bool = False, out_gate: bool = False, cache_window="same"):
+                 slope_exp=None, q_temp=None, unit_qk_norm: bool = False, out_gate: bool = False, cache_window="same",
+                 sink: bool = False, v_mix=None):
         """`position`: a PartSpec of the 'position' category.  `shares_cache`: this layer keeps no
         keys and values (it has no k/v weights) and reads those of the run its schedule entry
         names."""
@@ -46,10 +54,13 @@ class Attention(Mixer):
             raise ConfigError(f"attention: {self.H} heads are not a multiple of {self.G} kv heads")
         self.unit_qk_norm, self.out_gate = bool(unit_qk_norm), bool(out_gate)
         self.in_place = self.unit_qk_norm or self.out_gate        # rotation and norm where the product left q and k
-        general = bool(softcap or chunk or head_gate or (v_dim is not None and int(v_dim) != self.hd) or bias
+        self.sink, self.v_mix = bool(sink), v_mix
+        if self.v_mix not in (None, "first", "mix"):
+            raise ConfigError(f"attention: v_mix is {v_mix!r} (None, 'first' or 'mix')")
+        general = bool(sink or v_mix or softcap or chunk or head_gate or (v_dim is not None and int(v_dim) != self.hd) or bias
                        or values_are_keys or slope_exp or q_temp or self.in_place)
-        if general and not 1 <= self.hd <= 256:
-            raise ConfigError(f"attention: head_dim {self.hd} must be in 1..256")
+        if general and not 1 <= self.hd <= (ops.ATTENTION_SIMT_MAX_HD if sink or v_mix else 256):
+            raise ConfigError(f"attention: head_dim {self.hd} must be in 1..256 (1..1024 with a sink or value mixing)")
         if not general and (self.hd % 16 or not 16 <= self.hd <= 256):       # the tensor-core kernels' sizes
             raise ConfigError(f"attention: head_dim {self.hd} must be a multiple of 16 in 16..256")
         self.qk_norm, self.eps = bool(qk_norm), float(norm_eps)
@@ -87,15 +98,25 @@ class Attention(Mixer):
         # of a row's sums is the same in every step
         span = min(x for x in (self.window, None if chunk is None else int(chunk), 1 << 30) if x)
         self.simt_warps = max(1, min(8, -(-span // 128)))
-        if self.general:
+        # rotation, value mixing and the cache write in one kernel, attention over the pages behind it
+        self.written = self.sink or self.v_mix is not None or (
+            self.position.inv_freq is not None and float(getattr(self.position, "magnitude", 1.0)) != 1.0)
+        if self.written:
+            if self.qk_norm or self.in_place or self.shares_cache or softcap or chunk or head_gate or values_are_keys or slope_exp or q_temp or bias:
+                raise ConfigError("attention: a sink, value mixing or a rotation with a magnitude goes with a cache of the layer's own "
+                                  "and no QK norm, output gate, soft cap, chunk, head gate, bias, distance slopes, query "
+                                  "temperature or values that are keys")
+            self.general = True
+        elif self.general:
             if self.qk_norm or ((self.position.inv_freq is not None or self.shares_cache) and not self.in_place):
                 raise ConfigError("attention: a soft cap, v_dim, chunk or head gate goes with no weighted QK norm and, without "
                                   "unit_qk_norm or out_gate, with no rotation and a cache of the layer's own")
             if self.in_place and (self.hd > 512 or values_are_keys or head_gate or slope_exp or q_temp or bias):
                 raise ConfigError(f"attention: unit_qk_norm and out_gate take heads of up to 512 (got {self.hd}) and go with no "
                                   "bias, head gate, distance slopes, query temperature or values that are keys")
-            if self.vd > 256 or self.vd < 1 or (self.chunk is not None and self.chunk < 1):
-                raise ConfigError(f"attention: v_dim {self.vd} must be in 1..256 and chunk positive")
+        if self.general:
+            if self.vd > (ops.ATTENTION_SIMT_MAX_HD if self.written else 256) or self.vd < 1 or (self.chunk is not None and self.chunk < 1):
+                raise ConfigError(f"attention: v_dim {self.vd} must be in 1..256 (1..1024 with a sink or value mixing) and chunk positive")
         d, H, G, hd = self.size, self.H, self.G, self.hd
         self.decls = {"q_proj.weight": ParamDecl((H * hd, d)), "out_proj.weight": ParamDecl((d, H * self.vd))}
         if not self.shares_cache:
@@ -111,6 +132,10 @@ class Attention(Mixer):
             self.decls["gate.weight"] = ParamDecl((H, d), init=("normal", 0.1))
         if self.out_gate:
             self.decls["out_gate.weight"] = ParamDecl((H * self.vd, d), init=("normal", 0.05))
+        if self.sink:
+            self.decls["sink"] = ParamDecl((H,), role="vector", init=("normal", 1.0))
+        if self.v_mix == "mix":
+            self.decls["vmix"] = ParamDecl((), role="vector", init=("uniform", 0.2, 0.8))
         if self.qk_norm:
             self.decls["q_norm.weight"] = ParamDecl((hd,), role="vector", init=("ones",))
             if not self.shares_cache:
@@ -162,6 +187,9 @@ class Attention(Mixer):
         if self.w["qkv.weight"].dtype == torch.bfloat16 and not self.general:
             floats, counters = ops.decode_scratch_need(max_rows, self.H, self.G, self.hd, n_ctx)
             ops.reserve_decode_scratch(device, 1, self.H, self.G, self.hd, 1, floats=floats, counters=counters)
+        elif self.w["qkv.weight"].dtype == torch.bfloat16 and self.written:
+            floats, counters = ops.decode_scratch_need(max_rows, self.H, self.G, self.vd, n_ctx)
+            ops.reserve_decode_scratch(device, 1, self.H, self.G, self.vd, 1, floats=floats, counters=counters)
 
     can_store = property(lambda self: self.general)        # (the general path's forward(store=True) writes its rows)
 
@@ -199,6 +227,8 @@ class Attention(Mixer):
         qkv = linear(xn, self.w["qkv.weight"], self.w.get("qkv.bias"))
         if self.values_are_keys:
             vd = 0              # nothing is kept beside the keys; the read-out has their size
+        if self.written:
+            return self._forward_written(qkv, ctx, cache, out, store)
         if self.in_place:
             return self._forward_in_place(qkv, ctx, cache, out, store)
         if ctx.all_single:
@@ -208,7 +238,7 @@ class Attention(Mixer):
                                             chunk=self.chunk, softcap=self.softcap, gate=gate,
                                             slopes=self.w.get("slopes"), q_temp=self.q_temp, warps=self.simt_warps,
                                             write_new=(H * hd, (H + G) * hd, ctx.status))
-            linear(a, self.w["out_proj.weight"], self.w.get("out_proj.bias"), out=out, accumulate=True)
+            linear(a, self.w["out_proj.weight"], self.w.get("out_proj.bias"), out=out, accumulate=not store)
             return out
         ops.kv_write(qkv, H * hd, (H + G) * hd, cache.pool, cache.block_table, ctx.positions, ctx.row_slot, cache.layer,
                      cache.page_tokens, G, hd, vd, status=ctx.status)
@@ -224,7 +254,23 @@ class Attention(Mixer):
                                             cache.layer, cache.page_tokens, G, self.scale, window=self.window,
                                             chunk=self.chunk, softcap=self.softcap, gate=gate,
                                             slopes=self.w.get("slopes"), q_temp=self.q_temp, warps=self.simt_warps)
-        linear(a, self.w["out_proj.weight"], self.w.get("out_proj.bias"), out=out, accumulate=True)
+        linear(a, self.w["out_proj.weight"], self.w.get("out_proj.bias"), out=out, accumulate=not store)
+        return out
+
+    def _forward_written(self, qkv, ctx, cache, out, store):
+        H, G, hd, vd = self.H, self.G, self.hd, self.vd
+        v_first = None
+        if self.v_mix == "first":
+            at = (H + G) * hd
+            ctx.carried["v_first"] = qkv[:, at:at + G * vd]           # (as the product left them: nothing writes these columns)
+        elif self.v_mix == "mix":
+            v_first = ctx.carried["v_first"]
+        ops.qkv_rotate_write(qkv, H, G, hd, vd, self.rot_dim, self.position.inv_freq, self.position.pairing,
+                             getattr(self.position, "magnitude", 1.0), ctx.positions, ctx.row_slot, cache, v_first=v_first,
+                             lam=self.w.get("vmix"), status=ctx.status)
+        a = ops.attention_written(qkv, H, G, hd, vd, cache, ctx, self.scale, window=self.window, sinks=self.w.get("sink"),
+                                  warps=self.simt_warps)
+        linear(a, self.w["out_proj.weight"], out=out, accumulate=not store)
         return out
 
     def _forward_in_place(self, qkv, ctx, cache, out, store):
@@ -262,6 +308,9 @@ class Attention(Mixer):
         return [self.w["qkv.weight"], self.w["out_proj.weight"]]
 
     def kernel_modules(self, dtype):
+        if self.written:
+            return linear_modules(dtype) + [("qk_rope_write", None)] + ops.written_attention_modules(
+                dtype, self.H, self.G, self.hd, self.vd, 64, self.window, self.scale)
         if self.general:
             mma = dtype == "bfloat16" and self.vd == self.hd and self.hd % 16 == 0 and self.H // self.G <= 64
             extra = ([("qk_rope_write", None)] if self.in_place else []) + ([("sublayer", None)] if self.out_gate else [])

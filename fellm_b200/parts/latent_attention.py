@@ -12,8 +12,8 @@ Nothing per head is ever stored: with qa_i,h = W_uk,h^T qn_i,h the unrotated par
 sum_j p_ij v_j,h = W_uv,h sum_j p_ij c_j.  So the attention kernel runs over the cached rows [c_j | rot_j(kr_j)] with
 queries [qa_i,h | rot_i(qr_i,h)], one key "head" for all query heads, the keys read as the values and only their
 first rk elements read out; a product per head before it (W_uk^T) and one behind it (W_uv) do the rest.  `scale` is
-the layer's own and is used as given.  The rotation is the position part's (pairs (2i, 2i+1), scaled frequencies and
-a magnitude where the part has them); norms, angles, scores and the softmax are float32 in both engines.
+the layer's own and is used as given.  The rotation is the position part's (pairs (2i, 2i+1) or, r elements being
+rotated, (i, i + r/2); scaled frequencies and a magnitude where the part has them); norms, angles, scores and the softmax are float32 in both engines.
 """
 from __future__ import annotations
 
@@ -31,7 +31,7 @@ class LatentAttention(Mixer):
     def __init__(self, *, dtype: str, size: int, heads: int, dim: int, rot_dim: int, v_dim: int, q_rank: int,
                  kv_rank: int, scale: float, norm_eps: float, position, window=None, sink: bool = False):
         """`dim` / `rot_dim`: the unrotated / rotated elements of a head's query and key; `position`: a PartSpec of the
-        'position' category for the rot_dim part (adjacent pairs; it may rotate fewer than rot_dim elements, or none).
+        'position' category for the rot_dim part (either pairing; it may rotate fewer than rot_dim elements, or none).
         Tensors: dq.weight [q_rank, size], dq.norm [q_rank], uq.weight [heads (dim + rot_dim), q_rank],
         dkv.weight [kv_rank + rot_dim, size], dkv.norm [kv_rank], uk.weight [heads dim, kv_rank],
         uv.weight [heads v_dim, kv_rank], o.weight [size, heads v_dim], sink [heads] (with sink=True)."""
@@ -51,9 +51,8 @@ class LatentAttention(Mixer):
         self.n_rot = 0
         if self.position.inv_freq is not None:
             self.n_rot = int(self.position.rot_dim)
-            if self.position.pairing != "adjacent" or self.n_rot > self.dr:
-                raise ConfigError(f"latent_attention: the rotation pairs neighbours and covers at most rot_dim = {self.dr} "
-                                  f"elements (got {self.position.pairing}, {self.n_rot})")
+            if self.n_rot > self.dr:
+                raise ConfigError(f"latent_attention: the rotation covers at most rot_dim = {self.dr} elements (got {self.n_rot})")
         self.magnitude = float(getattr(self.position, "magnitude", 1.0))
         H, d = self.H, self.size
         self.decls = {"dq.weight": ParamDecl((self.rq, d)), "dq.norm": ParamDecl((self.rq,), role="vector", init=("uniform", 0.5, 1.5)),
@@ -76,6 +75,16 @@ class LatentAttention(Mixer):
     def prepare(self):
         w = self.w
         H, dn, dr, dv, rq, rk = self.H, self.dn, self.dr, self.dv, self.rq, self.rk
+        if self.n_rot and self.position.pairing == "split_half":
+            # The kernels rotate neighbours.  The rotated parts enter the scores alone, as a sum over their elements: the
+            # rows that make element i and element i + n/2 of the queries' and the key's part are put side by side here,
+            # and the sum is the same.
+            half = self.n_rot // 2
+            order = [j for i in range(half) for j in (i, i + half)] + list(range(self.n_rot, dr))
+            take = torch.tensor(order, device=w["uq.weight"].device)
+            uq = w["uq.weight"].view(H, dn + dr, rq)
+            w["uq.weight"] = torch.cat([uq[:, :dn], uq[:, dn:].index_select(1, take)], 1).reshape(H * (dn + dr), rq).contiguous()
+            w["dkv.weight"] = torch.cat([w["dkv.weight"][:rk], w["dkv.weight"][rk:].index_select(0, take)], 0).contiguous()
         # both down projections read the same input: one product, rows [query latent | key-value latent | key part]
         w["down.weight"], offs = stack_rows([w.pop("dq.weight"), w.pop("dkv.weight")])
         self.q_off, self.c_off = offs[0], offs[1]

@@ -45,25 +45,25 @@ class LazyNorm:
         return rms and self._done is None and ops.norm_fusable(self.x, w, self.norm.w["weight"])
 
 
-def linear(x, w, bias=None, *, out=None, out_dtype=None, accumulate=False, swiglu=False):
+def linear(x, w, bias=None, *, out=None, out_dtype=None, accumulate=False, swiglu=False, act=None):
     """x [T, K] (a tensor or a LazyNorm), w [N, K] -> [T, N].  accumulate=True adds into the
     float32 `out` (the residual stream) instead of storing; swiglu=True: w is the interleaved
-    gate/up matrix and the result is SiLU(gate)*up."""
+    gate/up matrix and the result is SiLU(gate)*up; act="relu2": the result is max(., 0)^2 in x's dtype."""
     if isinstance(x, LazyNorm):
         h = x.handed_on()
         if (h is not None and ops.fast_gemm_takes(h.xg, w) and w.data_ptr() % 16 == 0
                 and ops.row_scale_takes(h.rows, w.shape[0], w.shape[1])
                 and not (swiglu and out is not None and out.stride(0) % 8)):
-            return ops.gemm_bf16(h.xg, w, bias, out=out, out_dtype=out_dtype, accumulate=accumulate, swiglu=swiglu,
+            return ops.gemm_bf16(h.xg, w, bias, out=out, out_dtype=out_dtype, accumulate=accumulate, swiglu=swiglu, act=act,
                                  row_scale=(h.ssq, h.parts, x.norm.eps))
         if x.fusable_with(w):
-            return ops.gemm_bf16(x.x, w, bias, out=out, out_dtype=out_dtype, accumulate=accumulate, swiglu=swiglu,
+            return ops.gemm_bf16(x.x, w, bias, out=out, out_dtype=out_dtype, accumulate=accumulate, swiglu=swiglu, act=act,
                                  norm=(x.norm.w["weight"], x.norm.eps))
         x = x.tensor()
     if ops.fast_gemm_takes(x, w):
-        return ops.gemm_bf16(x, w, bias, out=out, out_dtype=out_dtype, accumulate=accumulate, swiglu=swiglu)
+        return ops.gemm_bf16(x, w, bias, out=out, out_dtype=out_dtype, accumulate=accumulate, swiglu=swiglu, act=act)
     assert not swiglu
-    return ops.gemm_simt(x, w, bias, out=out, out_dtype=out_dtype, accumulate=accumulate)
+    return ops.gemm_simt(x, w, bias, out=out, out_dtype=out_dtype, accumulate=accumulate, act=act)
 
 
 def linear_modules(dtype: str):

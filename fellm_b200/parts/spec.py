@@ -42,6 +42,8 @@ class LayerSpec:
     'prenorm': h = x + mixer(norm1(x)); out = h + ffn(norm2(h))   (graph.rs:1650-1777).
     'parallel': h = norm1(x); out = x + mixer(h) + ffn(h).
     'parallel_gated': the same with each sublayer's result through the gates of `gate` on its way into the stream.
+    'sandwich': h = x + norm1b(mixer(norm1(x))); out = h + norm2b(ffn(norm2(h))): `norm1b` and `norm2b` stand on the
+    sublayers' outputs.
     norm1, norm2 and ffn may be None where an arrangement has no use for them (a layer without a
     feed-forward, a block with one norm).  `gate` (category 'gate'): gates on the sublayers' results, for the
     arrangements that use them.  `side` (category 'side'): what every token adds to the stream by itself after the
@@ -53,6 +55,8 @@ class LayerSpec:
     arrangement: str = "prenorm"
     gate: Optional[PartSpec] = None
     side: Optional[PartSpec] = None
+    norm1b: Optional[PartSpec] = None
+    norm2b: Optional[PartSpec] = None
 
 
 @dataclass(frozen=True)
@@ -81,6 +85,7 @@ class ModelSpec:
     schedule: List[Run] = field(default_factory=list)
     connectors: List[PartSpec] = field(default_factory=list)
     shared: List[PartSpec] = field(default_factory=list)        # parts (category 'shared') whose tensors other parts read
+    unused: List[str] = field(default_factory=list)             # tensors a file may hold although no part reads them
 
     def __post_init__(self):
         if not self.schedule:

@@ -47,7 +47,8 @@ def check_and_collect(model, available: Dict[str, tuple]):
     table = model.param_table()
     aliases = model.tied_aliases()
     missing = [n for n in table if n not in available]
-    unexpected = [n for n in available if n not in table and n not in aliases]
+    unused = set(model.spec.unused)
+    unexpected = [n for n in available if n not in table and n not in aliases and n not in unused]
     wrong = []
     for alias, owner in aliases.items():
         if alias in available and owner in available and tuple(available[alias]) != tuple(available[owner]):
