@@ -390,9 +390,27 @@ def nalizen_config(width, ff, layers, vocab):
                 token_side=dict(dim=64), layers=out)
 
 
-DESIGNS = {"robazen": robazen_config, "samusun": samusun_config, "meresun": meresun_config, "nalizen": nalizen_config}
-# the model a design is measured beside (default: LFM2 of the same width, depth, feed-forward and vocabulary)
-BESIDE = {"meresun": "samusun", "nalizen": "samusun"}
+def vofezen_config(width, ff, layers, vocab):
+    """A Vofezen model of real-looking layers at this width: three of four layers are attention with keys of 128 and values
+    of 64 (one head per 64 of width, four per key head), a quarter of a key rotated with frequencies scaled by 8 beyond 4,096
+    positions, a sink per head and values mixed with the first layer's; the fourth is latent attention with heads of 128 +
+    64, values of 128, one head per 128 of width, a key-value latent of 512 and a query latent of 3/4 of the width; every
+    layer with a plain feed-forward of `ff`, norms before and behind every sublayer."""
+    H = max(width // 64, 1)
+    att = dict(dim=128, heads=H, kv_heads=max(H // 4, 1), scale=128 ** -0.5, v_mix=True, vdim=64,
+               rot=dict(base=10000.0, dims=32, scaling=dict(factor=8.0, fast=32.0, original=4096, slow=1.0)))
+    lat = dict(dim=128, heads=max(width // 128, 1), kv_rank=512, q_rank=width * 3 // 4, rot=dict(base=500000.0, dims=64), rot_dim=64,
+               scale=192 ** -0.5, vdim=128)
+    return dict(architecture="Vofezen", vocab=vocab, width=width, norm=dict(eps=1e-5),
+                layers=[dict(type="latent_attention" if i % 4 == 2 else "attention", mixer=lat if i % 4 == 2 else att,
+                             mlp=dict(ff=ff, kind="dense")) for i in range(layers)])
+
+
+DESIGNS = {"robazen": robazen_config, "samusun": samusun_config, "meresun": meresun_config, "nalizen": nalizen_config,
+           "vofezen": vofezen_config}
+# the models a design is measured beside (default: LFM2 of the same width, depth, feed-forward and vocabulary);
+# "lfm2_attention": LFM2 with attention in every layer
+BESIDE = {"meresun": ("samusun",), "nalizen": ("samusun",), "vofezen": ("lfm2_attention", "meresun")}
 
 
 def run_design(design, shapes, layers, batches, steps, warmup):
@@ -410,9 +428,13 @@ def run_design(design, shapes, layers, batches, steps, warmup):
         lfm2["block_auto_adjust_ff_dim"] = False
         width, ff, vocab = lfm2["hidden_size"], lfm2["block_ff_dim"], lfm2["vocab_size"]
         row = {}
-        beside = BESIDE.get(design)
-        other = ("lfm2", lfm2) if beside is None else (beside, DESIGNS[beside](width, ff, layers, vocab))
-        for name, cfg in ((design, DESIGNS[design](width, ff, layers, vocab)), other):
+        models = [(design, DESIGNS[design](width, ff, layers, vocab))]
+        for beside in BESIDE.get(design, ("lfm2",)):
+            if beside == "lfm2_attention":
+                models.append((beside, dict(lfm2, full_attn_idxs=list(range(layers)))))
+            else:
+                models.append((beside, lfm2 if beside == "lfm2" else DESIGNS[beside](width, ff, layers, vocab)))
+        for name, cfg in models:
             ctx_end = PROMPT + warmup + steps + 80
             opts = EngineOptions(dtype="bfloat16", n_ctx=ctx_end, ctx_past_model=True, n_batch=4096, n_ubatch=2048,
                                  page_tokens=64, max_requests=max(batches), max_tokens=max(batches) * ctx_end, cuda_graphs=True)
@@ -584,7 +606,7 @@ def main():
     ap.add_argument("--context", type=int, default=PROMPT)
     ap.add_argument("--design", choices=sorted(DESIGNS), default=None,
                     help="prefill and decode throughput of this design at a few real-looking sizes beside the closest model of "
-                         "equal width, depth and feed-forward (LFM2; Samusun for meresun and nalizen) (--layers layers, default 8; --steps decode steps, default 64); "
+                         "equal width, depth and feed-forward (LFM2; Samusun for meresun and nalizen; LFM2 with attention in every layer and Meresun for vofezen) (--layers layers, default 8; --steps decode steps, default 64); "
                          "prints one line of its own and leaves the headline measurement alone")
     args = ap.parse_args()
 
