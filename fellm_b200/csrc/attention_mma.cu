@@ -48,6 +48,9 @@ __device__ __forceinline__ int tile_off(int row, int chunk) {
 __device__ __forceinline__ int tile_off_v(int row, int chunk) {
   return row * ROWBV + ((SWZV ? (chunk ^ (row & 7)) : chunk) << 4);
 }
+template <int ATOM> __device__ __forceinline__ int atom_off(int row, int chunk) {
+  return (chunk >> 3) * ATOM + row * 128 + (((chunk & 7) ^ (row & 7)) << 4);
+}
 __device__ __forceinline__ void cp_async16(unsigned smem_addr, const void* gmem) {
   asm volatile("cp.async.cg.shared.global [%0], [%1], 16;\n" ::"r"(smem_addr), "l"(gmem));
 }
@@ -82,7 +85,9 @@ __device__ __forceinline__ unsigned pack_bf16(float lo, float hi) {
 // CAPPED: scores are soft-capped, cap * tanh(s * scale / cap), with cap_log2 = cap * log2(e).
 // BIASED: row r's scores are multiplied by rs[r] (a query temperature: the factor of q taken out of the dot product)
 // and sl[r] * (hi[r] - key) is taken off them (a bias by distance; sl = slope * log2(e), hi[r] = the row's position).
-template <int NKT, bool MASKED = true, bool CAPPED = false, bool BIASED = false>
+// ATOM > 0: the tiles lie as bulk tensor copies bring them, 64 elements of every key (128 bytes, swizzled) in ATOM bytes,
+// one such atom after the other; 0: a key's whole row at a time.
+template <int NKT, bool MASKED = true, bool CAPPED = false, bool BIASED = false, int ATOM = 0>
 __device__ __forceinline__ void attend_tile(const unsigned (&qf)[KS][4], unsigned k_s, unsigned v_s, int key0,
                                             const int (&lo)[2], const int (&hi)[2], float scale_log2,
                                             float (&o)[DN][4], float (&m)[2], float (&l)[2], int lane,
@@ -100,7 +105,7 @@ __device__ __forceinline__ void attend_tile(const unsigned (&qf)[KS][4], unsigne
       int row = np * 16 + (lane & 7) + ((lane >> 4) << 3);
       int chunk = ks * 2 + ((lane >> 3) & 1);
       unsigned r[4];
-      ldsm_x4(r, k_s + tile_off(row, chunk));
+      ldsm_x4(r, k_s + (ATOM ? atom_off<ATOM>(row, chunk) : tile_off(row, chunk)));
       mma16816(s[2 * np], qf[ks], r[0], r[1]);
       mma16816(s[2 * np + 1], qf[ks], r[2], r[3]);
     }
@@ -162,7 +167,7 @@ __device__ __forceinline__ void attend_tile(const unsigned (&qf)[KS][4], unsigne
       int row = j * 16 + (lane & 7) + (((lane >> 3) & 1) << 3);
       int chunk = dn * 2 + (lane >> 4);
       unsigned r[4];
-      ldsm_x4_trans(r, v_s + tile_off_v(row, chunk));
+      ldsm_x4_trans(r, v_s + (ATOM ? atom_off<ATOM>(row, chunk) : tile_off_v(row, chunk)));
       mma16816(o[2 * dn], a, r[0], r[1]);
       mma16816(o[2 * dn + 1], a, r[2], r[3]);
     }
@@ -209,7 +214,7 @@ __device__ __forceinline__ void load_q_as_b(unsigned (&qb)[KS][2], F row_ptr, in
 // NKT*8 keys at k_s / v_s against the heads in qb; a key counts iff lo <= key0 + i <= hi.  ot[dm] = O^T of dims
 // dm*16 + g (elements 0, 1: heads 2c, 2c+1) and dm*16 + g + 8 (elements 2, 3); m, l per head 2c, 2c+1 (l: this
 // thread's keys only).
-template <int NKT, bool MASKED>
+template <int NKT, bool MASKED, int ATOM = 0>
 __device__ __forceinline__ void attend_tile_keys_as_rows(const unsigned (&qb)[KS][2], unsigned k_s, unsigned v_s, int key0,
                                                          int lo, int hi, float scale_log2, float (&ot)[VD / 16][4],
                                                          float (&m)[2], float (&l)[2], int lane) {
@@ -226,7 +231,7 @@ __device__ __forceinline__ void attend_tile_keys_as_rows(const unsigned (&qb)[KS
       const int row = b * 16 + (lane & 7) + (((lane >> 3) & 1) << 3);
       const int chunk = ks * 2 + (lane >> 4);
       unsigned r[4];
-      ldsm_x4(r, k_s + tile_off(row, chunk));
+      ldsm_x4(r, k_s + (ATOM ? atom_off<ATOM>(row, chunk) : tile_off(row, chunk)));
       mma16816(s[b], r, qb[ks][0], qb[ks][1]);
     }
   }
@@ -276,7 +281,7 @@ __device__ __forceinline__ void attend_tile_keys_as_rows(const unsigned (&qb)[KS
       const int row = b * 16 + (lane & 7) + ((lane >> 4) << 3);
       const int chunk = dm * 2 + ((lane >> 3) & 1);
       unsigned r[4];
-      ldsm_x4_trans(r, v_s + tile_off_v(row, chunk));
+      ldsm_x4_trans(r, v_s + (ATOM ? atom_off<ATOM>(row, chunk) : tile_off_v(row, chunk)));
       mma16816(ot[dm], r, p0, p1);
     }
   }
@@ -663,7 +668,7 @@ __global__ void __launch_bounds__(DC_WARPS * 32) attention_decode_kernel(AttnArg
 // a third of the instructions of the cp.async kernel, which stays for other head and page sizes.
 // Waits are bounded (a second): a warp that gives up sets *status = 301 and the CTA finishes with
 // what it has.
-#if HD == 64 && VD == 64
+#if (HD == 64 && VD == 64) || defined(WIDE)
 #define DT_PT 64
 #define DT_HALF 32                     // keys per tile: half a page, so that a warp has two tiles in flight
 #define DT_TILE_B (DT_HALF * 128)
@@ -700,6 +705,61 @@ __device__ __forceinline__ void at_tma_load_2d(unsigned dst, const CUtensorMap* 
                ::"r"(dst), "l"(map), "r"(bar), "r"(c0), "r"(c1) : "memory");
 }
 
+__device__ __forceinline__ float ld_cluster_f32(unsigned addr) {
+  float v;
+  asm volatile("ld.shared::cluster.f32 %0, [%1];\n" : "=f"(v) : "r"(addr) : "memory");
+  return v;
+}
+__device__ __forceinline__ unsigned mapa_cta(unsigned smem_addr, unsigned rank) {
+  unsigned r;
+  asm volatile("mapa.shared::cluster.u32 %0, %1, %2;\n" : "=r"(r) : "r"(smem_addr), "r"(rank));
+  return r;
+}
+__device__ __forceinline__ void cluster_barrier() {       // every thread of every CTA of the cluster, the same number of times
+  asm volatile("barrier.cluster.arrive.release.aligned;\n" ::: "memory");
+  asm volatile("barrier.cluster.wait.acquire.aligned;\n" ::: "memory");
+}
+
+// The clusters' merge: the key ranges of a (row, kv head) are the CTAs of one cluster, their records in shared memory
+// ([row][VD + 2] at cta_rec); the first active one adds them up in range order.  Every thread of every CTA, active or not.
+__device__ __forceinline__ void decode_cluster_merges(const AttnArgs& a, const float* cta_rec, bool active, int n_active, int s, int s_lo,
+                                                      int t, int g, int R) {
+  cluster_barrier();                                     // the records of all ranges are written
+  if (active && n_active > 1 && s == s_lo) {
+    const int SW = VD + 2;
+    const unsigned mine = (unsigned)__cvta_generic_to_shared(cta_rec);
+    for (int i = threadIdx.x; i < R * VD; i += DC_WARPS * 32) {
+      const int r = i / VD, d = i - r * VD;
+      float mj[8], lj[8], aj[8];
+#pragma unroll
+      for (int j = 0; j < 8; ++j) {
+        if (j < n_active) {
+          const unsigned rec = mapa_cta(mine + (unsigned)(r * SW) * 4u, (unsigned)(s_lo + j));
+          aj[j] = ld_cluster_f32(rec + d * 4);
+          mj[j] = ld_cluster_f32(rec + VD * 4);
+          lj[j] = ld_cluster_f32(rec + (VD + 1) * 4);
+        } else {
+          aj[j] = 0.f; mj[j] = -INFINITY; lj[j] = 0.f;
+        }
+      }
+      float mx = -INFINITY;
+#pragma unroll
+      for (int j = 0; j < 8; ++j) mx = fmaxf(mx, mj[j]);
+      float lt = 0.f, at = 0.f;
+#pragma unroll
+      for (int j = 0; j < 8; ++j) {
+        const float cj = j < n_active ? exp2f(mj[j] - mx) : 0.f;
+        lt += lj[j] * cj;
+        at += aj[j] * cj;
+      }
+      a.out[((size_t)t * a.H + g * R + r) * VD + d] = __float2bfloat16_rn(a.sinks ? at * denominator_inv(a, g * R + r, mx, lt) : at / lt);
+    }
+  }
+  cluster_barrier();                                     // nobody leaves while its record may be read
+}
+#endif
+
+#if HD == 64 && VD == 64 && !defined(WIDE)
 // The step's own q, k, v taken straight from the QKV product's output [T, (H+2G)*64], so that the
 // per-head RMSNorm, the rotation and the write of k and v into the cache need no kernel of their
 // own (formulas: qk_rope_write.cu).  qkv null: q comes normed and rotated in AttnArgs::q.
@@ -753,21 +813,6 @@ __device__ __forceinline__ float2 norm_rope_head64(const bf16* src, bool norm, f
 }
 
 // NS: half-page stages a warp keeps in flight (2: 64 KB a CTA, three CTAs to an SM; 3: 96 KB, two; 4: 128 KB, one).
-__device__ __forceinline__ float ld_cluster_f32(unsigned addr) {
-  float v;
-  asm volatile("ld.shared::cluster.f32 %0, [%1];\n" : "=f"(v) : "r"(addr) : "memory");
-  return v;
-}
-__device__ __forceinline__ unsigned mapa_cta(unsigned smem_addr, unsigned rank) {
-  unsigned r;
-  asm volatile("mapa.shared::cluster.u32 %0, %1, %2;\n" : "=r"(r) : "r"(smem_addr), "r"(rank));
-  return r;
-}
-__device__ __forceinline__ void cluster_barrier() {       // every thread of every CTA of the cluster, the same number of times
-  asm volatile("barrier.cluster.arrive.release.aligned;\n" ::: "memory");
-  asm volatile("barrier.cluster.wait.acquire.aligned;\n" ::: "memory");
-}
-
 // KR: keys as the MMA's rows (up to 8 heads a kv head).  CL: the key ranges of a (row, kv head) are the CTAs of
 // one cluster (up to 8): their records stay in shared memory and the first active one adds them up in range order
 // through distributed shared memory, instead of records in a scratch buffer, a fence, a counter and the last CTA
@@ -925,38 +970,7 @@ attention_decode_tma_kernel(const __grid_constant__ CUtensorMap pool_map, AttnAr
   if constexpr (!CL) decode_last_cta_merges(a, &sm_last, t, g, R, n_active);
   }                                                        // active
   if constexpr (CL) {
-    cluster_barrier();                                     // the records of all ranges are written
-    if (active && n_active > 1 && s == s_lo) {
-      const int SW = VD + 2;
-      const unsigned mine = (unsigned)__cvta_generic_to_shared(cta_rec);
-      for (int i = threadIdx.x; i < R * HD; i += DC_WARPS * 32) {
-        const int r = i / HD, d = i - r * HD;
-        float mj[8], lj[8], aj[8];
-#pragma unroll
-        for (int j = 0; j < 8; ++j) {
-          if (j < n_active) {
-            const unsigned rec = mapa_cta(mine + (unsigned)(r * SW) * 4u, (unsigned)(s_lo + j));
-            aj[j] = ld_cluster_f32(rec + d * 4);
-            mj[j] = ld_cluster_f32(rec + HD * 4);
-            lj[j] = ld_cluster_f32(rec + (HD + 1) * 4);
-          } else {
-            aj[j] = 0.f; mj[j] = -INFINITY; lj[j] = 0.f;
-          }
-        }
-        float mx = -INFINITY;
-#pragma unroll
-        for (int j = 0; j < 8; ++j) mx = fmaxf(mx, mj[j]);
-        float lt = 0.f, at = 0.f;
-#pragma unroll
-        for (int j = 0; j < 8; ++j) {
-          const float cj = j < n_active ? exp2f(mj[j] - mx) : 0.f;
-          lt += lj[j] * cj;
-          at += aj[j] * cj;
-        }
-        a.out[((size_t)t * a.H + g * R + r) * HD + d] = __float2bfloat16_rn(a.sinks ? at * denominator_inv(a, g * R + r, mx, lt) : at / lt);
-      }
-    }
-    cluster_barrier();                                     // nobody leaves while its record may be read
+    decode_cluster_merges(a, cta_rec, active, n_active, s, s_lo, t, g, R);
   }
 }
 
@@ -1132,6 +1146,278 @@ static int fill_args(AttnArgs& a, const void* q, const void* pool, const int* bl
   return 0;
 }
 
+// ------------------------------------------------------------------------------------ decode, TMA, any sizes
+// Compiled with -DWIDE: single tokens of layers whose keys and values are of any size (a multiple of 16), whose rotation
+// covers a part of the head (with a magnitude) and whose values may be mixed with an earlier layer's; pages of 64 tokens,
+// up to 16 heads a kv head.  As attention_decode_tma_kernel: a warp takes every fourth page of the CTA's key range in
+// halves of 32 keys, the first of them asked for before the wait for the input product; q, k and v come straight from that
+// product's rows [q | k | v]: q is rotated into shared memory, the warp whose tile holds the step's own position puts the
+// rotated k and the (mixed) v into the tile and into the page.  A tile is the atoms of K, then of V: 64 elements of 32
+// keys each; what an atom has beyond the size comes as zeros.
+#ifdef WIDE
+#define DW_ATOM (DT_HALF * 128)
+#define DW_KA ((HD + 63) / 64)
+#define DW_VA ((VD + 63) / 64)
+#define DW_STAGE ((DW_KA + DW_VA) * DW_ATOM)
+
+struct WideFuse {
+  const bf16* qkv; const bf16* v0; const float* lam; const float* inv_freq;
+  int ld, ldv0, rot_dim, pairing;
+  float mag;
+};
+
+__device__ __forceinline__ void dw_tma_load_3d(unsigned dst, const CUtensorMap* map, int c0, int c1, int c2, unsigned bar) {
+  asm volatile("cp.async.bulk.tensor.3d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%3, %4, %5}], [%2];\n"
+               ::"r"(dst), "l"(map), "r"(bar), "r"(c0), "r"(c1), "r"(c2) : "memory");
+}
+// Element e of a head, rotated (sines and cosines of its pairs in sn, cs).
+__device__ __forceinline__ float dw_rotated(const bf16* src, int e, int rot_dim, int pairing, const float* sn, const float* cs) {
+  const float x = __bfloat162float(src[e]);
+  if (e >= rot_dim) return x;
+  const int half = rot_dim >> 1, i = pairing ? (e < half ? e : e - half) : e >> 1;
+  const bool first = pairing ? e < half : !(e & 1);
+  const float y = __bfloat162float(src[pairing ? (first ? e + half : e - half) : (e ^ 1)]);
+  return first ? x * cs[i] - y * sn[i] : x * cs[i] + y * sn[i];
+}
+
+template <int NS, bool KR, bool CL>
+__global__ void __launch_bounds__(DC_WARPS * 32)
+attention_decode_wide_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_constant__ CUtensorMap v_map, AttnArgs a, WideFuse f,
+                             int* status) {
+  FELLM_TRACE_SCOPE(TRACE_ATTENTION_DECODE);
+  extern __shared__ unsigned char smem_raw[];
+  __shared__ __align__(8) unsigned long long bars[DC_WARPS * NS];
+  __shared__ int sm_pages[DC_MAX_PAGES];
+  __shared__ int sm_last;
+  __shared__ __align__(16) bf16 q_s[16 * HD];            // the group's heads, rotated
+  __shared__ float sn_s[HD / 2], cs_s[HD / 2];
+  const int s = blockIdx.x, g = blockIdx.y, t = blockIdx.z;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int pos = a.positions[t];
+  const int kb = (a.window > 0 && pos - a.window + 1 > 0) ? pos - a.window + 1 : 0;
+  // (a launch with fewer key ranges than the longest row has: the last range takes every key behind it)
+  const int s_end = (int)gridDim.x - 1;
+  const int s_lo = min(kb / a.split_len, s_end), s_hi = min(pos / a.split_len, s_end);
+  pdl_launch_dependents();
+  const bool active = s >= s_lo && s <= s_hi;
+  if (!CL && !active) return;
+  const int n_active = s_hi - s_lo + 1;
+  const int R = a.H / a.G;                              // <= 16 (the launcher checks)
+  const unsigned base = ((unsigned)__cvta_generic_to_shared(smem_raw) + 1023u) & ~1023u;      // the swizzle is by address
+  float* merge = (float*)(smem_raw + (base - (unsigned)__cvta_generic_to_shared(smem_raw)));  // over the tiles, once the warps are done
+  float* cta_rec = CL ? merge + DC_WARPS * 16 * (VD + 2) : nullptr;
+  if (active) {
+    const int k0 = max(kb, s * a.split_len), k1 = s == s_end ? pos + 1 : min(pos + 1, (s + 1) * a.split_len);
+    const int* bt = a.block_table + (size_t)a.row_slot[t] * a.max_pages;
+    const int pg0 = k0 / DT_PT, n_pg = (k1 - 1) / DT_PT - pg0 + 1;
+    const bool pages_in_smem = n_pg <= DC_MAX_PAGES;
+    if (pages_in_smem)
+      for (int i = threadIdx.x; i < n_pg; i += DC_WARPS * 32) sm_pages[i] = bt[pg0 + i];
+    if (threadIdx.x < DC_WARPS * NS) at_mbar_init((unsigned)__cvta_generic_to_shared(&bars[threadIdx.x]), 1);
+    asm volatile("fence.mbarrier_init.release.cluster;\n" ::: "memory");
+    __syncthreads();
+    const unsigned stage0 = base + warp * NS * DW_STAGE;
+    const unsigned bar0 = (unsigned)__cvta_generic_to_shared(&bars[warp * NS]);
+    const int my_pages = (n_pg - warp + DC_WARPS - 1) / DC_WARPS;                              // may be <= 0
+    const int n_tiles = my_pages > 0 ? my_pages * 2 : 0;
+    auto request = [&](int q) {                           // lane 0: K and V of the q-th half page of this warp
+      const int lp = pg0 + warp + (q >> 1) * DC_WARPS;
+      const int page = max(pages_in_smem ? sm_pages[lp - pg0] : bt[lp], 0);
+      const int rec = page * a.layers_in_group + a.layer, row = g * DT_PT + (q & 1) * DT_HALF;
+      const unsigned st = stage0 + (q % NS) * DW_STAGE, bar = bar0 + (q % NS) * 8;
+      at_mbar_expect_tx(bar, DW_STAGE);
+#pragma unroll
+      for (int i = 0; i < DW_KA; ++i) dw_tma_load_3d(st + i * DW_ATOM, &k_map, 64 * i, row, rec, bar);
+#pragma unroll
+      for (int i = 0; i < DW_VA; ++i) dw_tma_load_3d(st + (DW_KA + i) * DW_ATOM, &v_map, 64 * i, row, rec, bar);
+    };
+    // The kernel in front (the input product) writes nothing of the cache, and the row of the step's own position is
+    // replaced in its tile: the first tiles are asked for before the wait.
+    if (lane == 0) {
+#pragma unroll
+      for (int q = 0; q < NS; ++q) if (q < n_tiles) request(q);
+    }
+    for (int i = threadIdx.x; i < f.rot_dim / 2; i += DC_WARPS * 32) {
+      float sn, cs;
+      sincosf((float)pos * f.inv_freq[i], &sn, &cs);
+      sn_s[i] = sn * f.mag; cs_s[i] = cs * f.mag;
+    }
+    __syncthreads();
+    pdl_wait(); FELLM_TRACE_WAITED();
+    const bf16* row = f.qkv + (size_t)t * f.ld;
+    for (int i = threadIdx.x; i < R * HD; i += DC_WARPS * 32) {
+      const int r = i / HD, e = i - r * HD;
+      q_s[i] = __float2bfloat16_rn(dw_rotated(row + (size_t)(g * R + r) * HD, e, f.rot_dim, f.pairing, sn_s, cs_s));
+    }
+    __syncthreads();
+    auto q_row = [&](int i) -> const bf16* { return i < R ? q_s + i * HD : nullptr; };
+    unsigned qf[KR ? 1 : KS][4], qb[KR ? KS : 1][2];
+    float o[KR ? 1 : DN][4], ot[KR ? VD / 16 : 1][4], m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
+    if constexpr (KR) {
+      load_q_as_b(qb, q_row, lane);
+#pragma unroll
+      for (int d = 0; d < VD / 16; ++d) { ot[d][0] = ot[d][1] = ot[d][2] = ot[d][3] = 0.f; }
+    } else {
+      load_q(qf, q_row, lane);
+#pragma unroll
+      for (int d = 0; d < DN; ++d) { o[d][0] = o[d][1] = o[d][2] = o[d][3] = 0.f; }
+    }
+    const int lo[2] = {k0, k0}, hi[2] = {k1 - 1, k1 - 1};
+    for (int q = 0; q < n_tiles; ++q) {
+      const unsigned st = stage0 + (q % NS) * DW_STAGE, vt = st + DW_KA * DW_ATOM, bar = bar0 + (q % NS) * 8;
+      const bool arrived = __all_sync(0xffffffffu, at_mbar_wait(bar, (q / NS) & 1));
+      if (!arrived) {
+        if (lane == 0 && status) atomicExch(status, 301);
+        break;
+      }
+      const int key0 = (pg0 + warp + (q >> 1) * DC_WARPS) * DT_PT + (q & 1) * DT_HALF;
+      if (s == s_hi && key0 <= pos && pos < key0 + DT_HALF) {
+        // this tile holds the step's own position; no other CTA or warp reads this page's tile in this step
+        const int lp = pos / DT_PT;
+        const int page = pages_in_smem ? sm_pages[lp - pg0] : bt[lp];
+        bf16* rec = const_cast<bf16*>(a.pool) + ((size_t)max(page, 0) * a.layers_in_group + a.layer) * record_elems(a);
+        bf16* krow = rec + ((size_t)g * DT_PT + (pos - lp * DT_PT)) * HD;
+        bf16* vrow = rec + (size_t)a.G * DT_PT * HD + ((size_t)g * DT_PT + (pos - lp * DT_PT)) * VD;
+        const bf16* ksrc = row + (size_t)(a.H + g) * HD;
+        const bf16* vsrc = row + (size_t)(a.H + a.G) * HD + (size_t)g * VD;
+        const float lam = f.v0 ? *f.lam : 0.f;
+        const int at = pos - key0;
+        for (int e = lane; e < HD; e += 32) {
+          const bf16 v = __float2bfloat16_rn(dw_rotated(ksrc, e, f.rot_dim, f.pairing, sn_s, cs_s));
+          asm volatile("st.shared.b16 [%0], %1;\n" ::"r"(st + atom_off<DW_ATOM>(at, e >> 3) + (e & 7) * 2), "h"(*(const unsigned short*)&v) : "memory");
+          if (page >= 0) krow[e] = v;
+        }
+        for (int e = lane; e < VD; e += 32) {
+          float x = __bfloat162float(vsrc[e]);
+          if (f.v0) x = (1.0f - lam) * x + lam * __bfloat162float(f.v0[(size_t)t * f.ldv0 + g * VD + e]);
+          const bf16 v = __float2bfloat16_rn(x);
+          asm volatile("st.shared.b16 [%0], %1;\n" ::"r"(vt + atom_off<DW_ATOM>(at, e >> 3) + (e & 7) * 2), "h"(*(const unsigned short*)&v) : "memory");
+          if (page >= 0) vrow[e] = v;
+        }
+        if (page < 0 && lane == 0 && status) atomicExch(status, 302);                          // no page mapped for the step's own position
+        __syncwarp();
+      }
+      if (key0 < k1 && key0 + DT_HALF > k0) {              // else: a half page with no key of the range
+        if (key0 + DT_HALF > k1) {
+          // rows past the last key hold whatever the page held before: zero the V rows, so that 0 * V is 0
+          for (int i = (k1 - key0) * CPRV + lane; i < DT_HALF * CPRV; i += 32) st_shared_zero16(vt + atom_off<DW_ATOM>(i / CPRV, i % CPRV));
+          __syncwarp();
+        }
+        const bool edge = key0 < k0 || key0 + DT_HALF > k1;
+        if constexpr (KR) {
+          if (edge) attend_tile_keys_as_rows<DT_HALF / 8, true, DW_ATOM>(qb, st, vt, key0, k0, k1 - 1, a.scale_log2, ot, m, l, lane);
+          else attend_tile_keys_as_rows<DT_HALF / 8, false, DW_ATOM>(qb, st, vt, key0, k0, k1 - 1, a.scale_log2, ot, m, l, lane);
+        } else {
+          if (edge) attend_tile<DT_HALF / 8, true, false, false, DW_ATOM>(qf, st, vt, key0, lo, hi, a.scale_log2, o, m, l, lane);
+          else attend_tile<DT_HALF / 8, false, false, false, DW_ATOM>(qf, st, vt, key0, lo, hi, a.scale_log2, o, m, l, lane);
+        }
+      }
+      __syncwarp();
+      if (q + NS < n_tiles) {
+        asm volatile("fence.proxy.async.shared::cta;\n" ::: "memory");      // this warp's reads before the next copy's writes
+        if (lane == 0) request(q + NS);
+      }
+    }
+    __syncthreads();                                         // every warp has left its tiles
+    if constexpr (KR) decode_warps_to_cta_keys_as_rows(a, ot, m, l, merge, warp, lane, t, g, R, s - s_lo, n_active, cta_rec);
+    else decode_warps_to_cta(a, o, m, l, merge, warp, lane, t, g, 0, R, s - s_lo, n_active, cta_rec);
+    if constexpr (!CL) decode_last_cta_merges(a, &sm_last, t, g, R, n_active);
+  }
+  if constexpr (CL) decode_cluster_merges(a, cta_rec, active, n_active, s, s_lo, t, g, R);
+}
+
+// A page-layer record's keys (or values) as a 3-D tensor [elements, rows of all kv heads, records]; a box: 64 elements of
+// half a page of one kv head.  Kept per (base, records, G).
+typedef CUresult (*DwEncodeTiledFn)(CUtensorMap*, CUtensorMapDataType, cuuint32_t, void*, const cuuint64_t*, const cuuint64_t*,
+                                    const cuuint32_t*, const cuuint32_t*, CUtensorMapInterleave, CUtensorMapSwizzle,
+                                    CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
+static int dw_pool_map(const bf16* base, int size, long long records, int G, CUtensorMap* out) {
+  static std::mutex mu;
+  static struct { const void* base; long long records; int G, size; CUtensorMap map; } cache[16];
+  static int n_cached = 0, next = 0;
+  std::lock_guard<std::mutex> lock(mu);
+  for (int i = 0; i < n_cached; ++i)
+    if (cache[i].base == base && cache[i].records == records && cache[i].G == G && cache[i].size == size) { *out = cache[i].map; return 0; }
+  static DwEncodeTiledFn fn = nullptr;
+  if (!fn) {
+    void* p = nullptr;
+    cudaDriverEntryPointQueryResult q;
+    if (cudaGetDriverEntryPoint("cuTensorMapEncodeTiled", &p, cudaEnableDefault, &q) != cudaSuccess || q != cudaDriverEntryPointSuccess)
+      return FELLM_ERR_ARG;
+    fn = (DwEncodeTiledFn)p;
+  }
+  cuuint64_t dims[3] = {(cuuint64_t)size, (cuuint64_t)G * DT_PT, (cuuint64_t)records};
+  cuuint64_t strides[2] = {(cuuint64_t)size * 2, (cuuint64_t)G * DT_PT * (HD + VD) * 2};
+  cuuint32_t box[3] = {64, DT_HALF, 1};
+  cuuint32_t estr[3] = {1, 1, 1};
+  CUtensorMap m;
+  CUresult r = fn(&m, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, const_cast<bf16*>(base), dims, strides, box, estr,
+                  CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_128B,
+                  CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+  if (r != CUDA_SUCCESS) return 1000 + (int)r;
+  cache[next].base = base; cache[next].records = records; cache[next].G = G; cache[next].size = size; cache[next].map = m;
+  next = (next + 1) % 16;
+  if (n_cached < 16) ++n_cached;
+  *out = m;
+  return 0;
+}
+
+template <int NS>
+static int launch_wide(const CUtensorMap& k_map, const CUtensorMap& v_map, const AttnArgs& a, const WideFuse& f, int* status, bool cl, cudaStream_t stream) {
+  const size_t tiles = (size_t)DC_WARPS * NS * DW_STAGE, mrg = (size_t)(DC_WARPS + 1) * 16 * (VD + 2) * sizeof(float);
+  const size_t smem = (tiles > mrg ? tiles : mrg) + 1024;
+  const bool kr = a.H / a.G <= 8;
+  void (*kern)(const CUtensorMap, const CUtensorMap, AttnArgs, WideFuse, int*) =
+      kr ? (cl ? attention_decode_wide_kernel<NS, true, true> : attention_decode_wide_kernel<NS, true, false>)
+         : (cl ? attention_decode_wide_kernel<NS, false, true> : attention_decode_wide_kernel<NS, false, false>);
+  cudaError_t ce = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+  if (ce != cudaSuccess) return (int)ce;
+  return launch_k_class(1, kern, dim3(a.max_splits, a.G, a.T), dim3(DC_WARPS * 32), smem, stream, cl ? a.max_splits : 1, k_map, v_map, a, f, status);
+}
+#endif
+
+// Single tokens through the kernel above (libraries compiled with -DWIDE; FELLM_ERR_SIZE otherwise and for sizes it does not
+// take).  qkv [T, ld]: the input product's rows [q (H hd) | k (G hd) | v (G vd)]; v0 (or null) [T, ldv0] with lam (one float
+// on the device): the values the layer's are mixed with; inv_freq [rot_dim / 2] or null, pairing 0 adjacent / 1 split-half,
+// cos and sin times mag; sinks [H] or null; scratch and counters as fellm_attn_decode_mma; stages: half pages a warp keeps in
+// flight (2, or 4 where they fit); status 301: a wait ran out, 302: a row's position has no page.
+FELLM_API int fellm_attn_decode_wide(const void* qkv, int ld, const void* pool, long long n_pages, const int* block_table, int max_pages,
+                                     const int* positions, const int* row_slot, void* out, float* scratch, int* counters, int T, int H,
+                                     int G, int hd, int vd, int page_tokens, int layer, int layers_in_group, float scale, int window,
+                                     int split_len, int max_splits, const float* inv_freq, int rot_dim, int pairing, float mag,
+                                     const void* v0, int ldv0, const float* lam, const float* sinks, int stages, int cluster, int* status,
+                                     cudaStream_t stream) {
+#ifdef WIDE
+  if (T <= 0) return 0;
+  if (vd != VD) return FELLM_ERR_SIZE;
+  AttnArgs a;
+  int e = fill_args(a, qkv, pool, block_table, max_pages, positions, row_slot, out, T, H, G, hd, page_tokens, layer,
+                    layers_in_group, scale, window);
+  if (e) return e;
+  if (!scratch || !counters || split_len < 1 || max_splits < 1 || (v0 && !lam)) return FELLM_ERR_ARG;
+  if (!inv_freq) rot_dim = 0;
+  const long long records = n_pages * layers_in_group;
+  if (page_tokens != DT_PT || H / G > 16 || (split_len % DT_PT) || records >= (1ll << 31) || ((uintptr_t)pool & 15) ||
+      ld < H * hd + G * (hd + vd) || (v0 && ldv0 < G * vd) || rot_dim < 0 || rot_dim > hd || (rot_dim & 1)) return FELLM_ERR_SIZE;
+  a.ldq = ld; a.sinks = sinks; a.scratch = scratch; a.counters = counters; a.split_len = split_len; a.max_splits = max_splits;
+  WideFuse f;
+  f.qkv = (const bf16*)qkv; f.v0 = (const bf16*)v0; f.lam = lam; f.inv_freq = inv_freq; f.ld = ld; f.ldv0 = ldv0;
+  f.rot_dim = rot_dim; f.pairing = pairing; f.mag = mag;
+  CUtensorMap k_map, v_map;
+  e = dw_pool_map((const bf16*)pool, HD, records, G, &k_map);
+  if (!e) e = dw_pool_map((const bf16*)pool + (size_t)G * DT_PT * HD, VD, records, G, &v_map);
+  if (e) return e;
+  const bool cl = cluster && max_splits >= 2 && max_splits <= 8;
+  if constexpr (DC_WARPS * 4 * DW_STAGE <= 216 * 1024) {
+    if (stages >= 4) return launch_wide<4>(k_map, v_map, a, f, status, cl, stream);
+  }
+  if constexpr (DC_WARPS * 2 * DW_STAGE <= 216 * 1024) return launch_wide<2>(k_map, v_map, a, f, status, cl, stream);
+  else return FELLM_ERR_SIZE;
+#else
+  return FELLM_ERR_SIZE;
+#endif
+}
+
 FELLM_API int fellm_attn_head_dim() { return HD; }
 FELLM_API int fellm_attn_value_dim() { return VD; }
 
@@ -1242,7 +1528,7 @@ FELLM_API int fellm_attn_decode_tma(const void* q, const void* pool, long long n
                                     int layer, int layers_in_group, float scale, int window, int split_len,
                                     int max_splits, int* status, const void* qkv, const float* q_w, const float* k_w,
                                     float eps, const float* inv_freq, int pairing, int stages, cudaStream_t stream) {
-#if HD == 64 && VD == 64
+#if HD == 64 && VD == 64 && !defined(WIDE)
   if (T <= 0) return 0;
   AttnArgs a;
   if (!q) q = qkv;
@@ -1311,7 +1597,7 @@ FELLM_API int fellm_attn_prefill_tma(const void* q, const void* pool, long long 
                                      int n_items, int max_item_rows, void* out, int T, int H, int G, int hd,
                                      int page_tokens, int layer, int layers_in_group, float scale, int window,
                                      int* status, cudaStream_t stream) {
-#if HD == 64 && VD == 64
+#if HD == 64 && VD == 64 && !defined(WIDE)
   if (T <= 0 || n_items <= 0) return 0;
   AttnArgs a;
   int e = fill_args(a, q, pool, block_table, max_pages, positions, row_slot, out, T, H, G, hd, page_tokens, layer,

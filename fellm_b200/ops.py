@@ -1934,15 +1934,104 @@ def _prefill_umma(q, ldq, H, G, hd, vd, pool, block_table, positions, row_slot, 
     return out
 
 
-def _mma_defines(hd: int, vd: int):
-    return {"HD": hd} if hd == vd else {"HD": hd, "VD": vd}
+def _mma_defines(hd: int, vd: int, wide: bool = False):
+    d = {"HD": hd} if hd == vd else {"HD": hd, "VD": vd}
+    if wide and _wide_stage_bytes(hd, vd) * 8 <= 216 * 1024:
+        d["WIDE"] = 1                   # with the decode kernel that takes the input product's rows as they are
+    return d
+
+
+USE_WIDE_DECODE = os.environ.get("FELLM_B200_WIDE_DECODE", "1") != "0"
+WIDE_MAX_RANGES = int(os.environ.get("FELLM_B200_WIDE_MAX_RANGES", 8))
+WIDE_STAGES = int(os.environ.get("FELLM_B200_WIDE_STAGES", 0))
+WIDE_CLUSTER = os.environ.get("FELLM_B200_WIDE_CLUSTER", "1") != "0"
+
+
+def _wide_stage_bytes(hd: int, vd: int) -> int:
+    """Bytes of 32 keys and their values in shared memory (whole atoms of 64 elements)."""
+    return (-(-hd // 64) + -(-vd // 64)) * 4096
+
+
+def decode_wide_takes(qkv, H: int, G: int, hd: int, vd: int, page_tokens: int, pool) -> bool:
+    """Whether attention_decode_wide takes a layer of these sizes (it then needs no qkv_rotate_write in front)."""
+    return (USE_WIDE_DECODE and qkv.dtype == torch.bfloat16 and pool.dtype == torch.bfloat16 and page_tokens == 64
+            and _mma_takes(H, G, hd, vd) and H // G <= 16 and _wide_stage_bytes(hd, vd) * 8 <= 216 * 1024
+            and pool.data_ptr() % 16 == 0)
+
+
+def decode_wide_plan(max_len: int, rows: int, kv_heads: int, hd: int, vd: int):
+    """(split_len, ranges, stages, cluster): the key ranges of a row and kv head, how many half pages a warp keeps in flight,
+    and whether the ranges merge as one cluster.  Chosen for contexts up to the next multiple of 1,024."""
+    bucket = -(-max(max_len, 1) // 1024) * 1024
+    items = max(rows * kv_heads, 1)
+    stage = _wide_stage_bytes(hd, vd)
+    per_sm = max(1, 227 * 1024 // (8 * stage + 9 * 1024 + 32 * hd))
+    want = max(1, min(WIDE_MAX_RANGES, per_sm * sm_count() // items))
+    split_len = max(64, -(-(-(-bucket // want)) // 64) * 64)
+    if split_len > 256:
+        split_len = -(-split_len // 256) * 256          # whole rounds of the kernel's four warps, a page each
+    ranges = -(-bucket // split_len)
+    stages = 2
+    if 16 * stage <= 216 * 1024 and items * ranges <= sm_count():
+        stages = 4                                      # one CTA an SM anyway: twice as much on the way
+    if WIDE_STAGES:
+        stages = WIDE_STAGES
+    cluster = WIDE_CLUSTER and 2 <= ranges <= 8 and items * ranges <= sm_count() * (per_sm if stages == 2 else 1)
+    return split_len, ranges, stages, cluster
+
+
+def decode_wide_scratch_need(max_rows: int, heads: int, kv_heads: int, hd: int, vd: int, n_ctx: int):
+    """(floats, counters) attention_decode_wide can ask for with up to max_rows rows and contexts up to n_ctx."""
+    floats = 0
+    for rows in range(1, max(max_rows, 1) + 1):
+        for bucket in range(1024, max(n_ctx, 1) + 1024, 1024):
+            floats = max(floats, rows * heads * decode_wide_plan(bucket, rows, kv_heads, hd, vd)[1] * (vd + 2))
+    return floats, max(max_rows, 1) * kv_heads
+
+
+def attention_decode_wide(qkv, H, G, hd, vd, cache, ctx, scale, *, rot_dim=0, inv_freq=None, pairing="split_half", mag=1.0, v_first=None,
+                          lam=None, window=None, sinks=None, out=None):
+    """A decode step (every row its request's only one) straight from the input product's rows [q (H hd) | k (G hd) | v (G
+    vd)]: what qkv_rotate_write and attention_written do, in one kernel (see decode_wide_takes); q stays as it was in
+    qkv.  Returns [T, H * vd]."""
+    pool, bt = cache.pool, cache.block_table
+    _dev(qkv, inv_freq, ctx.positions, ctx.row_slot, pool, bt, v_first, lam, sinks)
+    T = qkv.shape[0]
+    assert decode_wide_takes(qkv, H, G, hd, vd, cache.page_tokens, pool)
+    assert qkv.stride(1) == 1 and qkv.shape[1] >= H * hd + G * (hd + vd) and pool.is_contiguous()
+    assert pool[0, 0].numel() == G * cache.page_tokens * (hd + vd)
+    rot_dim = 0 if inv_freq is None else int(rot_dim)
+    if rot_dim % 2 or not 0 <= rot_dim <= hd:
+        raise KernelError(f"attention_decode_wide: rotated part {rot_dim} must be even and within the head ({hd})")
+    if inv_freq is not None:
+        assert inv_freq.dtype == torch.float32 and inv_freq.numel() == rot_dim // 2 and inv_freq.is_contiguous()
+    if v_first is not None:
+        assert v_first.shape == (T, G * vd) and v_first.dtype == qkv.dtype and v_first.stride(1) == 1
+        assert lam is not None and lam.dtype == torch.float32 and lam.numel() == 1
+    if sinks is not None:
+        assert sinks.dtype == torch.float32 and sinks.numel() == H and sinks.is_contiguous()
+    _i32(ctx.positions, "positions"), _i32(ctx.row_slot, "row_slot"), _i32(bt, "block_table")
+    split_len, ranges, stages, cluster = decode_wide_plan(ctx.max_len, T, G, hd, vd)
+    scratch, counters = reserve_decode_scratch(pool.device, T, H, G, vd, ranges)
+    if out is None:
+        out = torch.empty((T, H * vd), dtype=torch.bfloat16, device=qkv.device)
+    f = _fn("attention_mma", "fellm_attn_decode_wide",
+            [_c_p, _c_int, _c_p, _c_ll, _c_p, _c_int, _c_p, _c_p, _c_p, _c_p, _c_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int,
+             _c_int, _c_f, _c_int, _c_int, _c_int, _c_p, _c_int, _c_int, _c_f, _c_p, _c_int, _c_p, _c_p, _c_int, _c_int, _c_p, _c_p],
+            defines=_mma_defines(hd, vd, True))
+    _check(f(_p(qkv), qkv.stride(0), _p(pool), pool.shape[0], _p(bt), bt.shape[1], _p(ctx.positions), _p(ctx.row_slot), _p(out),
+             _p(scratch), _p(counters), T, H, G, hd, vd, cache.page_tokens, cache.layer, pool.shape[1], float(scale), int(window or 0),
+             split_len, ranges, _p(inv_freq), rot_dim, PAIRINGS[pairing], float(mag), _p(v_first),
+             v_first.stride(0) if v_first is not None else 0, _p(lam), _p(sinks), stages, int(cluster), _p(umma_status(pool.device)),
+             _stream()), "attention_decode_wide")
+    return out
 
 
 def written_attention_modules(dtype: str, H: int, G: int, hd: int, vd: int, page_tokens: int, window, scale: float):
     """The modules attention_written launches for a layer of these sizes."""
     mods = [("attention_simt", None)]
     if dtype == "bfloat16" and _mma_takes(H, G, hd, vd):
-        mods.append(("attention_mma", _mma_defines(hd, vd)))
+        mods.append(("attention_mma", _mma_defines(hd, vd, True)))
         if umma_prefill_takes(H, G, hd, vd, page_tokens, window, scale):
             mods.append(("attention_umma", _umma_defines(hd, vd)))
     return mods
@@ -1978,7 +2067,7 @@ def attention_written(qkv, H, G, hd, vd, cache, ctx, scale, *, window=None, sink
         scratch, counters = reserve_decode_scratch(pool.device, T, H, G, vd, max_splits)
         f = _fn("attention_mma", "fellm_attn_decode_mma",
                 [_c_p, _c_int, _c_p, _c_p, _c_int, _c_p, _c_p, _c_p, _c_p, _c_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int,
-                 _c_int, _c_f, _c_int, _c_int, _c_int, _c_p, _c_p], defines=_mma_defines(hd, vd))
+                 _c_int, _c_f, _c_int, _c_int, _c_int, _c_p, _c_p], defines=_mma_defines(hd, vd, True))
         _check(f(_p(qkv), qkv.stride(0), _p(pool), _p(bt), bt.shape[1], _p(positions), _p(row_slot), _p(out), _p(scratch),
                  _p(counters), T, H, G, hd, pt, cache.layer, pool.shape[1], float(scale), int(window or 0), split_len,
                  max_splits, _p(sinks), _stream()), "attention_decode")
@@ -1988,18 +2077,18 @@ def attention_written(qkv, H, G, hd, vd, cache, ctx, scale, *, window=None, sink
         return _prefill_umma(qkv, qkv.stride(0), H, G, hd, vd, pool, bt, positions, row_slot, ctx.item_start, ctx.n_items,
                              ctx.max_item_rows, cache.layer, pt, scale, sinks, out)
     _prefill_biased(qkv, pool, bt, positions, row_slot, ctx.item_start, ctx.n_items, ctx.max_item_rows, out, T, H, G, hd, vd, pt,
-                    cache.layer, scale, window, sinks=sinks)
+                    cache.layer, scale, window, sinks=sinks, wide=True)
     return out
 
 
 def _prefill_biased(qkv, pool, block_table, positions, row_slot, item_start, n_items, max_item_rows, out, T, H, G, hd, vd,
                     page_tokens, layer, scale, window, *, chunk=None, softcap=None, gate=None, slopes=None, q_temp=None,
-                    values_are_keys=False, sinks=None):
+                    values_are_keys=False, sinks=None, wide=False):
     qt_coef, qt_every = q_temp if q_temp else (0.0, 0)
     f = _fn("attention_mma", "fellm_attn_prefill_mma_biased",
             [_c_p, _c_int, _c_p, _c_p, _c_int, _c_p, _c_p, _c_p, _c_int, _c_int, _c_p, _c_int, _c_int, _c_int, _c_int, _c_int,
              _c_int, _c_int, _c_f, _c_int, _c_int, _c_f, _c_p, _c_int, _c_p, _c_f, _c_int, _c_int, _c_p, _c_p],
-            defines=_mma_defines(hd, vd))
+            defines=_mma_defines(hd, vd, wide))
     _check(f(_p(qkv), qkv.stride(0), _p(pool), _p(block_table), block_table.shape[1], _p(positions), _p(row_slot),
              _p(item_start), n_items, max_item_rows, _p(out), T, H, G, hd, page_tokens, layer, pool.shape[1], float(scale),
              int(window or 0), int(chunk or 0), float(softcap or 0.0), _p(gate), gate.stride(0) if gate is not None else 0,

@@ -25,7 +25,8 @@ value) and `v_mix` (values mixed with those of an earlier layer of the same toke
 number: 'first' is the layer whose values the others, 'mix', mix with; the mixed value is what the cache keeps).  With
 either of them, or with a rotation whose cos and sin carry a magnitude, one kernel behind the input product rotates q
 where it lies and writes the rotated k and the (mixed) v into the pages (ops.qkv_rotate_write), and attention reads the
-pages: on tensor cores in the bfloat16 engine, keys and values of different sizes included (ops.attention_written)."""
+pages: on tensor cores in the bfloat16 engine, keys and values of different sizes included (ops.attention_written).  In a
+decode step of the bfloat16 engine the attention kernel does both (ops.attention_decode_wide)."""
 from __future__ import annotations
 
 import math
@@ -189,6 +190,7 @@ class Attention(Mixer):
             ops.reserve_decode_scratch(device, 1, self.H, self.G, self.hd, 1, floats=floats, counters=counters)
         elif self.w["qkv.weight"].dtype == torch.bfloat16 and self.written:
             floats, counters = ops.decode_scratch_need(max_rows, self.H, self.G, self.vd, n_ctx)
+            floats = max(floats, ops.decode_wide_scratch_need(max_rows, self.H, self.G, self.hd, self.vd, n_ctx)[0])
             ops.reserve_decode_scratch(device, 1, self.H, self.G, self.vd, 1, floats=floats, counters=counters)
 
     can_store = property(lambda self: self.general)        # (the general path's forward(store=True) writes its rows)
@@ -265,9 +267,16 @@ class Attention(Mixer):
             ctx.carried["v_first"] = qkv[:, at:at + G * vd]           # (as the product left them: nothing writes these columns)
         elif self.v_mix == "mix":
             v_first = ctx.carried["v_first"]
-        ops.qkv_rotate_write(qkv, H, G, hd, vd, self.rot_dim, self.position.inv_freq, self.position.pairing,
-                             getattr(self.position, "magnitude", 1.0), ctx.positions, ctx.row_slot, cache, v_first=v_first,
-                             lam=self.w.get("vmix"), status=ctx.status)
+        mag = getattr(self.position, "magnitude", 1.0)
+        if ctx.all_single and ops.decode_wide_takes(qkv, H, G, hd, vd, cache.page_tokens, cache.pool):
+            # a decode step: rotation, mixing and the cache write happen inside the attention kernel
+            a = ops.attention_decode_wide(qkv, H, G, hd, vd, cache, ctx, self.scale, rot_dim=self.rot_dim, inv_freq=self.position.inv_freq,
+                                          pairing=self.position.pairing, mag=mag, v_first=v_first, lam=self.w.get("vmix"),
+                                          window=self.window, sinks=self.w.get("sink"))
+            linear(a, self.w["out_proj.weight"], out=out, accumulate=not store)
+            return out
+        ops.qkv_rotate_write(qkv, H, G, hd, vd, self.rot_dim, self.position.inv_freq, self.position.pairing, mag, ctx.positions,
+                             ctx.row_slot, cache, v_first=v_first, lam=self.w.get("vmix"), status=ctx.status)
         a = ops.attention_written(qkv, H, G, hd, vd, cache, ctx, self.scale, window=self.window, sinks=self.w.get("sink"),
                                   warps=self.simt_warps)
         linear(a, self.w["out_proj.weight"], out=out, accumulate=not store)
