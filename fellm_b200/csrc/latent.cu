@@ -72,6 +72,74 @@ latent_prep_kernel(const float* __restrict__ z, int ldz, int q_off, int rq, int 
   for (int i = n_rot + threadIdx.x; i < dr; i += blockDim.x) rec[rk + i] = from_f<TC>(zr[r_off + i]);
 }
 
+__device__ __forceinline__ void lp_put4(float* o, float4 v) { *(float4*)o = v; }
+__device__ __forceinline__ void lp_put4(bf16* o, float4 v) {
+  const __nv_bfloat162 p0 = __floats2bfloat162_rn(v.x, v.y), p1 = __floats2bfloat162_rn(v.z, v.w);
+  *(uint2*)o = make_uint2(*(const unsigned*)&p0, *(const unsigned*)&p1);
+}
+
+// The same where every part is a multiple of 4 and lies on 16 bytes: 16-byte loads, a row's latents kept in registers
+// between the sums and the results (LP_VPT vectors a thread), the page's number and the rotation's sines and cosines
+// (a pair a thread) before the wait for the product.
+#define LP_THREADS 256
+#define LP_VPT 4
+template <typename TO, typename TC>
+__global__ void __launch_bounds__(LP_THREADS)
+latent_prep_vec_kernel(const float* __restrict__ z, int ldz, int q_off, int rq, int c_off, int rk, int r_off, int dr,
+                       const float* __restrict__ wq, const float* __restrict__ wc, float eps,
+                       const float* __restrict__ freq, int n_rot, float mag,
+                       const int* __restrict__ positions, const int* __restrict__ row_slot,
+                       const int* __restrict__ block_table, int max_pages, TC* __restrict__ pool, int page_tokens, int layer,
+                       int layers_in_group, TO* __restrict__ cq, int* __restrict__ status) {
+  __shared__ float part[2][LP_THREADS / 32];
+  pdl_launch_dependents();
+  const int row = blockIdx.x, tid = threadIdx.x, nq = rq >> 2, nv = nq + (rk >> 2);
+  const int pos = positions[row];
+  const int page = block_table[(size_t)row_slot[row] * max_pages + pos / page_tokens];
+  float sn = 0.f, cs = 0.f;
+  if (tid < n_rot / 2) { sincosf((float)pos * freq[tid], &sn, &cs); sn *= mag; cs *= mag; }
+  pdl_wait();
+  const float* zr = z + (size_t)row * ldz;
+  float4 v[LP_VPT];
+  float sq = 0.f, sc = 0.f;
+#pragma unroll
+  for (int j = 0; j < LP_VPT; ++j) {
+    const int i = tid + j * LP_THREADS;
+    v[j] = i < nv ? *(const float4*)(zr + (i < nq ? q_off + 4 * i : c_off + 4 * (i - nq))) : make_float4(0.f, 0.f, 0.f, 0.f);
+  }
+#pragma unroll
+  for (int j = 0; j < LP_VPT; ++j) {
+    const float t = fmaf(v[j].x, v[j].x, fmaf(v[j].y, v[j].y, fmaf(v[j].z, v[j].z, v[j].w * v[j].w)));
+    if (tid + j * LP_THREADS < nq) sq += t; else sc += t;
+  }
+  sq = warp_sum(sq); sc = warp_sum(sc);
+  if ((tid & 31) == 0) { part[0][tid >> 5] = sq; part[1][tid >> 5] = sc; }
+  __syncthreads();
+  sq = sc = 0.f;
+#pragma unroll
+  for (int i = 0; i < LP_THREADS / 32; ++i) { sq += part[0][i]; sc += part[1][i]; }
+  sq = 1.0f / sqrtf(sq / (float)rq + eps); sc = 1.0f / sqrtf(sc / (float)rk + eps);
+  if (page < 0 && tid == 0 && status) atomicExch(status, 2);
+  TC* rec = pool + (((size_t)max(page, 0) * layers_in_group + layer) * page_tokens + (pos % page_tokens)) * (rk + dr);
+#pragma unroll
+  for (int j = 0; j < LP_VPT; ++j) {
+    const int i = tid + j * LP_THREADS;
+    if (i < nq) {
+      const float4 w = *(const float4*)(wq + 4 * i);
+      lp_put4(cq + (size_t)row * rq + 4 * i, make_float4((v[j].x * sq) * w.x, (v[j].y * sq) * w.y, (v[j].z * sq) * w.z, (v[j].w * sq) * w.w));
+    } else if (i < nv && page >= 0) {
+      const float4 w = *(const float4*)(wc + 4 * (i - nq));
+      lp_put4(rec + 4 * (i - nq), make_float4((v[j].x * sc) * w.x, (v[j].y * sc) * w.y, (v[j].z * sc) * w.z, (v[j].w * sc) * w.w));
+    }
+  }
+  if (page < 0) return;
+  if (tid < n_rot / 2) {
+    const float a = zr[r_off + 2 * tid], b = zr[r_off + 2 * tid + 1];
+    rec[rk + 2 * tid] = from_f<TC>(a * cs - b * sn); rec[rk + 2 * tid + 1] = from_f<TC>(b * cs + a * sn);
+  }
+  for (int i = n_rot + tid; i < dr; i += LP_THREADS) rec[rk + i] = from_f<TC>(zr[r_off + i]);
+}
+
 FELLM_API int fellm_latent_prep(const float* z, int ldz, int q_off, int rq, int c_off, int rk, int r_off, int dr,
                                 const float* wq, const float* wc, float eps, const float* freq, int n_rot, float mag,
                                 const int* positions, const int* row_slot, const int* block_table, int max_pages,
@@ -81,6 +149,16 @@ FELLM_API int fellm_latent_prep(const float* z, int ldz, int q_off, int rq, int 
   if (!z || !wq || !wc || !positions || !row_slot || !block_table || !pool || !cq) return FELLM_ERR_ARG;
   if (rq < 1 || rk < 1 || dr < 0 || n_rot < 0 || n_rot > dr || (n_rot & 1) || (n_rot && !freq)) return FELLM_ERR_SIZE;
   const int cls = launch_class_for_rows(T, 0);
+  const bool vec = rq % 4 == 0 && rk % 4 == 0 && dr % 4 == 0 && ((q_off | c_off | ldz) % 4) == 0 && (rq + rk) / 4 <= LP_THREADS * LP_VPT &&
+                   n_rot / 2 <= LP_THREADS && (((uintptr_t)z | (uintptr_t)wq | (uintptr_t)wc | (uintptr_t)pool | (uintptr_t)cq) & 15) == 0;
+  if (vec && bf16_)
+    return launch_k_class(cls, latent_prep_vec_kernel<bf16, bf16>, dim3(T), dim3(LP_THREADS), 0, stream, 1, z, ldz, q_off, rq, c_off, rk, r_off, dr,
+                          wq, wc, eps, freq, n_rot, mag, positions, row_slot, block_table, max_pages, (bf16*)pool, page_tokens,
+                          layer, layers_in_group, (bf16*)cq, status);
+  if (vec)
+    return launch_k_class(cls, latent_prep_vec_kernel<float, float>, dim3(T), dim3(LP_THREADS), 0, stream, 1, z, ldz, q_off, rq, c_off, rk, r_off, dr,
+                          wq, wc, eps, freq, n_rot, mag, positions, row_slot, block_table, max_pages, (float*)pool, page_tokens,
+                          layer, layers_in_group, (float*)cq, status);
   if (bf16_)
     return launch_k_class(cls, latent_prep_kernel<bf16, bf16>, dim3(T), dim3(128), 0, stream, 1, z, ldz, q_off, rq, c_off, rk, r_off, dr,
                           wq, wc, eps, freq, n_rot, mag, positions, row_slot, block_table, max_pages, (bf16*)pool, page_tokens,

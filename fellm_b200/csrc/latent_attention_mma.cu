@@ -283,7 +283,7 @@ __global__ void __launch_bounds__(NG * NC * 32, 1) latent_attention_kernel(LatAr
 
 // The ranges of a split key walk put together, in the order of the ranges: out = sum_s O_s 2^(m_s - m) / (sum_s l_s
 // 2^(m_s - m) + 2^(sink - m)), m = max_s m_s.  A block per (token, head) row.
-__global__ void __launch_bounds__(128) latent_merge_kernel(const float* __restrict__ scratch, bf16* __restrict__ out,
+__global__ void __launch_bounds__(256) latent_merge_kernel(const float* __restrict__ scratch, bf16* __restrict__ out,
                                                            const float* __restrict__ sinks, int H, int n_splits) {
   __shared__ float sm_m[MAX_SPLITS], sm_w[MAX_SPLITS];
   pdl_launch_dependents();
@@ -304,11 +304,15 @@ __global__ void __launch_bounds__(128) latent_merge_kernel(const float* __restri
   __syncthreads();
   if (threadIdx.x < n_splits) sm_w[threadIdx.x] = sm_m[threadIdx.x] > -INFINITY ? exp2f(sm_m[threadIdx.x] - m) : 0.f;
   __syncthreads();
-  for (int e = threadIdx.x; e < RK; e += blockDim.x) {
-    float acc = 0.f;
-#pragma unroll 4
-    for (int s = 0; s < n_splits; ++s) acc = fmaf(base[(size_t)s * (RK + 2) + e], sm_w[s], acc);
-    out[row * RK + e] = __float2bfloat16_rn(acc * inv);
+  const int e = 2 * threadIdx.x;                   // RK / 2 threads: two neighbouring elements each, all ranges asked for at once
+  if (e < RK) {
+    float2 acc = make_float2(0.f, 0.f);
+#pragma unroll 16
+    for (int s = 0; s < n_splits; ++s) {
+      const float2 v = *(const float2*)(base + (size_t)s * (RK + 2) + e);
+      acc.x = fmaf(v.x, sm_w[s], acc.x); acc.y = fmaf(v.y, sm_w[s], acc.y);
+    }
+    *(__nv_bfloat162*)(out + row * RK + e) = __floats2bfloat162_rn(acc.x * inv, acc.y * inv);
   }
 }
 
@@ -324,7 +328,7 @@ static int launch_latent(const LatArgs& a, int n_items, int max_item_rows, int r
   const int cls = launch_class_for_rows(rows_total, 0);
   int rc = launch_k_class(cls, kern, grid, dim3(NG * NC * 32), smem, stream, 1, a);
   if (rc || a.n_splits == 1) return rc;
-  return launch_k_class(cls, latent_merge_kernel, dim3(rows_total * a.H), dim3(128), 0, stream, 1, (const float*)a.scratch, a.out,
+  return launch_k_class(cls, latent_merge_kernel, dim3(rows_total * a.H), dim3(RK / 2 < 32 ? 32 : RK / 2), 0, stream, 1, (const float*)a.scratch, a.out,
                         a.sinks, a.H, a.n_splits);
 }
 

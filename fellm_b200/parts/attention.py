@@ -136,7 +136,7 @@ class Attention(Mixer):
         if self.sink:
             self.decls["sink"] = ParamDecl((H,), role="vector", init=("normal", 1.0))
         if self.v_mix == "mix":
-            self.decls["vmix"] = ParamDecl((), role="vector", init=("uniform", 0.2, 0.8))
+            self.decls["vmix"] = ParamDecl((), role="vector", init=("uniform", 0.2, 0.8), also=((1,),))
         if self.qk_norm:
             self.decls["q_norm.weight"] = ParamDecl((hd,), role="vector", init=("ones",))
             if not self.shares_cache:
