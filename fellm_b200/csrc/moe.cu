@@ -8,7 +8,7 @@
 //                 (expert, first row, rows) that the grouped products walk
 //   moe_gemm      grouped product over the table: C[r, :] = A[row(r), :] W[e]^T, with the input rows gathered by
 //                 token (first product, SiLU(gate) * up in the epilogue) or taken in sorted order (second product)
-//   moe_combine   x[t, :] += sum_c score[t, c] * y[place(t, c), :], c in order
+//   moe_combine   x[t, :] += sum_c score[t, c] * y[place(t, c), :], c in order (an identity expert: score[t, c] * h[t, :])
 //
 // A row's arithmetic depends on the row alone: a pair's place among its expert's rows moves it inside a tile, never
 // into another sum; every sum over K runs in the order of K; the sum over a token's experts runs in the order of the
@@ -61,15 +61,24 @@ __device__ __forceinline__ void route_warp(const float* z, int E, int top, int r
   }
 }
 
-// One warp, the sigmoid form: scores s_e = sigmoid(z_e); the choice looks at s_e + corr_e (corr may be null) and only
-// inside the `keep` groups (of n_groups equal groups of neighbouring experts) whose `gtop` largest choice scores sum
+// One warp, the choice form: scores s_e = sigmoid(z_e) or, soft, softmax(z)_e over all E; the choice looks at s_e + corr_e
+// (corr may be null, and either may be negative) and only inside the `keep` groups (of n_groups equal groups of neighbouring experts) whose `gtop` largest choice scores sum
 // highest (ties: the lower group); the `top` largest choice scores among those (ties: the lower expert); weights = the
 // chosen experts' plain scores, over their sum + 1e-20 when renorm.  work: shared memory of E + n_groups floats.
-__device__ __forceinline__ void route_sigmoid_warp(const float* z, const float* corr, int E, int top, int renorm,
+__device__ __forceinline__ void route_choice_warp(int soft, const float* z, const float* corr, int E, int top, int renorm,
                                                    int n_groups, int keep, int gtop, float* work, int* idx, float* w, int lane) {
   float* choice = work;                 // [E]
   float* gscore = work + E;             // [n_groups]; -inf once a group is taken, then +inf marks the kept ones
-  for (int e = lane; e < E; e += 32) choice[e] = 1.0f / (1.0f + expf(-z[e])) + (corr ? corr[e] : 0.f);
+  float zmax = 0.f, zsum = 1.f;
+  if (soft) {
+    zmax = -INFINITY; zsum = 0.f;
+    for (int e = lane; e < E; e += 32) zmax = fmaxf(zmax, z[e]);
+    zmax = warp_max(zmax);
+    for (int e = lane; e < E; e += 32) zsum += expf(z[e] - zmax);
+    zsum = warp_sum(zsum);
+  }
+  auto score = [&](int e) { return soft ? expf(z[e] - zmax) / zsum : 1.0f / (1.0f + expf(-z[e])); };
+  for (int e = lane; e < E; e += 32) choice[e] = score(e) + (corr ? corr[e] : 0.f);
   __syncwarp();
   if (n_groups > 1 && keep < n_groups) {
     const int per = E / n_groups;
@@ -128,7 +137,7 @@ __device__ __forceinline__ void route_sigmoid_warp(const float* z, const float* 
       if (oi != 0x7fffffff && (bi == 0x7fffffff || ov > best || (ov == best && oi < bi))) { best = ov; bi = oi; }
     }
     taken[c] = bi;
-    tw[c] = 1.0f / (1.0f + expf(-z[bi]));
+    tw[c] = score(bi);
     chosen += tw[c];
   }
   if (lane == 0) {
@@ -166,9 +175,9 @@ FELLM_API int fellm_moe_route(const float* logits, int ld, int T, int E, int top
 template <typename TA, typename TW>
 __global__ void __launch_bounds__(ROUTER_WARPS * 32)
 moe_router_kernel(const TA* __restrict__ h, int ldh, const TW* __restrict__ Wr, int K, int E, int top, int renorm,
-                  int* __restrict__ idx, float* __restrict__ w, int sigmoid, const float* __restrict__ corr,
+                  int* __restrict__ idx, float* __restrict__ w, int form, const float* __restrict__ corr,
                   int n_groups, int keep, int gtop, const float* __restrict__ bias) {
-  extern __shared__ float zs[];                 // [E]; the sigmoid form: + [E + n_groups]
+  extern __shared__ float zs[];                 // [E]; the choice forms: + [E + n_groups]
   const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const TA* hr = h + (size_t)t * ldh;
   for (int e = warp; e < E; e += ROUTER_WARPS) {
@@ -180,24 +189,25 @@ moe_router_kernel(const TA* __restrict__ h, int ldh, const TW* __restrict__ Wr, 
   }
   __syncthreads();
   if (warp == 0) {
-    if (sigmoid) route_sigmoid_warp(zs, corr, E, top, renorm, n_groups, keep, gtop, zs + E, idx + (size_t)t * top, w + (size_t)t * top, lane);
+    if (form) route_choice_warp(form == 2, zs, corr, E, top, renorm, n_groups, keep, gtop, zs + E, idx + (size_t)t * top, w + (size_t)t * top, lane);
     else route_warp(zs, E, top, renorm, idx + (size_t)t * top, w + (size_t)t * top, lane);
   }
 }
 
 FELLM_API int fellm_moe_router(const void* h, int h_bf16, int ldh, const void* Wr, int w_bf16, int T, int K, int E, int top,
-                               int renorm, int* idx, float* w, int sigmoid, const float* corr, int n_groups, int keep,
+                               int renorm, int* idx, float* w, int form, const float* corr, int n_groups, int keep,
                                int gtop, const float* bias, cudaStream_t stream) {
   // bias (float32 [E] or null) is added to the logits before anything looks at them.
-  // sigmoid = 0: softmax scores over all experts.  sigmoid = 1: sigmoid scores, a correction added for the choice
-  // (corr float32 [E] or null), the choice limited to `keep` of n_groups groups ranked by their gtop best choice scores.
+  // form = 0: softmax scores over all experts, the largest chosen.  form = 1: sigmoid scores, form = 2: softmax scores over
+  // all experts, both with a correction added for the choice (corr float32 [E] or null) and the choice limited to `keep` of
+  // n_groups groups ranked by their gtop best choice scores.
   if (T <= 0) return 0;
   if (n_groups < 1) n_groups = 1;
   if (E < 1 || top < 1 || top > E || top > MOE_MAX_TOP || (size_t)(2 * E + n_groups) * sizeof(float) > 48 * 1024) return FELLM_ERR_SIZE;
-  if (sigmoid && (E % n_groups || keep < 1 || keep > n_groups || gtop < 1 || top > (E / n_groups) * keep)) return FELLM_ERR_SIZE;
+  if (form < 0 || form > 2 || (form && (E % n_groups || keep < 1 || keep > n_groups || gtop < 1 || top > (E / n_groups) * keep))) return FELLM_ERR_SIZE;
   if (!h || !Wr || !idx || !w) return FELLM_ERR_ARG;
-  const size_t sh = (size_t)(sigmoid ? 2 * E + n_groups : E) * sizeof(float);
-#define ROUTER(TA_, TW_) moe_router_kernel<TA_, TW_><<<T, ROUTER_WARPS * 32, sh, stream>>>((const TA_*)h, ldh, (const TW_*)Wr, K, E, top, renorm, idx, w, sigmoid, corr, n_groups, keep, gtop, bias)
+  const size_t sh = (size_t)(form ? 2 * E + n_groups : E) * sizeof(float);
+#define ROUTER(TA_, TW_) moe_router_kernel<TA_, TW_><<<T, ROUTER_WARPS * 32, sh, stream>>>((const TA_*)h, ldh, (const TW_*)Wr, K, E, top, renorm, idx, w, form, corr, n_groups, keep, gtop, bias)
   if (h_bf16) { if (w_bf16) ROUTER(bf16, bf16); else ROUTER(bf16, float); }
   else { if (w_bf16) ROUTER(float, bf16); else ROUTER(float, float); }
 #undef ROUTER
@@ -205,13 +215,14 @@ FELLM_API int fellm_moe_router(const void* h, int h_bf16, int ldh, const void* W
 }
 
 // ---------------------------------------------------------------- the plan
-// Pairs p = t * top + c, P of them.  Tile i of PLAN_TILE pairs: counts[i][e] and each pair's rank among the pairs of
+// Pairs p = t * top + c, P of them.  A choice beyond the E experts (an identity expert: the token's input handed on, no
+// product) is no row of the plan: its place is -1.  n_tiles[0]: row tiles, n_tiles[1]: sorted rows.  Tile i of PLAN_TILE pairs: counts[i][e] and each pair's rank among the pairs of
 // its tile that chose the same expert before it.
 __global__ void __launch_bounds__(PLAN_TILE)
 moe_count_kernel(const int* __restrict__ idx, int P, int E, int* __restrict__ counts, int* __restrict__ rank) {
   __shared__ int ex[PLAN_TILE];
   const int p = blockIdx.x * PLAN_TILE + threadIdx.x;
-  const int e = p < P ? idx[p] : -1;
+  const int e = p < P && idx[p] < E ? idx[p] : -1;
   ex[threadIdx.x] = e;
   for (int i = threadIdx.x; i < E; i += PLAN_TILE) counts[(size_t)blockIdx.x * E + i] = 0;
   __syncthreads();
@@ -241,7 +252,7 @@ moe_scan_kernel(const int* __restrict__ counts, int n_plan_tiles, int E, int BM,
   if (threadIdx.x == 0) {
     int at = 0, tiles = 0;
     for (int e = 0; e < E; ++e) { first[e] = at; first_tile[e] = tiles; at += rows[e]; tiles += (rows[e] + BM - 1) / BM; }
-    *n_tiles = tiles;
+    n_tiles[0] = tiles; n_tiles[1] = at;
   }
   __syncthreads();
   for (int e = threadIdx.x; e < E; e += blockDim.x) {
@@ -254,11 +265,12 @@ moe_scan_kernel(const int* __restrict__ counts, int n_plan_tiles, int E, int BM,
   }
 }
 
-// sorted[place] = pair, place_of[pair] = place
+// sorted[place] = pair, place_of[pair] = place (-1: an identity expert's)
 __global__ void moe_place_kernel(const int* __restrict__ idx, const int* __restrict__ rank, const int* __restrict__ base,
                                  int P, int E, int* __restrict__ sorted, int* __restrict__ place_of) {
   const int p = blockIdx.x * blockDim.x + threadIdx.x;
   if (p >= P) return;
+  if (idx[p] >= E) { place_of[p] = -1; return; }
   const int place = base[(size_t)(p / PLAN_TILE) * E + idx[p]] + rank[p];
   sorted[place] = p;
   place_of[p] = place;
@@ -272,7 +284,7 @@ moe_plan_small_kernel(const int* __restrict__ idx, int P, int E, int BM, int* __
   extern __shared__ int sh[];            // [E] rows of an expert, then [E] its first row
   int* rows = sh; int* first = sh + E;
   const int p = threadIdx.x;
-  const int e = p < P ? idx[p] : -1;
+  const int e = p < P && idx[p] < E ? idx[p] : -1;
   ex[p] = e;
   for (int i = p; i < E; i += PLAN_TILE) rows[i] = 0;
   __syncthreads();
@@ -293,9 +305,10 @@ moe_plan_small_kernel(const int* __restrict__ idx, int P, int E, int BM, int* __
       }
       at += rows[i];
     }
-    *n_tiles = tiles;
+    n_tiles[0] = tiles; n_tiles[1] = at;
   }
   __syncthreads();
+  if (p < P && e < 0) place_of[p] = -1;
   if (e >= 0) {
     const int place = first[e] + r;
     sorted[place] = p;
@@ -620,37 +633,47 @@ FELLM_API int fellm_moe_gemm(const void* A, int a_bf16, int lda, const int* gath
 // out[r, :] = a[sorted[r] / top, :]   (bfloat16, K a multiple of 8: 16 bytes a thread): the input of the tcgen05
 // grouped product, whose TMA boxes want an expert's rows side by side.
 __global__ void moe_gather_kernel(const bf16* __restrict__ a, int lda, const int* __restrict__ sorted, int top,
-                                  bf16* __restrict__ out, int K) {
+                                  bf16* __restrict__ out, int K, const int* __restrict__ n_tiles) {
   const int r = blockIdx.x;
+  if (r >= n_tiles[1]) return;
   const bf16* src = a + (size_t)(sorted[r] / top) * lda;
   bf16* dst = out + (size_t)r * K;
   for (int k = threadIdx.x * 8; k < K; k += blockDim.x * 8) *(uint4*)(dst + k) = *(const uint4*)(src + k);
 }
 
-FELLM_API int fellm_moe_gather(const void* a, int lda, const int* sorted, int top, void* out, int P, int K, cudaStream_t stream) {
+FELLM_API int fellm_moe_gather(const void* a, int lda, const int* sorted, int top, void* out, int P, int K, const int* n_tiles,
+                               cudaStream_t stream) {
   if (P <= 0) return 0;
-  if (!a || !sorted || !out) return FELLM_ERR_ARG;
+  if (!a || !sorted || !out || !n_tiles) return FELLM_ERR_ARG;
   if (K % 8 || lda % 8 || ((uintptr_t)a % 16) || ((uintptr_t)out % 16)) return FELLM_ERR_SIZE;
-  moe_gather_kernel<<<P, 128, 0, stream>>>((const bf16*)a, lda, sorted, top, (bf16*)out, K);
+  moe_gather_kernel<<<P, 128, 0, stream>>>((const bf16*)a, lda, sorted, top, (bf16*)out, K, n_tiles);
   return launch_status();
 }
 
 // ---------------------------------------------------------------- the weighted sum into the residual stream
-// x[t, :] += sum_c w[t, c] * y[place_of[t * top + c], :], c = 0 .. top-1 in order, float32 (store: x[t, :] = the sum).
+// x[t, :] += sum_c w[t, c] * r_c, c = 0 .. top-1 in order, float32 (store: x[t, :] = the sum); r_c = y[place_of[t * top +
+// c], :], or, place -1 (an identity expert), the token's input h[t, :].
+template <typename TH>
 __global__ void moe_combine_kernel(float* __restrict__ x, const float* __restrict__ y, const int* __restrict__ place_of,
-                                   const float* __restrict__ w, int top, int d, int store) {
+                                   const float* __restrict__ w, const TH* __restrict__ h, int ldh, int top, int d, int store) {
   const int t = blockIdx.x;
   for (int i = threadIdx.x; i < d; i += blockDim.x) {
     float s = 0.f;
-    for (int c = 0; c < top; ++c) s = fmaf(w[(size_t)t * top + c], y[(size_t)place_of[(size_t)t * top + c] * d + i], s);
+    for (int c = 0; c < top; ++c) {
+      const int place = place_of[(size_t)t * top + c];
+      s = fmaf(w[(size_t)t * top + c], place < 0 ? to_f(h[(size_t)t * ldh + i]) : y[(size_t)place * d + i], s);
+    }
     x[(size_t)t * d + i] = store ? s : x[(size_t)t * d + i] + s;
   }
 }
 
-FELLM_API int fellm_moe_combine(float* x, const float* y, const int* place_of, const float* w, int T, int top, int d,
-                                int store, cudaStream_t stream) {
+// h [T, ldh] (bfloat16 or float32): needed where a plan has identity experts, else null.
+FELLM_API int fellm_moe_combine(float* x, const float* y, const int* place_of, const float* w, const void* h, int h_bf16, int ldh,
+                                int T, int top, int d, int store, cudaStream_t stream) {
   if (T <= 0) return 0;
   if (!x || !y || !place_of || !w) return FELLM_ERR_ARG;
-  moe_combine_kernel<<<T, d >= 256 ? 256 : 128, 0, stream>>>(x, y, place_of, w, top, d, store);
+  const int threads = d >= 256 ? 256 : 128;
+  if (h_bf16) moe_combine_kernel<bf16><<<T, threads, 0, stream>>>(x, y, place_of, w, (const bf16*)h, ldh, top, d, store);
+  else moe_combine_kernel<float><<<T, threads, 0, stream>>>(x, y, place_of, w, (const float*)h, ldh, top, d, store);
   return launch_status();
 }

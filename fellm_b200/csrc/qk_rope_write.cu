@@ -535,3 +535,167 @@ FELLM_API int fellm_qkv_rotate_write(void* qkv, int is_bf16, int ld, int T, int 
   if (is_bf16) return launch_k_class(cls, qkv_rotate_write_kernel<bf16>, dim3(T), dim3(128), 0, stream, 1, (bf16*)qkv, (const bf16*)v0, (bf16*)pool, a);
   return launch_k_class(cls, qkv_rotate_write_kernel<float>, dim3(T), dim3(128), 0, stream, 1, (float*)qkv, (const float*)v0, (float*)pool, a);
 }
+
+// ---------------------------------------------------------------- norm over the whole projection, rotation and the cache write
+// The rows of the input product are [q (H hd) | k (G hd) | v (G vd) | ...], ld elements apart.  All of a row's q, and all
+// of its k, are divided by their root mean square (eps inside the root) and multiplied by a weight per row element (qw
+// [H hd], kw [G hd]); then every head is rotated on its first rot_dim elements (pairs (2i, 2i + 1) or (i, i + rot_dim/2)).
+// q stays where it lies; k and v go into the row's page, a page-layer record being the keys [G][page_tokens][hd], then
+// the values [G][page_tokens][vd].  G = 0: the rows hold no k and v (the layer reads another layer's pages).  A block a
+// row; the row's sines and cosines and its page's number before the wait for the product; float32 throughout, rounded
+// once; the sums' order depends on the sizes alone.
+#define NRW_THREADS 256
+
+struct NormRotateWriteArgs {
+  int ld, H, G, hd, vd, rot_dim, pairing, max_pages, page_tokens, layer, layers_in_group;
+  float eps;
+  const float* inv_freq; const float* qw; const float* kw;
+  const int* positions; const int* row_slot; const int* block_table;
+  int* status;
+};
+
+// The block's sums of two values, the same in every thread: warps in order.
+__device__ __forceinline__ void nrw_block_sums(float& x, float& y, float (*red)[NRW_THREADS / 32]) {
+  const int warp = threadIdx.x >> 5;
+  x = warp_sum(x); y = warp_sum(y);
+  if ((threadIdx.x & 31) == 0) { red[0][warp] = x; red[1][warp] = y; }
+  __syncthreads();
+  x = y = 0.f;
+#pragma unroll
+  for (int w = 0; w < NRW_THREADS / 32; ++w) { x += red[0][w]; y += red[1][w]; }
+}
+
+template <typename T>
+__global__ void __launch_bounds__(NRW_THREADS)
+qkv_norm_rotate_write_kernel(T* __restrict__ qkv, T* __restrict__ pool, NormRotateWriteArgs a) {
+  __shared__ float sn_s[RWM_HALF], cs_s[RWM_HALF], red[2][NRW_THREADS / 32];
+  pdl_launch_dependents();
+  const int row = blockIdx.x, pos = a.positions[row], half = a.rot_dim >> 1;
+  const int page = a.G ? a.block_table[(size_t)a.row_slot[row] * a.max_pages + pos / a.page_tokens] : 0;
+  for (int i = threadIdx.x; i < half; i += NRW_THREADS) sincosf((float)pos * a.inv_freq[i], &sn_s[i], &cs_s[i]);
+  pdl_wait();
+  T* p = qkv + (size_t)row * a.ld;
+  const int nq = a.H * a.hd, nk = a.G * a.hd;
+  float sq = 0.f, sk = 0.f;
+  for (int e = threadIdx.x; e < nq; e += NRW_THREADS) { const float v = to_f(p[e]); sq = fmaf(v, v, sq); }
+  for (int e = threadIdx.x; e < nk; e += NRW_THREADS) { const float v = to_f(p[nq + e]); sk = fmaf(v, v, sk); }
+  nrw_block_sums(sq, sk, red);                       // (its barrier is also the one behind the sines and cosines)
+  const float rq = 1.0f / sqrtf(sq / (float)nq + a.eps), rk = nk ? 1.0f / sqrtf(sk / (float)nk + a.eps) : 0.f;
+  if (a.G && page < 0 && threadIdx.x == 0 && a.status) atomicExch(a.status, 2);          // never write outside the pool: record and skip
+  const bool write = a.G && page >= 0;
+  const int in_page = pos % a.page_tokens;
+  T* rec = write ? pool + ((size_t)page * a.layers_in_group + a.layer) * ((size_t)a.G * a.page_tokens * (a.hd + a.vd)) : nullptr;
+  const int per = a.hd - half, heads = a.H + (write ? a.G : 0);       // a pair, or one element behind the rotated part
+  for (int u = threadIdx.x; u < heads * per; u += NRW_THREADS) {
+    const int h = u / per, i = u - h * per;
+    const bool is_q = h < a.H;
+    const T* src = p + (size_t)h * a.hd;
+    T* dst = is_q ? p + (size_t)h * a.hd : rec + ((size_t)(h - a.H) * a.page_tokens + in_page) * a.hd;
+    const float* w = is_q ? a.qw + (size_t)h * a.hd : a.kw + (size_t)(h - a.H) * a.hd;
+    const float r = is_q ? rq : rk;
+    if (i < half) {
+      const int ia = a.pairing ? i : 2 * i, ib = a.pairing ? i + half : 2 * i + 1;
+      const float x = to_f(src[ia]) * r * w[ia], y = to_f(src[ib]) * r * w[ib];
+      dst[ia] = from_f<T>(x * cs_s[i] - y * sn_s[i]); dst[ib] = from_f<T>(y * cs_s[i] + x * sn_s[i]);
+    } else {
+      dst[i + half] = from_f<T>(to_f(src[i + half]) * r * w[i + half]);
+    }
+  }
+  if (!write) return;
+  const T* vp = p + nq + nk;
+  T* vrec = rec + (size_t)a.G * a.page_tokens * a.hd;
+  for (int u = threadIdx.x; u < a.G * a.vd; u += NRW_THREADS) {
+    const int g = u / a.vd, c = u - g * a.vd;
+    vrec[((size_t)g * a.page_tokens + in_page) * a.vd + c] = vp[u];
+  }
+}
+
+// bfloat16, hd and vd multiples of 8, rot_dim of 8 (pairs of neighbours: SPLIT false) or 16, rows on 16-byte boundaries:
+// a thread eight elements by 16-byte loads and stores (and, SPLIT, the eight they are paired with).
+template <bool SPLIT>
+__global__ void __launch_bounds__(NRW_THREADS)
+qkv_norm_rotate_write_vec_kernel(bf16* __restrict__ qkv, bf16* __restrict__ pool, NormRotateWriteArgs a) {
+  __shared__ float sn_s[RWM_HALF], cs_s[RWM_HALF], red[2][NRW_THREADS / 32];
+  pdl_launch_dependents();
+  const int row = blockIdx.x, pos = a.positions[row], half = a.rot_dim >> 1;
+  const int page = a.G ? a.block_table[(size_t)a.row_slot[row] * a.max_pages + pos / a.page_tokens] : 0;
+  for (int i = threadIdx.x; i < half; i += NRW_THREADS) sincosf((float)pos * a.inv_freq[i], &sn_s[i], &cs_s[i]);
+  pdl_wait();
+  bf16* p = qkv + (size_t)row * a.ld;
+  const int nq = a.H * a.hd, nk = a.G * a.hd;
+  float sq = 0.f, sk = 0.f;
+  for (int u = threadIdx.x; u < (nq + nk) >> 3; u += NRW_THREADS) {
+    float x[8], s = 0.f;
+    rw_unpack8(*(const uint4*)(p + 8 * u), x);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) s = fmaf(x[e], x[e], s);
+    if (8 * u < nq) sq += s; else sk += s;
+  }
+  nrw_block_sums(sq, sk, red);                       // (its barrier is also the one behind the sines and cosines)
+  const float rq = 1.0f / sqrtf(sq / (float)nq + a.eps), rk = nk ? 1.0f / sqrtf(sk / (float)nk + a.eps) : 0.f;
+  if (a.G && page < 0 && threadIdx.x == 0 && a.status) atomicExch(a.status, 2);          // never write outside the pool: record and skip
+  const bool write = a.G && page >= 0;
+  const int in_page = pos % a.page_tokens;
+  bf16* rec = write ? pool + ((size_t)page * a.layers_in_group + a.layer) * ((size_t)a.G * a.page_tokens * (a.hd + a.vd)) : nullptr;
+  const int hc = SPLIT ? half >> 3 : 0, per = (a.hd >> 3) - hc, vc = a.vd >> 3;
+  const int n_heads = a.H * per + (write ? a.G * per : 0), n_units = n_heads + (write ? a.G * vc : 0);
+  for (int u = threadIdx.x; u < n_units; u += NRW_THREADS) {
+    if (u < n_heads) {
+      const int h = u / per, c = u - h * per;
+      const bool is_q = h < a.H;
+      const bf16* src = p + (size_t)h * a.hd;
+      bf16* dst = is_q ? p + (size_t)h * a.hd : rec + ((size_t)(h - a.H) * a.page_tokens + in_page) * a.hd;
+      const float* w = is_q ? a.qw + (size_t)h * a.hd : a.kw + (size_t)(h - a.H) * a.hd;
+      const float r = is_q ? rq : rk;
+      const int at = (SPLIT && c >= hc) ? 8 * c + half : 8 * c;        // behind the rotated part, SPLIT skips its second half
+      float x[8];
+      rw_unpack8(*(const uint4*)(src + at), x);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) x[e] = x[e] * r * w[at + e];
+      if (SPLIT && c < hc) {
+        float y[8];
+        rw_unpack8(*(const uint4*)(src + half + at), y);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) {
+          const float sn = sn_s[at + e], cs = cs_s[at + e], xe = x[e], ye = y[e] * r * w[half + at + e];
+          x[e] = xe * cs - ye * sn; y[e] = ye * cs + xe * sn;
+        }
+        *(uint4*)(dst + half + at) = rw_pack8(y);
+      } else if (!SPLIT && at < a.rot_dim) {
+#pragma unroll
+        for (int e = 0; e < 8; e += 2) {
+          const float sn = sn_s[(at + e) >> 1], cs = cs_s[(at + e) >> 1], xe = x[e], ye = x[e + 1];
+          x[e] = xe * cs - ye * sn; x[e + 1] = ye * cs + xe * sn;
+        }
+      }
+      *(uint4*)(dst + at) = rw_pack8(x);
+    } else {
+      const int w = u - n_heads, g = w / vc, c = w - g * vc;
+      *(uint4*)(rec + (size_t)a.G * a.page_tokens * a.hd + ((size_t)g * a.page_tokens + in_page) * a.vd + 8 * c) =
+          *(const uint4*)(p + nq + nk + 8 * w);
+    }
+  }
+}
+
+FELLM_API int fellm_qkv_norm_rotate_write(void* qkv, int is_bf16, int ld, int T, int H, int G, int hd, int vd, const float* qw,
+                                          const float* kw, float eps, int rot_dim, const float* inv_freq, int pairing,
+                                          const int* positions, const int* row_slot, const int* block_table, int max_pages,
+                                          void* pool, int cache_bf16, int page_tokens, int layer, int layers_in_group, int* status,
+                                          cudaStream_t stream) {
+  if (T <= 0) return 0;
+  if (!inv_freq) rot_dim = 0;
+  if (H < 1 || G < 0 || hd < 1 || vd < 1 || rot_dim < 0 || rot_dim > hd || (rot_dim & 1) || rot_dim > 2 * RWM_HALF || page_tokens < 1) return FELLM_ERR_SIZE;
+  if (ld < H * hd + G * (hd + vd)) return FELLM_ERR_SIZE;
+  if (!qkv || !positions || !qw || (G && (!kw || !row_slot || !block_table || !pool || is_bf16 != cache_bf16))) return FELLM_ERR_ARG;
+  NormRotateWriteArgs a;
+  a.ld = ld; a.H = H; a.G = G; a.hd = hd; a.vd = vd; a.rot_dim = rot_dim; a.pairing = pairing; a.max_pages = max_pages;
+  a.page_tokens = page_tokens; a.layer = layer; a.layers_in_group = layers_in_group; a.eps = eps; a.inv_freq = inv_freq;
+  a.qw = qw; a.kw = kw; a.positions = positions; a.row_slot = row_slot; a.block_table = block_table; a.status = status;
+  const int cls = launch_class_for_rows(T, 2);
+  const bool vec = is_bf16 && hd % 8 == 0 && vd % 8 == 0 && rot_dim % (pairing ? 16 : 8) == 0 && ld % 8 == 0 &&
+                   (((uintptr_t)qkv | (uintptr_t)pool) & 15) == 0;
+  if (vec && pairing) return launch_k_class(cls, qkv_norm_rotate_write_vec_kernel<true>, dim3(T), dim3(NRW_THREADS), 0, stream, 1, (bf16*)qkv, (bf16*)pool, a);
+  if (vec) return launch_k_class(cls, qkv_norm_rotate_write_vec_kernel<false>, dim3(T), dim3(NRW_THREADS), 0, stream, 1, (bf16*)qkv, (bf16*)pool, a);
+  if (is_bf16) return launch_k_class(cls, qkv_norm_rotate_write_kernel<bf16>, dim3(T), dim3(NRW_THREADS), 0, stream, 1, (bf16*)qkv, (bf16*)pool, a);
+  return launch_k_class(cls, qkv_norm_rotate_write_kernel<float>, dim3(T), dim3(NRW_THREADS), 0, stream, 1, (float*)qkv, (float*)pool, a);
+}

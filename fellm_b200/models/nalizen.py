@@ -64,7 +64,7 @@ def _feed_forward(p: str, d: int, f) -> PartSpec:
                          router_bias=True, plain="relu2")
 
 
-def _kept_windows(cfg: NalizenConfig):
+def kept_windows(cfg):
     """Per attention layer that keeps pages: the window they are kept for, the widest among the layer itself and the
     layers that read its pages (None: no window, nothing is given back before the request ends)."""
     kept = {}
@@ -82,7 +82,7 @@ def _kept_windows(cfg: NalizenConfig):
 
 def build_spec(cfg: NalizenConfig) -> ModelSpec:
     d, eps = cfg.width, cfg.norm_eps
-    kept = _kept_windows(cfg)
+    kept = kept_windows(cfg)
     layers, schedule = [], []
     for i, L in enumerate(cfg.layers):
         p = f"l{i}."

@@ -874,10 +874,10 @@ def moe_route(logits, E: int, top: int, renormalize: bool = False):
 def moe_router(h, w_router, top: int, renormalize: bool = False, *, score: str = "softmax", correction=None,
                groups=None, bias=None):
     """The router's product and the routing in one launch: z = h W_router^T in float32 (h [T, K] and W_router [E, K]
-    bfloat16 or float32), then as moe_route.  score = "sigmoid": the scores are sigmoid(z); the choice looks at
-    score + correction (float32 [E]) and, with groups = (count, keep, best), only inside the `keep` of `count` equal
+    bfloat16 or float32), then as moe_route.  score = "sigmoid": the scores are sigmoid(z), else softmax(z) over all E.  The
+    choice looks at score + correction (float32 [E]) and, with groups = (count, keep, best), only inside the `keep` of `count` equal
     groups of neighbouring experts whose `best` largest choice scores sum highest; the weights are the plain scores
-    (renormalize: over their sum + 1e-20).  bias float32 [E]: added to z first.  Softmax scores renormalised over the
+    (renormalize: over their sum, + 1e-20 in the form with a choice of its own).  bias float32 [E]: added to z first.  Softmax scores renormalised over the
     chosen are the softmax over the chosen logits alone.  Returns (idx int32 [T, top], w float32 [T, top])."""
     _dev(h, w_router, correction, bias)
     if bias is not None:
@@ -889,8 +889,7 @@ def moe_router(h, w_router, top: int, renormalize: bool = False, *, score: str =
         raise KernelError(f"moe_router: top {top} must be in 1..{min(E, MOE_MAX_TOP)}")
     if score not in ("softmax", "sigmoid"):
         raise KernelError(f"moe_router: unknown score {score!r}")
-    if score == "softmax" and (correction is not None or groups):
-        raise KernelError("moe_router: a correction and groups go with sigmoid scores")
+    form = 1 if score == "sigmoid" else (2 if correction is not None or groups else 0)
     n_groups, keep, best = groups if groups else (1, 1, 1)
     if correction is not None:
         assert correction.dtype == torch.float32 and correction.numel() == E and correction.is_contiguous()
@@ -899,7 +898,7 @@ def moe_router(h, w_router, top: int, renormalize: bool = False, *, score: str =
     f = _fn("moe", "fellm_moe_router", [_c_p, _c_int, _c_int, _c_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_p, _c_p,
                                         _c_int, _c_p, _c_int, _c_int, _c_int, _c_p, _c_p])
     _check(f(_p(h), _is_bf16(h), h.stride(0), _p(w_router), _is_bf16(w_router), T, K, E, top, int(renormalize), _p(idx),
-             _p(w), int(score == "sigmoid"), _p(correction), int(n_groups), int(keep), int(best), _p(bias), _stream()),
+             _p(w), form, _p(correction), int(n_groups), int(keep), int(best), _p(bias), _stream()),
            "moe_router")
     return idx, w
 
@@ -907,8 +906,9 @@ def moe_router(h, w_router, top: int, renormalize: bool = False, *, score: str =
 class MoePlan:
     """The (token, choice) pairs of a step sorted by expert: sorted[place] = pair, place_of[pair] = place, and the
     table of row tiles (expert, first row, rows <= row_tile) with their count on the device; max_tiles bounds it on
-    the host."""
-    __slots__ = ("sorted", "place_of", "table", "n_tiles", "max_tiles", "pairs", "top", "row_tile")
+    the host.  Choices beyond the E experts of moe_plan (identity experts) are no rows of it: place_of is -1, and
+    n_rows, on the device too, counts the rows that are."""
+    __slots__ = ("sorted", "place_of", "table", "n_tiles", "n_rows", "max_tiles", "pairs", "top", "row_tile")
 
 
 def moe_row_tile(pairs: int, bf16: bool, K_ok: bool) -> int:
@@ -926,12 +926,12 @@ def moe_plan(idx, E: int, row_tile: int = MOE_ROW_TILE) -> MoePlan:
     plan = MoePlan()
     plan.pairs, plan.top, plan.row_tile = P, top, row_tile
     plan.max_tiles = min(P, E) + P // row_tile
-    ints = torch.empty(2 * tiles * E + P + 2 * P + 3 * plan.max_tiles + 1, dtype=torch.int32, device=idx.device)
+    ints = torch.empty(2 * tiles * E + P + 2 * P + 3 * plan.max_tiles + 2, dtype=torch.int32, device=idx.device)
     at = 2 * tiles * E + P
     scratch = ints[:at]
     plan.sorted, plan.place_of = ints[at:at + P], ints[at + P:at + 2 * P]
     plan.table = ints[at + 2 * P:at + 2 * P + 3 * plan.max_tiles]
-    plan.n_tiles = ints[at + 2 * P + 3 * plan.max_tiles:]
+    plan.n_tiles, plan.n_rows = ints[-2:-1], ints[-1:]            # (side by side: the kernels take one pointer)
     f = _fn("moe", "fellm_moe_plan", [_c_p, _c_int, _c_int, _c_int, _c_p, _c_p, _c_p, _c_p, _c_p, _c_p])
     _check(f(_p(idx), P, E, row_tile, _p(scratch), _p(plan.sorted), _p(plan.place_of), _p(plan.table),
              _p(plan.n_tiles), _stream()), "moe_plan")
@@ -961,8 +961,8 @@ def moe_gemm(a, w, plan: MoePlan, *, gated: bool, gather: bool, interleaved: boo
             and w.data_ptr() % 16 == 0):
         if gather:
             rows = torch.empty((P, K), dtype=a.dtype, device=a.device)
-            f = _fn("moe", "fellm_moe_gather", [_c_p, _c_int, _c_p, _c_int, _c_p, _c_int, _c_int, _c_p])
-            _check(f(_p(a), a.stride(0), _p(plan.sorted), plan.top, _p(rows), P, K, _stream()), "moe_gather")
+            f = _fn("moe", "fellm_moe_gather", [_c_p, _c_int, _c_p, _c_int, _c_p, _c_int, _c_int, _c_p, _c_p])
+            _check(f(_p(a), a.stride(0), _p(plan.sorted), plan.top, _p(rows), P, K, _p(plan.n_tiles), _stream()), "moe_gather")
             a = rows
         assert a.stride(0) % 8 == 0 and a.data_ptr() % 16 == 0
         f = _fn("gemm_umma", "fellm_gemm_umma_grouped", [_c_p, _c_p, _c_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int,
@@ -981,15 +981,19 @@ def moe_gemm(a, w, plan: MoePlan, *, gated: bool, gather: bool, interleaved: boo
     return out
 
 
-def moe_combine(x, y, plan: MoePlan, w, store: bool = False):
-    """x float32 [T, d] += sum over a token's choices c, in order, of w[t, c] * y[place of (t, c)] (store: x = the sum)."""
-    _dev(x, y, w)
+def moe_combine(x, y, plan: MoePlan, w, store: bool = False, identity=None):
+    """x float32 [T, d] += sum over a token's choices c, in order, of w[t, c] * y[place of (t, c)] (store: x = the sum).
+    identity [T, d] (bfloat16 or float32): the rows a choice that is no row of the plan stands for."""
+    _dev(x, y, w, identity)
+    if identity is not None:
+        assert identity.shape == x.shape and identity.stride(1) == 1
     T, d = x.shape
     assert x.dtype == torch.float32 and y.dtype == torch.float32 and w.dtype == torch.float32
     assert x.is_contiguous() and y.is_contiguous() and w.is_contiguous() and y.shape == (plan.pairs, d)
     residual_written(x)
-    f = _fn("moe", "fellm_moe_combine", [_c_p, _c_p, _c_p, _c_p, _c_int, _c_int, _c_int, _c_int, _c_p])
-    _check(f(_p(x), _p(y), _p(plan.place_of), _p(w), T, plan.top, d, int(store), _stream()), "moe_combine")
+    f = _fn("moe", "fellm_moe_combine", [_c_p, _c_p, _c_p, _c_p, _c_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_p])
+    _check(f(_p(x), _p(y), _p(plan.place_of), _p(w), _p(identity), int(identity is not None and _is_bf16(identity)),
+             identity.stride(0) if identity is not None else 0, T, plan.top, d, int(store), _stream()), "moe_combine")
     return x
 
 
@@ -1082,6 +1086,35 @@ def qkv_rotate_write(qkv, H, G, hd, vd, rot_dim, inv_freq, pairing, mag, positio
              _p(v_first), v_first.stride(0) if v_first is not None else 0, _p(lam), _p(positions), _p(row_slot), _p(bt),
              bt.shape[1], _p(pool), _is_bf16(pool), cache.page_tokens, cache.layer, pool.shape[1], _p(status), _stream()),
            "qkv_rotate_write")
+
+
+def qkv_norm_rotate_write(qkv, H, G, hd, vd, q_w, k_w, eps, rot_dim, inv_freq, pairing, positions, row_slot, cache, *, status=None):
+    """The rows of a layer's input product, [q (H hd) | k (G hd) | v (G vd) | ...]: all of a row's q, and all of its k, over
+    their root mean square (eps inside the root) times a weight per element (q_w float32 [H hd], k_w [G hd]), then every head
+    rotated on its first rot_dim elements (inv_freq None: no rotation); q stays where it lies, k and v go into the rows'
+    pages.  G = 0: the rows hold no k and v and nothing is written (k_w and cache may be None)."""
+    pool, bt = (cache.pool, cache.block_table) if G else (None, None)
+    _dev(qkv, inv_freq, positions, row_slot, pool, bt, q_w, k_w)
+    T = qkv.shape[0]
+    assert qkv.stride(1) == 1 and qkv.shape[1] >= H * hd + G * (hd + vd)
+    assert q_w.dtype == torch.float32 and q_w.numel() == H * hd and q_w.is_contiguous()
+    if G:
+        assert k_w.dtype == torch.float32 and k_w.numel() == G * hd and k_w.is_contiguous()
+        assert pool.is_contiguous() and pool.dtype == qkv.dtype and pool[0, 0].numel() == G * cache.page_tokens * (hd + vd)
+        _i32(bt, "block_table"), _i32(row_slot, "row_slot")
+    rot_dim = 0 if inv_freq is None else int(rot_dim)
+    if rot_dim % 2 or not 0 <= rot_dim <= min(hd, 512):
+        raise KernelError(f"qkv_norm_rotate_write: rotated part {rot_dim} must be even, within the head ({hd}) and at most 512")
+    if inv_freq is not None:
+        assert inv_freq.dtype == torch.float32 and inv_freq.numel() == rot_dim // 2 and inv_freq.is_contiguous()
+    _i32(positions, "positions")
+    f = _fn("qk_rope_write", "fellm_qkv_norm_rotate_write",
+            [_c_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_p, _c_p, _c_f, _c_int, _c_p, _c_int, _c_p, _c_p, _c_p,
+             _c_int, _c_p, _c_int, _c_int, _c_int, _c_int, _c_p, _c_p])
+    _check(f(_p(qkv), _is_bf16(qkv), qkv.stride(0), T, H, G, hd, vd, _p(q_w), _p(k_w), float(eps), rot_dim, _p(inv_freq),
+             PAIRINGS[pairing], _p(positions), _p(row_slot), _p(bt), bt.shape[1] if G else 0, _p(pool), _is_bf16(qkv),
+             cache.page_tokens if G else 1, cache.layer if G else 0, pool.shape[1] if G else 1, _p(status), _stream()),
+           "qkv_norm_rotate_write")
 
 
 def paged_attention_simt(q, pool, block_table, positions, row_slot, layer, scale, window=None, out=None):
@@ -2042,15 +2075,17 @@ def _mma_takes(H: int, G: int, hd: int, vd: int) -> bool:
             and H // G <= 64)
 
 
-def attention_written(qkv, H, G, hd, vd, cache, ctx, scale, *, window=None, sinks=None, warps=8, out=None):
+def attention_written(qkv, H, G, hd, vd, cache, ctx, scale, *, window=None, softcap=None, sinks=None, gate=None, warps=8, out=None):
     """Attention of a step's rows over pages that already hold the rows' own keys and values (qkv_rotate_write): query head
     h of row t is qkv[t, h hd : (h + 1) hd] as it lies; keys of hd, values of vd; sinks float32 [H]: exp(sinks[h]) joins
-    head h's softmax denominator.  bfloat16 on tensor cores (portions: tcgen05 where the sizes allow, else mma.sync; single
+    head h's softmax denominator; softcap: scores c tanh(s / c); gate [T, H * vd] (qkv's dtype, rows of any stride): the result
+    times sigmoid(gate), element by element.  bfloat16 on tensor cores (portions: tcgen05 where the sizes allow, else mma.sync; single
     tokens: the key walk split over CTAs), everything else on CUDA cores.  Returns [T, H * vd] in qkv's dtype."""
     pool, bt, positions, row_slot = cache.pool, cache.block_table, ctx.positions, ctx.row_slot
     if qkv.dtype != torch.bfloat16 or not _mma_takes(H, G, hd, vd) or qkv.stride(0) % 8 or qkv.data_ptr() % 16 or pool.data_ptr() % 16:
-        return paged_attention_general(qkv, H, hd, vd, pool, bt, positions, row_slot, cache.layer, cache.page_tokens, G, scale,
-                                       window=window, warps=warps, sinks=sinks, out=out)
+        out = paged_attention_general(qkv, H, hd, vd, pool, bt, positions, row_slot, cache.layer, cache.page_tokens, G, scale,
+                                      window=window, softcap=softcap, warps=warps, sinks=sinks, out=out)
+        return out if gate is None else gate_mul(out, gate)
     _dev(qkv, pool, bt, positions, row_slot, sinks)
     T, pt = qkv.shape[0], cache.page_tokens
     if H % G:
@@ -2062,6 +2097,10 @@ def attention_written(qkv, H, G, hd, vd, cache, ctx, scale, *, window=None, sink
     _i32(bt, "block_table"), _i32(positions, "positions"), _i32(row_slot, "row_slot")
     if out is None:
         out = torch.empty((T, H * vd), dtype=torch.bfloat16, device=qkv.device)
+    if ctx.all_single and softcap:
+        paged_attention_general(qkv, H, hd, vd, pool, bt, positions, row_slot, cache.layer, pt, G, scale, window=window,
+                                softcap=softcap, warps=warps, sinks=sinks, out=out)
+        return out if gate is None else gate_mul(out, gate)
     if ctx.all_single:
         split_len, max_splits = decode_split(ctx.max_len, T, G)
         scratch, counters = reserve_decode_scratch(pool.device, T, H, G, vd, max_splits)
@@ -2073,12 +2112,12 @@ def attention_written(qkv, H, G, hd, vd, cache, ctx, scale, *, window=None, sink
                  max_splits, _p(sinks), _stream()), "attention_decode")
         return out
     _i32(ctx.item_start, "item_start")
-    if umma_prefill_takes(H, G, hd, vd, pt, window, scale):
+    if umma_prefill_takes(H, G, hd, vd, pt, window, scale) and not softcap and gate is None:
         return _prefill_umma(qkv, qkv.stride(0), H, G, hd, vd, pool, bt, positions, row_slot, ctx.item_start, ctx.n_items,
                              ctx.max_item_rows, cache.layer, pt, scale, sinks, out)
     _prefill_biased(qkv, pool, bt, positions, row_slot, ctx.item_start, ctx.n_items, ctx.max_item_rows, out, T, H, G, hd, vd, pt,
-                    cache.layer, scale, window, sinks=sinks, wide=True)
-    return out
+                    cache.layer, scale, window, softcap=softcap, sinks=sinks, wide=True)
+    return out if gate is None else gate_mul(out, gate)
 
 
 def _prefill_biased(qkv, pool, block_table, positions, row_slot, item_start, n_items, max_item_rows, out, T, H, G, hd, vd,

@@ -26,7 +26,12 @@ number: 'first' is the layer whose values the others, 'mix', mix with; the mixed
 either of them, or with a rotation whose cos and sin carry a magnitude, one kernel behind the input product rotates q
 where it lies and writes the rotated k and the (mixed) v into the pages (ops.qkv_rotate_write), and attention reads the
 pages: on tensor cores in the bfloat16 engine, keys and values of different sizes included (ops.attention_written).  In a
-decode step of the bfloat16 engine the attention kernel does both (ops.attention_decode_wide)."""
+decode step of the bfloat16 engine the attention kernel does both (ops.attention_decode_wide).
+
+qk_norm='whole': the norm of q and k runs over a row's whole projection, all heads at once (weights [heads * head_dim]), in
+front of the rotation, in that same kernel (ops.qkv_norm_rotate_write).  A `sink` that is a number is every head's fixed
+score (0.0: one more in the denominator), no tensor.  With either, a soft cap, a window, an output gate and a layer that reads
+another layer's pages (its own queries rotated and normed, nothing written) go along."""
 from __future__ import annotations
 
 import math
@@ -41,12 +46,13 @@ from .linear import linear, linear_modules
 
 @register_part("mixer", "attention")
 class Attention(Mixer):
-    def __init__(self, *, dtype: str, size: int, heads: int, kv_heads: int, head_dim: int, qk_norm: bool,
+    def __init__(self, *, dtype: str, size: int, heads: int, kv_heads: int, head_dim: int, qk_norm,
                  norm_eps: float, position, window=None, shares_cache: bool = False, scale=None, softcap=None,
                  v_dim=None, chunk=None, head_gate: bool = False, bias: bool = False, values_are_keys: bool = False,
                  slope_exp=None, q_temp=None, unit_qk_norm: bool = False, out_gate: bool = False, cache_window="same",
-                 sink: bool = False, v_mix=None):
-        """`position`: a PartSpec of the 'position' category.  `shares_cache`: this layer keeps no
+                 sink=False, v_mix=None):
+        """`position`: a PartSpec of the 'position' category.  `qk_norm`: False, True (per head) or 'whole'.  `sink`: False,
+        True (learned, a score per head) or a number (every head's score).  `shares_cache`: this layer keeps no
         keys and values (it has no k/v weights) and reads those of the run its schedule entry
         names."""
         super().__init__()
@@ -55,16 +61,20 @@ class Attention(Mixer):
             raise ConfigError(f"attention: {self.H} heads are not a multiple of {self.G} kv heads")
         self.unit_qk_norm, self.out_gate = bool(unit_qk_norm), bool(out_gate)
         self.in_place = self.unit_qk_norm or self.out_gate        # rotation and norm where the product left q and k
-        self.sink, self.v_mix = bool(sink), v_mix
+        self.sink_score = float(sink) if not isinstance(sink, bool) and sink is not None else None
+        self.sink, self.v_mix = bool(sink) or self.sink_score is not None, v_mix
+        self.whole_norm = qk_norm == "whole"
+        if not self.whole_norm and not isinstance(qk_norm, bool):
+            raise ConfigError(f"attention: qk_norm is {qk_norm!r} (False, True or 'whole')")
         if self.v_mix not in (None, "first", "mix"):
             raise ConfigError(f"attention: v_mix is {v_mix!r} (None, 'first' or 'mix')")
-        general = bool(sink or v_mix or softcap or chunk or head_gate or (v_dim is not None and int(v_dim) != self.hd) or bias
+        general = bool(self.sink or self.whole_norm or v_mix or softcap or chunk or head_gate or (v_dim is not None and int(v_dim) != self.hd) or bias
                        or values_are_keys or slope_exp or q_temp or self.in_place)
-        if general and not 1 <= self.hd <= (ops.ATTENTION_SIMT_MAX_HD if sink or v_mix else 256):
-            raise ConfigError(f"attention: head_dim {self.hd} must be in 1..256 (1..1024 with a sink or value mixing)")
+        if general and not 1 <= self.hd <= (ops.ATTENTION_SIMT_MAX_HD if self.sink or self.whole_norm or v_mix else 256):
+            raise ConfigError(f"attention: head_dim {self.hd} must be in 1..256 (1..1024 with a sink, value mixing or a norm over the whole projection)")
         if not general and (self.hd % 16 or not 16 <= self.hd <= 256):       # the tensor-core kernels' sizes
             raise ConfigError(f"attention: head_dim {self.hd} must be a multiple of 16 in 16..256")
-        self.qk_norm, self.eps = bool(qk_norm), float(norm_eps)
+        self.qk_norm, self.eps = bool(qk_norm) and not self.whole_norm, float(norm_eps)
         self.window = None if window is None else int(window)
         self.cache_window = self.window if cache_window == "same" else (None if cache_window is None else int(cache_window))
         if self.cache_window is not None and (self.window is None or self.cache_window < self.window):
@@ -100,13 +110,18 @@ class Attention(Mixer):
         span = min(x for x in (self.window, None if chunk is None else int(chunk), 1 << 30) if x)
         self.simt_warps = max(1, min(8, -(-span // 128)))
         # rotation, value mixing and the cache write in one kernel, attention over the pages behind it
-        self.written = self.sink or self.v_mix is not None or (
+        self.written = self.sink or self.whole_norm or self.v_mix is not None or (
             self.position.inv_freq is not None and float(getattr(self.position, "magnitude", 1.0)) != 1.0)
         if self.written:
-            if self.qk_norm or self.in_place or self.shares_cache or softcap or chunk or head_gate or values_are_keys or slope_exp or q_temp or bias:
-                raise ConfigError("attention: a sink, value mixing or a rotation with a magnitude goes with a cache of the layer's own "
-                                  "and no QK norm, output gate, soft cap, chunk, head gate, bias, distance slopes, query "
-                                  "temperature or values that are keys")
+            if (self.qk_norm or self.unit_qk_norm or chunk or head_gate or values_are_keys or slope_exp or q_temp or bias
+                    or (self.whole_norm and (self.v_mix is not None or float(getattr(self.position, "magnitude", 1.0)) != 1.0))
+                    or (not self.whole_norm and (self.shares_cache or softcap or out_gate))):
+                raise ConfigError("attention: a sink, value mixing, a rotation with a magnitude or a norm over the whole projection goes "
+                                  "with no per-head or unit norm, chunk, head gate, bias, distance slopes, query temperature or values "
+                                  "that are keys; a soft cap, an output gate or another layer's cache then go with a norm over the "
+                                  "whole projection alone, and that norm with no value mixing and no magnitude")
+            if self.rot_dim > 512 and self.position.inv_freq is not None:
+                raise ConfigError(f"attention: rotary dimension {self.rot_dim} is above 512")
             self.general = True
         elif self.general:
             if self.qk_norm or ((self.position.inv_freq is not None or self.shares_cache) and not self.in_place):
@@ -133,14 +148,15 @@ class Attention(Mixer):
             self.decls["gate.weight"] = ParamDecl((H, d), init=("normal", 0.1))
         if self.out_gate:
             self.decls["out_gate.weight"] = ParamDecl((H * self.vd, d), init=("normal", 0.05))
-        if self.sink:
+        if self.sink and self.sink_score is None:
             self.decls["sink"] = ParamDecl((H,), role="vector", init=("normal", 1.0))
         if self.v_mix == "mix":
             self.decls["vmix"] = ParamDecl((), role="vector", init=("uniform", 0.2, 0.8), also=((1,),))
-        if self.qk_norm:
-            self.decls["q_norm.weight"] = ParamDecl((hd,), role="vector", init=("ones",))
+        if self.qk_norm or self.whole_norm:
+            init = ("uniform", 0.5, 1.5) if self.whole_norm else ("ones",)
+            self.decls["q_norm.weight"] = ParamDecl((H * hd if self.whole_norm else hd,), role="vector", init=init)
             if not self.shares_cache:
-                self.decls["k_norm.weight"] = ParamDecl((hd,), role="vector", init=("ones",))
+                self.decls["k_norm.weight"] = ParamDecl((G * hd if self.whole_norm else hd,), role="vector", init=init)
 
     takes_lazy_norm = True
 
@@ -183,6 +199,8 @@ class Attention(Mixer):
             if self.head_gate:
                 self.w["gate.weight"] = _pad_rows(self.w["gate.weight"])
         self.position.to(q.device)
+        if self.sink_score is not None:
+            self.w["sink"] = torch.full((self.H,), self.sink_score, dtype=torch.float32, device=q.device)
 
     def reserve(self, device, max_rows, n_ctx):
         if self.w["qkv.weight"].dtype == torch.bfloat16 and not self.general:
@@ -268,17 +286,22 @@ class Attention(Mixer):
         elif self.v_mix == "mix":
             v_first = ctx.carried["v_first"]
         mag = getattr(self.position, "magnitude", 1.0)
-        if ctx.all_single and ops.decode_wide_takes(qkv, H, G, hd, vd, cache.page_tokens, cache.pool):
+        gate = qkv[:, self.gate_off:self.gate_off + H * vd] if self.out_gate else None
+        kw = dict(window=self.window, sinks=self.w.get("sink"))
+        if ctx.all_single and not self.whole_norm and ops.decode_wide_takes(qkv, H, G, hd, vd, cache.page_tokens, cache.pool):
             # a decode step: rotation, mixing and the cache write happen inside the attention kernel
             a = ops.attention_decode_wide(qkv, H, G, hd, vd, cache, ctx, self.scale, rot_dim=self.rot_dim, inv_freq=self.position.inv_freq,
-                                          pairing=self.position.pairing, mag=mag, v_first=v_first, lam=self.w.get("vmix"),
-                                          window=self.window, sinks=self.w.get("sink"))
+                                          pairing=self.position.pairing, mag=mag, v_first=v_first, lam=self.w.get("vmix"), **kw)
             linear(a, self.w["out_proj.weight"], out=out, accumulate=not store)
             return out
-        ops.qkv_rotate_write(qkv, H, G, hd, vd, self.rot_dim, self.position.inv_freq, self.position.pairing, mag, ctx.positions,
-                             ctx.row_slot, cache, v_first=v_first, lam=self.w.get("vmix"), status=ctx.status)
-        a = ops.attention_written(qkv, H, G, hd, vd, cache, ctx, self.scale, window=self.window, sinks=self.w.get("sink"),
-                                  warps=self.simt_warps)
+        if self.whole_norm:
+            ops.qkv_norm_rotate_write(qkv, H, 0 if self.shares_cache else G, hd, vd, self.w["q_norm.weight"], self.w.get("k_norm.weight"),
+                                      self.eps, self.rot_dim, self.position.inv_freq, self.position.pairing, ctx.positions, ctx.row_slot,
+                                      cache, status=ctx.status)
+        else:
+            ops.qkv_rotate_write(qkv, H, G, hd, vd, self.rot_dim, self.position.inv_freq, self.position.pairing, mag, ctx.positions,
+                                 ctx.row_slot, cache, v_first=v_first, lam=self.w.get("vmix"), status=ctx.status)
+        a = ops.attention_written(qkv, H, G, hd, vd, cache, ctx, self.scale, softcap=self.softcap, gate=gate, warps=self.simt_warps, **kw)
         linear(a, self.w["out_proj.weight"], out=out, accumulate=not store)
         return out
 
@@ -318,8 +341,8 @@ class Attention(Mixer):
 
     def kernel_modules(self, dtype):
         if self.written:
-            return linear_modules(dtype) + [("qk_rope_write", None)] + ops.written_attention_modules(
-                dtype, self.H, self.G, self.hd, self.vd, 64, self.window, self.scale)
+            return linear_modules(dtype) + [("qk_rope_write", None)] + ([("sublayer", None)] if self.out_gate else []) + \
+                ops.written_attention_modules(dtype, self.H, self.G, self.hd, self.vd, 64, self.window, self.scale)
         if self.general:
             mma = dtype == "bfloat16" and self.vd == self.hd and self.hd % 16 == 0 and self.H // self.G <= 64
             extra = ([("qk_rope_write", None)] if self.in_place else []) + ([("sublayer", None)] if self.out_gate else [])

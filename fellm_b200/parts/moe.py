@@ -5,8 +5,8 @@
     weights = their scores as they are (renormalize=True: divided by their sum)
     out = sum over the chosen experts, in the order of their scores, of weight * W_down (SiLU(W_gate h) * (W_up h))
 
-With score="sigmoid" the scores are s = sigmoid(z); the choice is made on s + correction (a tensor of the layer), and
-with groups=(count, keep, best) only inside the `keep` of `count` equal groups of neighbouring experts whose `best`
+With score="sigmoid" the scores are s = sigmoid(z).  With correction=True the choice is made on s + correction (a tensor
+of the layer), and with groups=(count, keep, best) only inside the `keep` of `count` equal groups of neighbouring experts whose `best`
 largest choice scores sum highest; the weights stay the plain s (renormalize: over their sum).  With
 act=("clamped", limit, alpha) an expert computes min(g, limit) sigmoid(alpha min(g, limit)) (clamp(u, -limit, limit) + 1)
 in place of SiLU(g) u.
@@ -14,6 +14,10 @@ in place of SiLU(g) u.
 With router_bias=True the logits are z = W_router h + b (b a tensor of the layer).  With renormalize=True the softmax
 scores over their sum ARE the softmax over the chosen logits alone.  With plain="relu2" an expert has no gate:
 W_down relu(W_up h)^2 (the first grouped product leaves float32 rows, ops.relu2 squares them into the activation dtype).
+
+With identity=n the router has n outputs more, behind the experts': identity experts, whose output is the input h itself
+and which have no tensors.  Scores, choice and groups are over both kinds; a token's identity experts are no rows of the
+grouped products, the weighted sum reads h for them.
 
 Experts have no biases.  Nothing goes through the host: the router's choices are sorted by expert on the device
 (ops.moe_plan; the router's product and the routing are one launch, ops.moe_router) and two grouped products walk
@@ -35,23 +39,22 @@ from .linear import linear_modules
 class RoutedExperts(FeedForward):
     def __init__(self, *, dtype: str, size: int, ff: int, experts: int, top: int, renormalize: bool = False,
                  score: str = "softmax", correction: bool = False, groups=None, act=None, router_bias: bool = False,
-                 plain=None):
+                 plain=None, identity: int = 0):
         super().__init__()
         self.size, self.ff, self.E, self.top = int(size), int(ff), int(experts), int(top)
-        self.renormalize = bool(renormalize)
-        if not 1 <= self.top <= min(self.E, ops.MOE_MAX_TOP):
-            raise ConfigError(f"moe: top {self.top} must be in 1..{min(self.E, ops.MOE_MAX_TOP)} ({self.E} experts)")
+        self.renormalize, self.identity = bool(renormalize), int(identity)
+        n = self.E + self.identity                       # what the router chooses among
+        if self.identity < 0 or not 1 <= self.top <= min(n, ops.MOE_MAX_TOP):
+            raise ConfigError(f"moe: top {self.top} must be in 1..{min(n, ops.MOE_MAX_TOP)} ({n} experts)")
         if score not in ("softmax", "sigmoid"):
             raise ConfigError(f"moe: unknown score {score!r} (softmax, sigmoid)")
-        if score == "softmax" and (correction or groups):
-            raise ConfigError("moe: a correction of the choice and groups of experts go with sigmoid scores")
         self.score, self.groups = score, None
         if groups:
             count, keep, best = (int(v) for v in groups)
-            if count < 1 or self.E % count or not 1 <= keep <= count or best < 1:
-                raise ConfigError(f"moe: {count} groups (keep {keep}) do not divide {self.E} experts")
-            if self.top > (self.E // count) * keep:
-                raise ConfigError(f"moe: top {self.top} is above the {(self.E // count) * keep} experts of {keep} groups")
+            if count < 1 or n % count or not 1 <= keep <= count or best < 1:
+                raise ConfigError(f"moe: {count} groups (keep {keep}) do not divide {n} experts")
+            if self.top > (n // count) * keep:
+                raise ConfigError(f"moe: top {self.top} is above the {(n // count) * keep} experts of {keep} groups")
             self.groups = (count, keep, best)
         self.act = None
         if act:
@@ -64,11 +67,11 @@ class RoutedExperts(FeedForward):
         if plain and act:
             raise ConfigError("moe: plain experts have no gated activation")
         self.plain = plain
-        self.decls = {"router.weight": ParamDecl((self.E, self.size), init=("normal", 0.5))}
+        self.decls = {"router.weight": ParamDecl((n, self.size), init=("normal", 0.5))}
         if router_bias:
-            self.decls["router.bias"] = ParamDecl((self.E,), role="vector", init=("normal", 0.5))
+            self.decls["router.bias"] = ParamDecl((n,), role="vector", init=("normal", 0.5))
         if correction:
-            self.decls["correction"] = ParamDecl((self.E,), role="vector", init=("normal", 0.2))
+            self.decls["correction"] = ParamDecl((n,), role="vector", init=("normal", 0.2))
         for e in range(self.E):
             if not self.plain:
                 self.decls[f"e{e}.gate.weight"] = ParamDecl((self.ff, self.size))
@@ -104,6 +107,7 @@ class RoutedExperts(FeedForward):
         w = self.w
         idx, score = ops.moe_router(hn, w["router.weight"], self.top, self.renormalize, score=self.score,
                                     correction=w.get("correction"), groups=self.groups, bias=w.get("router.bias"))
+        h = hn if self.identity else None                # what an identity expert hands on
         first = w["up.weight"] if self.plain else w["gate_up.weight"]
         if hn.dtype != first.dtype:          # a file that stores some experts in 32-bit under a bfloat16 engine
             hn = hn.to(first.dtype)
@@ -114,11 +118,11 @@ class RoutedExperts(FeedForward):
         if self.plain:
             a = ops.relu2(ops.moe_gemm(hn, first, plan, gated=False, gather=True), hn.dtype)
             y = ops.moe_gemm(a, w["down.weight"], plan, gated=False, gather=False)
-            ops.moe_combine(out, y, plan, score, store=store)
+            ops.moe_combine(out, y, plan, score, store=store, identity=h)
             return out
         a = ops.moe_gemm(hn, w["gate_up.weight"], plan, gated=True, gather=True, interleaved=self.interleaved, act=self.act)
         y = ops.moe_gemm(a, w["down.weight"], plan, gated=False, gather=False)
-        ops.moe_combine(out, y, plan, score, store=store)
+        ops.moe_combine(out, y, plan, score, store=store, identity=h)
         return out
 
     def weight_order(self):
