@@ -29,6 +29,13 @@
 #ifndef VD
 #define VD HD
 #endif
+// -DEXT: the library of layers whose single tokens also take a soft cap, a gate on the outputs and q and k normed over their
+// whole projections (the others' decode kernels carry none of that code).
+#ifdef EXT
+constexpr bool EXTENDED = true;
+#else
+constexpr bool EXTENDED = false;
+#endif
 static_assert(HD % 16 == 0 && HD >= 16 && HD <= 256, "head size: a multiple of 16 in 16..256");
 static_assert(VD % 16 == 0 && VD >= 16 && VD <= 256, "size of values: a multiple of 16 in 16..256");
 
@@ -78,11 +85,37 @@ __device__ __forceinline__ unsigned pack_bf16(float lo, float hi) {
   return *(unsigned*)&v;
 }
 
+// s (N times four scores, elements 0 and 1 times f0, 2 and 3 times f1 in the log2 domain) under a soft cap of cap_log2; a whole
+// warp takes tanh's cheap form where all of its scores are small.
+template <int N>
+__device__ __forceinline__ void cap_scores(float (&s)[N][4], float f0, float f1, float cap_log2) {
+  const float inv = 1.0f / cap_log2, g0 = f0 * inv, g1 = f1 * inv;
+  float am = 0.f;
+#pragma unroll
+  for (int n = 0; n < N; ++n) {
+#pragma unroll
+    for (int e = 0; e < 4; ++e) { s[n][e] *= e < 2 ? g0 : g1; am = fmaxf(am, fabsf(s[n][e])); }
+  }
+  if (__all_sync(0xffffffffu, am <= SOFT_CAP_SERIES_TO)) {
+#pragma unroll
+    for (int n = 0; n < N; ++n) {
+#pragma unroll
+      for (int e = 0; e < 4; ++e) s[n][e] = cap_log2 * tanh_series(s[n][e]);
+    }
+  } else {
+#pragma unroll
+    for (int n = 0; n < N; ++n) {
+#pragma unroll
+      for (int e = 0; e < 4; ++e) s[n][e] = cap_log2 * tanh_any(s[n][e]);
+    }
+  }
+}
+
 // One 16-row block of queries (fragments qf) against NKT*8 keys staged at k_s / v_s (shared-memory
 // addresses of [keys][ROWB] and [keys][ROWBV] tiles).  Thread (g = lane/4, c = lane%4) owns rows g and g+8; a key at
 // tile index i (absolute index key0 + i) counts for row r iff lo[r] <= key0 + i <= hi[r].
 // m, l: running maximum (log2 domain) and this thread's share of the running sum per row.
-// CAPPED: scores are soft-capped, cap * tanh(s * scale / cap), with cap_log2 = cap * log2(e).
+// CAPPED: scores are soft-capped, cap * tanh(s * scale / cap), with cap_log2 = cap * log2(e) (0: no cap after all).
 // BIASED: row r's scores are multiplied by rs[r] (a query temperature: the factor of q taken out of the dot product)
 // and sl[r] * (hi[r] - key) is taken off them (a bias by distance; sl = slope * log2(e), hi[r] = the row's position).
 // ATOM > 0: the tiles lie as bulk tensor copies bring them, 64 elements of every key (128 bytes, swizzled) in ATOM bytes,
@@ -112,6 +145,8 @@ __device__ __forceinline__ void attend_tile(const unsigned (&qf)[KS][4], unsigne
   }
   // scale, mask, running maximum
   float mx[2] = {m[0], m[1]};
+  if (CAPPED && cap_log2 > 0.f) cap_scores<NKT>(s, BIASED ? rs[0] * scale_log2 : scale_log2, BIASED ? rs[1] * scale_log2 : scale_log2, cap_log2);
+  const bool scaled = CAPPED && cap_log2 > 0.f;
   // BIASED: the row's factor of the score, and the bias of the tile's key 2c for the row (the rest is slope * offset)
   float a_row[2] = {scale_log2, scale_log2}, b_row[2] = {0.f, 0.f};
   if (BIASED) {
@@ -124,8 +159,7 @@ __device__ __forceinline__ void attend_tile(const unsigned (&qf)[KS][4], unsigne
     for (int e = 0; e < 4; ++e) {
       int key = key0 + n * 8 + 2 * c + (e & 1);
       int r = e >> 1;
-      float sc = s[n][e] * (BIASED ? a_row[r] : scale_log2);
-      if (CAPPED) sc = cap_log2 * tanhf(sc / cap_log2);
+      float sc = scaled ? s[n][e] : s[n][e] * (BIASED ? a_row[r] : scale_log2);
       if (BIASED) sc += fmaf(sl[r], (float)(n * 8 + (e & 1)), b_row[r]);       // - slope * (hi - key)
       float v = (!MASKED || (key >= lo[r] && key <= hi[r])) ? sc : -INFINITY;
       s[n][e] = v;
@@ -214,10 +248,10 @@ __device__ __forceinline__ void load_q_as_b(unsigned (&qb)[KS][2], F row_ptr, in
 // NKT*8 keys at k_s / v_s against the heads in qb; a key counts iff lo <= key0 + i <= hi.  ot[dm] = O^T of dims
 // dm*16 + g (elements 0, 1: heads 2c, 2c+1) and dm*16 + g + 8 (elements 2, 3); m, l per head 2c, 2c+1 (l: this
 // thread's keys only).
-template <int NKT, bool MASKED, int ATOM = 0>
+template <int NKT, bool MASKED, int ATOM = 0, bool CAPPED = false>
 __device__ __forceinline__ void attend_tile_keys_as_rows(const unsigned (&qb)[KS][2], unsigned k_s, unsigned v_s, int key0,
                                                          int lo, int hi, float scale_log2, float (&ot)[VD / 16][4],
-                                                         float (&m)[2], float (&l)[2], int lane) {
+                                                         float (&m)[2], float (&l)[2], int lane, float cap_log2 = 0.f) {
   constexpr int KB = NKT / 2;                            // blocks of 16 keys
   const int g = lane >> 2;
   float s[KB][4];
@@ -236,12 +270,14 @@ __device__ __forceinline__ void attend_tile_keys_as_rows(const unsigned (&qb)[KS
     }
   }
   float mx[2] = {m[0], m[1]};
+  const bool scaled = CAPPED && cap_log2 > 0.f;
+  if (scaled) cap_scores<KB>(s, scale_log2, scale_log2, cap_log2);
 #pragma unroll
   for (int b = 0; b < KB; ++b) {
 #pragma unroll
     for (int e = 0; e < 4; ++e) {
       const int key = key0 + b * 16 + g + ((e >> 1) << 3);
-      const float v = (!MASKED || (key >= lo && key <= hi)) ? s[b][e] * scale_log2 : -INFINITY;
+      const float v = (!MASKED || (key >= lo && key <= hi)) ? (scaled ? s[b][e] : s[b][e] * scale_log2) : -INFINITY;
       s[b][e] = v;
       mx[e & 1] = fmaxf(mx[e & 1], v);
     }
@@ -304,7 +340,14 @@ struct AttnArgs {
   const float* slopes; float qt_coef; int qt_every, kv_planes;
   // sinks [H] (null: none): exp(sinks[h]) joins the denominator of head h's softmax once, with no key and no value
   const float* sinks;
+  // EXT: a gate [T, ldog] of H * VD elements a row (null: none): the outputs times its sigmoid, element by element
+  const bf16* og; int ldog;
 };
+// Element d of head h of row t on its way out.
+__device__ __forceinline__ float gated_out(const AttnArgs& a, int t, int h, int d, float v) {
+  if (EXTENDED && a.og) v *= 1.0f / (1.0f + expf(-__bfloat162float(a.og[(size_t)t * a.ldog + (size_t)h * VD + d])));
+  return v;
+}
 
 // One page of one layer: the keys [G][page_tokens][HD], then (unless they are the values too) the values [G][page_tokens][VD].
 __device__ __forceinline__ size_t record_elems(const AttnArgs& a) {
@@ -456,7 +499,8 @@ __global__ void __launch_bounds__(PF_WARPS * 32) attention_prefill_kernel(AttnAr
       bf16* dst = a.out + ((size_t)(row_begin + tok0 + tok[r]) * a.H + g * R + hr[r]) * VD;
 #pragma unroll
       for (int d = 0; d < DN; ++d)
-        *(unsigned*)(dst + d * 8 + 2 * c) = pack_bf16(o[d][2 * r] * inv, o[d][2 * r + 1] * inv);
+        *(unsigned*)(dst + d * 8 + 2 * c) = pack_bf16(gated_out(a, row_begin + tok0 + tok[r], g * R + hr[r], d * 8 + 2 * c, o[d][2 * r] * inv),
+                                                      gated_out(a, row_begin + tok0 + tok[r], g * R + hr[r], d * 8 + 2 * c + 1, o[d][2 * r + 1] * inv));
     }
   }
 }
@@ -532,7 +576,7 @@ __device__ __forceinline__ void decode_merge_records(const AttnArgs& a, const fl
     }
     int h = g * R + r0 + row;
     if (n_active == 1) {
-      a.out[((size_t)t * a.H + h) * VD + d] = __float2bfloat16_rn(a.sinks ? at * denominator_inv(a, h, mx, lt) : at / lt);
+      a.out[((size_t)t * a.H + h) * VD + d] = __float2bfloat16_rn(gated_out(a, t, h, d, a.sinks ? at * denominator_inv(a, h, mx, lt) : at / lt));
     } else {
       float* rec = cta_rec ? cta_rec + (size_t)(r0 + row) * SW
                            : a.scratch + (((size_t)t * a.H + h) * a.max_splits + split_index) * SW;
@@ -569,7 +613,7 @@ __device__ __forceinline__ void decode_last_cta_merges(const AttnArgs& a, int* s
       lt += rec[(size_t)j * SW + VD + 1] * cj;
       at += rec[(size_t)j * SW + d] * cj;
     }
-    a.out[((size_t)t * a.H + h) * VD + d] = __float2bfloat16_rn(a.sinks ? at * denominator_inv(a, h, mx, lt) : at / lt);
+    a.out[((size_t)t * a.H + h) * VD + d] = __float2bfloat16_rn(gated_out(a, t, h, d, a.sinks ? at * denominator_inv(a, h, mx, lt) : at / lt));
   }
 }
 
@@ -647,7 +691,7 @@ __global__ void __launch_bounds__(DC_WARPS * 32) attention_decode_kernel(AttnArg
       cp_async_wait<DC_STAGES - 1>();
       __syncwarp();
       unsigned ks = ring + (j % DC_STAGES) * STAGE_B, vs = ks + TILE_B;
-      attend_tile<DC_TK / 8>(qf, ks, vs, k0 + (j * DC_WARPS + warp) * DC_TK, lo, hi, a.scale_log2, o, m, l, lane);
+      attend_tile<DC_TK / 8, true, EXTENDED>(qf, ks, vs, k0 + (j * DC_WARPS + warp) * DC_TK, lo, hi, a.scale_log2, o, m, l, lane, a.cap_log2);
       __syncwarp();
     }
     cp_async_wait<0>();
@@ -752,7 +796,8 @@ __device__ __forceinline__ void decode_cluster_merges(const AttnArgs& a, const f
         lt += lj[j] * cj;
         at += aj[j] * cj;
       }
-      a.out[((size_t)t * a.H + g * R + r) * VD + d] = __float2bfloat16_rn(a.sinks ? at * denominator_inv(a, g * R + r, mx, lt) : at / lt);
+      a.out[((size_t)t * a.H + g * R + r) * VD + d] =
+          __float2bfloat16_rn(gated_out(a, t, g * R + r, d, a.sinks ? at * denominator_inv(a, g * R + r, mx, lt) : at / lt));
     }
   }
   cluster_barrier();                                     // nobody leaves while its record may be read
@@ -1143,6 +1188,7 @@ static int fill_args(AttnArgs& a, const void* q, const void* pool, const int* bl
   a.item_start = nullptr; a.scratch = nullptr; a.counters = nullptr; a.split_len = 1; a.max_splits = 1; a.n_items = 0;
   a.ldq = H * HD; a.chunk = 0; a.ldg = 0; a.cap_log2 = 0.f; a.gate = nullptr;
   a.slopes = nullptr; a.qt_coef = 0.f; a.qt_every = 0; a.kv_planes = 2; a.sinks = nullptr;
+  a.og = nullptr; a.ldog = 0;
   return 0;
 }
 
@@ -1164,19 +1210,28 @@ struct WideFuse {
   const bf16* qkv; const bf16* v0; const float* lam; const float* inv_freq;
   int ld, ldv0, rot_dim, pairing;
   float mag;
+  // EXT: all of a row's q, and all of its k, over their root mean square times a weight per element before the rotation (qw
+  // [H HD], kw [G HD]; null: no norm); reads_only: the rows hold no k and v, the pages are another layer's, which an
+  // earlier kernel of this step has written
+  const float* qw; const float* kw;
+  float eps;
+  int reads_only;
 };
 
 __device__ __forceinline__ void dw_tma_load_3d(unsigned dst, const CUtensorMap* map, int c0, int c1, int c2, unsigned bar) {
   asm volatile("cp.async.bulk.tensor.3d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%3, %4, %5}], [%2];\n"
                ::"r"(dst), "l"(map), "r"(bar), "r"(c0), "r"(c1), "r"(c2) : "memory");
 }
-// Element e of a head, rotated (sines and cosines of its pairs in sn, cs).
-__device__ __forceinline__ float dw_rotated(const bf16* src, int e, int rot_dim, int pairing, const float* sn, const float* cs) {
-  const float x = __bfloat162float(src[e]);
+// Element e of a head, rotated (sines and cosines of its pairs in sn, cs); EXT: times factor and its weight before that (w
+// null: neither).
+__device__ __forceinline__ float dw_rotated(const bf16* src, int e, int rot_dim, int pairing, const float* sn, const float* cs,
+                                            const float* w = nullptr, float factor = 1.f) {
+  auto at = [&](int i) { const float v = __bfloat162float(src[i]); return EXTENDED && w ? v * factor * w[i] : v; };
+  const float x = at(e);
   if (e >= rot_dim) return x;
   const int half = rot_dim >> 1, i = pairing ? (e < half ? e : e - half) : e >> 1;
   const bool first = pairing ? e < half : !(e & 1);
-  const float y = __bfloat162float(src[pairing ? (first ? e + half : e - half) : (e ^ 1)]);
+  const float y = at(pairing ? (first ? e + half : e - half) : (e ^ 1));
   return first ? x * cs[i] - y * sn[i] : x * cs[i] + y * sn[i];
 }
 
@@ -1191,13 +1246,15 @@ attention_decode_wide_kernel(const __grid_constant__ CUtensorMap k_map, const __
   __shared__ int sm_last;
   __shared__ __align__(16) bf16 q_s[16 * HD];            // the group's heads, rotated
   __shared__ float sn_s[HD / 2], cs_s[HD / 2];
+  __shared__ float ssq_s[2][DC_WARPS];
   const int s = blockIdx.x, g = blockIdx.y, t = blockIdx.z;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int pos = a.positions[t];
   const int kb = (a.window > 0 && pos - a.window + 1 > 0) ? pos - a.window + 1 : 0;
+  const int origin = kb / DT_PT * DT_PT;                // the ranges start at the window's first page
   // (a launch with fewer key ranges than the longest row has: the last range takes every key behind it)
   const int s_end = (int)gridDim.x - 1;
-  const int s_lo = min(kb / a.split_len, s_end), s_hi = min(pos / a.split_len, s_end);
+  const int s_lo = 0, s_hi = min((pos - origin) / a.split_len, s_end);
   pdl_launch_dependents();
   const bool active = s >= s_lo && s <= s_hi;
   if (!CL && !active) return;
@@ -1207,7 +1264,7 @@ attention_decode_wide_kernel(const __grid_constant__ CUtensorMap k_map, const __
   float* merge = (float*)(smem_raw + (base - (unsigned)__cvta_generic_to_shared(smem_raw)));  // over the tiles, once the warps are done
   float* cta_rec = CL ? merge + DC_WARPS * 16 * (VD + 2) : nullptr;
   if (active) {
-    const int k0 = max(kb, s * a.split_len), k1 = s == s_end ? pos + 1 : min(pos + 1, (s + 1) * a.split_len);
+    const int k0 = max(kb, origin + s * a.split_len), k1 = s == s_end ? pos + 1 : min(pos + 1, origin + (s + 1) * a.split_len);
     const int* bt = a.block_table + (size_t)a.row_slot[t] * a.max_pages;
     const int pg0 = k0 / DT_PT, n_pg = (k1 - 1) / DT_PT - pg0 + 1;
     const bool pages_in_smem = n_pg <= DC_MAX_PAGES;
@@ -1232,11 +1289,15 @@ attention_decode_wide_kernel(const __grid_constant__ CUtensorMap k_map, const __
       for (int i = 0; i < DW_VA; ++i) dw_tma_load_3d(st + (DW_KA + i) * DW_ATOM, &v_map, 64 * i, row, rec, bar);
     };
     // The kernel in front (the input product) writes nothing of the cache, and the row of the step's own position is
-    // replaced in its tile: the first tiles are asked for before the wait.
-    if (lane == 0) {
+    // replaced in its tile: the first tiles are asked for before the wait (another layer's pages: behind it).
+    auto request_first = [&]() {
+      if (lane == 0) {
 #pragma unroll
-      for (int q = 0; q < NS; ++q) if (q < n_tiles) request(q);
-    }
+        for (int q = 0; q < NS; ++q) if (q < n_tiles) request(q);
+      }
+    };
+    const bool reads_only = EXTENDED && f.reads_only;
+    if (!reads_only) request_first();
     for (int i = threadIdx.x; i < f.rot_dim / 2; i += DC_WARPS * 32) {
       float sn, cs;
       sincosf((float)pos * f.inv_freq[i], &sn, &cs);
@@ -1244,10 +1305,36 @@ attention_decode_wide_kernel(const __grid_constant__ CUtensorMap k_map, const __
     }
     __syncthreads();
     pdl_wait(); FELLM_TRACE_WAITED();
+    if (reads_only) request_first();
     const bf16* row = f.qkv + (size_t)t * f.ld;
+    float q_factor = 1.f, k_factor = 1.f;
+    if constexpr (EXTENDED) {
+      if (f.qw) {
+        // the whole projections' sums of squares: every thread's share in order, lanes by a butterfly, warps in order
+        const int nq = a.H * HD, nk = reads_only ? 0 : a.G * HD;
+        float sq = 0.f, sk = 0.f;
+        for (int u = threadIdx.x; u < (nq + nk) / 8; u += DC_WARPS * 32) {
+          const uint4 raw = *(const uint4*)(row + 8 * u);
+          const __nv_bfloat162* h2 = (const __nv_bfloat162*)&raw;
+          float ss = 0.f;
+#pragma unroll
+          for (int e = 0; e < 4; ++e) { const float2 v = __bfloat1622float2(h2[e]); ss = fmaf(v.x, v.x, ss); ss = fmaf(v.y, v.y, ss); }
+          if (8 * u < nq) sq += ss; else sk += ss;
+        }
+        sq = warp_sum(sq); sk = warp_sum(sk);
+        if (lane == 0) { ssq_s[0][warp] = sq; ssq_s[1][warp] = sk; }
+        __syncthreads();
+        sq = sk = 0.f;
+#pragma unroll
+        for (int w = 0; w < DC_WARPS; ++w) { sq += ssq_s[0][w]; sk += ssq_s[1][w]; }
+        q_factor = 1.0f / sqrtf(sq / (float)nq + f.eps);
+        if (nk) k_factor = 1.0f / sqrtf(sk / (float)nk + f.eps);
+      }
+    }
     for (int i = threadIdx.x; i < R * HD; i += DC_WARPS * 32) {
       const int r = i / HD, e = i - r * HD;
-      q_s[i] = __float2bfloat16_rn(dw_rotated(row + (size_t)(g * R + r) * HD, e, f.rot_dim, f.pairing, sn_s, cs_s));
+      q_s[i] = __float2bfloat16_rn(dw_rotated(row + (size_t)(g * R + r) * HD, e, f.rot_dim, f.pairing, sn_s, cs_s,
+                                              EXTENDED && f.qw ? f.qw + (size_t)(g * R + r) * HD : nullptr, q_factor));
     }
     __syncthreads();
     auto q_row = [&](int i) -> const bf16* { return i < R ? q_s + i * HD : nullptr; };
@@ -1271,7 +1358,7 @@ attention_decode_wide_kernel(const __grid_constant__ CUtensorMap k_map, const __
         break;
       }
       const int key0 = (pg0 + warp + (q >> 1) * DC_WARPS) * DT_PT + (q & 1) * DT_HALF;
-      if (s == s_hi && key0 <= pos && pos < key0 + DT_HALF) {
+      if (!reads_only && s == s_hi && key0 <= pos && pos < key0 + DT_HALF) {
         // this tile holds the step's own position; no other CTA or warp reads this page's tile in this step
         const int lp = pos / DT_PT;
         const int page = pages_in_smem ? sm_pages[lp - pg0] : bt[lp];
@@ -1283,7 +1370,8 @@ attention_decode_wide_kernel(const __grid_constant__ CUtensorMap k_map, const __
         const float lam = f.v0 ? *f.lam : 0.f;
         const int at = pos - key0;
         for (int e = lane; e < HD; e += 32) {
-          const bf16 v = __float2bfloat16_rn(dw_rotated(ksrc, e, f.rot_dim, f.pairing, sn_s, cs_s));
+          const bf16 v = __float2bfloat16_rn(dw_rotated(ksrc, e, f.rot_dim, f.pairing, sn_s, cs_s,
+                                                        EXTENDED && f.qw ? f.kw + (size_t)g * HD : nullptr, k_factor));
           asm volatile("st.shared.b16 [%0], %1;\n" ::"r"(st + atom_off<DW_ATOM>(at, e >> 3) + (e & 7) * 2), "h"(*(const unsigned short*)&v) : "memory");
           if (page >= 0) krow[e] = v;
         }
@@ -1305,11 +1393,11 @@ attention_decode_wide_kernel(const __grid_constant__ CUtensorMap k_map, const __
         }
         const bool edge = key0 < k0 || key0 + DT_HALF > k1;
         if constexpr (KR) {
-          if (edge) attend_tile_keys_as_rows<DT_HALF / 8, true, DW_ATOM>(qb, st, vt, key0, k0, k1 - 1, a.scale_log2, ot, m, l, lane);
-          else attend_tile_keys_as_rows<DT_HALF / 8, false, DW_ATOM>(qb, st, vt, key0, k0, k1 - 1, a.scale_log2, ot, m, l, lane);
+          if (edge) attend_tile_keys_as_rows<DT_HALF / 8, true, DW_ATOM, EXTENDED>(qb, st, vt, key0, k0, k1 - 1, a.scale_log2, ot, m, l, lane, a.cap_log2);
+          else attend_tile_keys_as_rows<DT_HALF / 8, false, DW_ATOM, EXTENDED>(qb, st, vt, key0, k0, k1 - 1, a.scale_log2, ot, m, l, lane, a.cap_log2);
         } else {
-          if (edge) attend_tile<DT_HALF / 8, true, false, false, DW_ATOM>(qf, st, vt, key0, lo, hi, a.scale_log2, o, m, l, lane);
-          else attend_tile<DT_HALF / 8, false, false, false, DW_ATOM>(qf, st, vt, key0, lo, hi, a.scale_log2, o, m, l, lane);
+          if (edge) attend_tile<DT_HALF / 8, true, EXTENDED, false, DW_ATOM>(qf, st, vt, key0, lo, hi, a.scale_log2, o, m, l, lane, a.cap_log2);
+          else attend_tile<DT_HALF / 8, false, EXTENDED, false, DW_ATOM>(qf, st, vt, key0, lo, hi, a.scale_log2, o, m, l, lane, a.cap_log2);
         }
       }
       __syncwarp();
@@ -1380,12 +1468,16 @@ static int launch_wide(const CUtensorMap& k_map, const CUtensorMap& v_map, const
 // take).  qkv [T, ld]: the input product's rows [q (H hd) | k (G hd) | v (G vd)]; v0 (or null) [T, ldv0] with lam (one float
 // on the device): the values the layer's are mixed with; inv_freq [rot_dim / 2] or null, pairing 0 adjacent / 1 split-half,
 // cos and sin times mag; sinks [H] or null; scratch and counters as fellm_attn_decode_mma; stages: half pages a warp keeps in
-// flight (2, or 4 where they fit); status 301: a wait ran out, 302: a row's position has no page.
+// flight (2, or 4 where they fit); status 301: a wait ran out, 302: a row's position has no page.  With -DEXT also: softcap (0:
+// none); og [T, ldog] (null: none), the outputs times its sigmoid; qw float32 [H hd] and kw [G hd] (null: none), q and k over
+// their projections' root mean squares (eps inside) times these before the rotation; reads_only: the rows are [q] alone and the
+// pages another layer's.
 FELLM_API int fellm_attn_decode_wide(const void* qkv, int ld, const void* pool, long long n_pages, const int* block_table, int max_pages,
                                      const int* positions, const int* row_slot, void* out, float* scratch, int* counters, int T, int H,
                                      int G, int hd, int vd, int page_tokens, int layer, int layers_in_group, float scale, int window,
                                      int split_len, int max_splits, const float* inv_freq, int rot_dim, int pairing, float mag,
                                      const void* v0, int ldv0, const float* lam, const float* sinks, int stages, int cluster, int* status,
+                                     float softcap, const void* og, int ldog, const float* qw, const float* kw, float eps, int reads_only,
                                      cudaStream_t stream) {
 #ifdef WIDE
   if (T <= 0) return 0;
@@ -1398,11 +1490,16 @@ FELLM_API int fellm_attn_decode_wide(const void* qkv, int ld, const void* pool, 
   if (!inv_freq) rot_dim = 0;
   const long long records = n_pages * layers_in_group;
   if (page_tokens != DT_PT || H / G > 16 || (split_len % DT_PT) || records >= (1ll << 31) || ((uintptr_t)pool & 15) ||
-      ld < H * hd + G * (hd + vd) || (v0 && ldv0 < G * vd) || rot_dim < 0 || rot_dim > hd || (rot_dim & 1)) return FELLM_ERR_SIZE;
+      ld < H * hd + (reads_only ? 0 : G * (hd + vd)) || (v0 && ldv0 < G * vd) || rot_dim < 0 || rot_dim > hd || (rot_dim & 1)) return FELLM_ERR_SIZE;
   a.ldq = ld; a.sinks = sinks; a.scratch = scratch; a.counters = counters; a.split_len = split_len; a.max_splits = max_splits;
   WideFuse f;
   f.qkv = (const bf16*)qkv; f.v0 = (const bf16*)v0; f.lam = lam; f.inv_freq = inv_freq; f.ld = ld; f.ldv0 = ldv0;
   f.rot_dim = rot_dim; f.pairing = pairing; f.mag = mag;
+  if (!EXTENDED && (softcap > 0.f || og || qw || reads_only)) return FELLM_ERR_SIZE;
+  if (softcap < 0.f || (og && ldog < H * vd) || (qw && !reads_only && !kw) || (reads_only && v0)) return FELLM_ERR_ARG;
+  if (qw && ((ld & 7) || ((uintptr_t)qkv & 15))) return FELLM_ERR_SIZE;
+  a.cap_log2 = softcap * 1.4426950408889634f; a.og = (const bf16*)og; a.ldog = ldog;
+  f.qw = qw; f.kw = kw; f.eps = eps; f.reads_only = reads_only;
   CUtensorMap k_map, v_map;
   e = dw_pool_map((const bf16*)pool, HD, records, G, &k_map);
   if (!e) e = dw_pool_map((const bf16*)pool + (size_t)G * DT_PT * HD, VD, records, G, &v_map);
@@ -1440,13 +1537,15 @@ FELLM_API int fellm_attn_prefill_mma(const void* q, const void* pool, const int*
 }
 
 // The same with a bias by distance (slopes float32 [H], null: none), a query temperature (qt_every 0: none) and values
-// that are the keys (v_is_k: a page-layer record is the keys [G][page_tokens][hd] alone); sinks: float32 [H] or null.
+// that are the keys (v_is_k: a page-layer record is the keys [G][page_tokens][hd] alone); sinks: float32 [H] or null; og [T,
+// ldog] (null: none; with -DEXT alone): the outputs times its sigmoid.
 FELLM_API int fellm_attn_prefill_mma_biased(const void* q, int ldq, const void* pool, const int* block_table, int max_pages,
                                             const int* positions, const int* row_slot, const int* item_start, int n_items,
                                             int max_item_rows, void* out, int T, int H, int G, int hd, int page_tokens,
                                             int layer, int layers_in_group, float scale, int window, int chunk,
                                             float softcap, const float* gate, int ldg, const float* slopes, float qt_coef,
-                                            int qt_every, int v_is_k, const float* sinks, cudaStream_t stream);
+                                            int qt_every, int v_is_k, const float* sinks, const void* og, int ldog,
+                                            cudaStream_t stream);
 
 FELLM_API int fellm_attn_prefill_mma_general(const void* q, int ldq, const void* pool, const int* block_table, int max_pages,
                                              const int* positions, const int* row_slot, const int* item_start, int n_items,
@@ -1455,7 +1554,7 @@ FELLM_API int fellm_attn_prefill_mma_general(const void* q, int ldq, const void*
                                              float softcap, const float* gate, int ldg, cudaStream_t stream) {
   return fellm_attn_prefill_mma_biased(q, ldq, pool, block_table, max_pages, positions, row_slot, item_start, n_items,
                                        max_item_rows, out, T, H, G, hd, page_tokens, layer, layers_in_group, scale, window,
-                                       chunk, softcap, gate, ldg, nullptr, 0.f, 0, 0, nullptr, stream);
+                                       chunk, softcap, gate, ldg, nullptr, 0.f, 0, 0, nullptr, nullptr, 0, stream);
 }
 
 FELLM_API int fellm_attn_prefill_mma_biased(const void* q, int ldq, const void* pool, const int* block_table, int max_pages,
@@ -1463,7 +1562,8 @@ FELLM_API int fellm_attn_prefill_mma_biased(const void* q, int ldq, const void* 
                                             int max_item_rows, void* out, int T, int H, int G, int hd, int page_tokens,
                                             int layer, int layers_in_group, float scale, int window, int chunk,
                                             float softcap, const float* gate, int ldg, const float* slopes, float qt_coef,
-                                            int qt_every, int v_is_k, const float* sinks, cudaStream_t stream) {
+                                            int qt_every, int v_is_k, const float* sinks, const void* og, int ldog,
+                                            cudaStream_t stream) {
   if (T <= 0 || n_items <= 0) return 0;
   AttnArgs a;
   int e = fill_args(a, q, pool, block_table, max_pages, positions, row_slot, out, T, H, G, hd, page_tokens, layer,
@@ -1473,7 +1573,8 @@ FELLM_API int fellm_attn_prefill_mma_biased(const void* q, int ldq, const void* 
   if (ldq < H * hd || (ldq & 1) || chunk < 0 || softcap < 0.f) return FELLM_ERR_ARG;
   a.ldq = ldq; a.chunk = chunk; a.cap_log2 = softcap * 1.4426950408889634f; a.gate = gate; a.ldg = ldg;
   if (qt_every < 0 || (v_is_k && VD != HD)) return FELLM_ERR_ARG;
-  a.sinks = sinks;
+  if (og && (!EXTENDED || ldog < H * VD)) return FELLM_ERR_SIZE;
+  a.sinks = sinks; a.og = (const bf16*)og; a.ldog = ldog;
   a.slopes = slopes; a.qt_coef = qt_coef; a.qt_every = qt_every; a.kv_planes = v_is_k ? 1 : 2;
   int R = H / G;
   if (R > PF_WARPS * 16) return FELLM_ERR_SIZE;
@@ -1490,19 +1591,21 @@ FELLM_API int fellm_attn_prefill_mma_biased(const void* q, int ldq, const void* 
 
 // One query row per item (head h of row t at q + t ldq + h hd).  scratch: float32 [T*H*max_splits*(VD+2)]; counters: int32 [T*G], zero
 // before the first launch (the kernel leaves them zero).  max_splits >= ceil(longest context / split_len).  sinks: float32
-// [H] or null.
+// [H] or null.  With -DEXT also softcap (0: none) and og [T, ldog] (null: none), the outputs times its sigmoid.
 FELLM_API int fellm_attn_decode_mma(const void* q, int ldq, const void* pool, const int* block_table, int max_pages,
                                     const int* positions, const int* row_slot, void* out, float* scratch,
                                     int* counters, int T, int H, int G, int hd, int page_tokens, int layer,
                                     int layers_in_group, float scale, int window, int split_len, int max_splits,
-                                    const float* sinks, cudaStream_t stream) {
+                                    const float* sinks, float softcap, const void* og, int ldog, cudaStream_t stream) {
   if (T <= 0) return 0;
   AttnArgs a;
   int e = fill_args(a, q, pool, block_table, max_pages, positions, row_slot, out, T, H, G, hd, page_tokens, layer,
                     layers_in_group, scale, window);
   if (e) return e;
   if (ldq < H * hd || (ldq & 1)) return FELLM_ERR_ARG;
-  a.ldq = ldq; a.sinks = sinks;
+  if (!EXTENDED && (softcap > 0.f || og)) return FELLM_ERR_SIZE;
+  if (softcap < 0.f || (og && ldog < H * VD)) return FELLM_ERR_ARG;
+  a.ldq = ldq; a.sinks = sinks; a.cap_log2 = softcap * 1.4426950408889634f; a.og = (const bf16*)og; a.ldog = ldog;
   if (!scratch || !counters || split_len < 1 || max_splits < 1) return FELLM_ERR_ARG;
   a.scratch = scratch; a.counters = counters; a.split_len = split_len; a.max_splits = max_splits;
   size_t ring = (size_t)DC_WARPS * DC_STAGES * DC_TK * (ROWB + ROWBV), mrg = (size_t)DC_WARPS * 16 * (VD + 2) * sizeof(float);

@@ -1,5 +1,5 @@
 // Causal attention of prompt portions over the paged cache on the Blackwell tensor path: pages of 64
-// tokens, no window, compiled for one size of keys and one of values (-DAU_KD, -DAU_VD: multiples of
+// tokens, no window (unless -DAU_EXT, below), compiled for one size of keys and one of values (-DAU_KD, -DAU_VD: multiples of
 // 16, 64 by default; what fits shared and tensor memory, AU_FITS below).  A CTA takes 128 rows (token, head of one kv head's group) and
 // walks over the pages of keys up to its last token:
 //   S = Q K^T      tcgen05.mma 128x64x16 (kind::f16), Q and the K page K-major in shared memory
@@ -9,6 +9,8 @@
 //                  with no shuffles, P rounded to bfloat16 into shared memory;
 //   O += P V       tcgen05.mma with the V page as the MN-major operand, accumulated in tensor memory.
 // A sink per head (a.sinks): exp(sink) joins the softmax's denominator once, with no key and no value.
+// With -DAU_EXT the kernel also takes a sliding window (the pages in front of a CTA's first window are not
+// walked), a soft cap on the scores and a gate on the outputs (o times sigmoid(gate), element by element).
 // A page-layer record of the pool is the keys [G][64][AU_KD], then the values [G][64][AU_VD].
 // The accumulator is scaled by 2^-m with m a row's REFERENCE maximum, which moves only when a tile's
 // maximum exceeds it by 2^8: only then is the accumulator read, scaled and written back.
@@ -39,6 +41,11 @@
 #ifndef AU_VD
 #define AU_VD 64
 #endif
+#ifdef AU_EXT
+constexpr bool AU_EXTENDED = true;
+#else
+constexpr bool AU_EXTENDED = false;
+#endif
 #define AU_PT 64                       // keys per tile: a page
 #define AU_ROWS 128
 #ifndef AU_GROUPS
@@ -67,6 +74,9 @@ struct AuArgs {
   const float* sinks;                  // [H] or null
   int max_pages, H, G, layer, layers_in_group, ldq;
   float scale_log2;
+  const bf16* og;                      // AU_EXT: a gate [T, ldog] (null: none), a window (0: none), a soft cap (cap_log2 0: none)
+  int ldog, window;
+  float cap_log2;
 };
 
 __device__ __forceinline__ unsigned au_smem(const void* p) { return (unsigned)__cvta_generic_to_shared(p); }
@@ -204,8 +214,10 @@ attention_prefill_umma_kernel(const __grid_constant__ CUtensorMap k_map, const _
   const int tok0 = blk * tokb, n_tok = min(tokb, n_rows - tok0);
   const int pos0 = a.positions[row_begin] + tok0;              // position of the block's first token
   const int k_last = pos0 + n_tok - 1;
-  const int n_tiles = k_last / AU_PT + 1;                      // pages 0 .. that of the last token
-  const int* bt = a.block_table + (size_t)a.row_slot[row_begin] * a.max_pages;
+  // tiles = pages first_page .. that of the last token; first_page: 0, or that of the first token's window
+  const int first_page = (AU_EXTENDED && a.window > 0) ? max(pos0 - a.window + 1, 0) / AU_PT : 0;
+  const int n_tiles = k_last / AU_PT + 1 - first_page;
+  const int* bt = a.block_table + (size_t)a.row_slot[row_begin] * a.max_pages + first_page;
 
   const unsigned base = (au_smem(smem_raw) + 1023u) & ~1023u;  // the swizzle is by address
   unsigned char* base_ptr = smem_raw + (base - au_smem(smem_raw));
@@ -306,7 +318,10 @@ attention_prefill_umma_kernel(const __grid_constant__ CUtensorMap k_map, const _
     const unsigned t_row = tmem_base + ((unsigned)(qd * 32) << 16);
     const unsigned t_acc = t_row + AU_COL_O + grp * AU_VC * 32;
     const unsigned s_full = s_full0 + 16 * grp, p_full = p_full0 + 16 * grp, o_full = o_full0 + 16 * grp;
-    const float scale = a.scale_log2;
+    const bool capped = AU_EXTENDED && a.cap_log2 > 0.f;
+    const float scale = capped ? 1.0f : a.scale_log2;            // (capped scores are in the log2 domain already)
+    const float cap_in = capped ? a.scale_log2 / a.cap_log2 : 0.f;
+    const int lo = (AU_EXTENDED && a.window > 0) ? pos - a.window + 1 : 0;         // the first key the row sees
     // The accumulator of P V stays in tensor memory, scaled by 2^-m where m is the row's REFERENCE
     // maximum; m only moves when a tile's maximum exceeds it by AU_RESCALE_AT (P then stays below 2^8,
     // well inside bfloat16 and float32), and only then is the accumulator read, scaled and written back.
@@ -314,7 +329,7 @@ attention_prefill_umma_kernel(const __grid_constant__ CUtensorMap k_map, const _
     bool ok = true;
     int n_mine = 0;
     for (int j = grp; j < n_tiles; j += AU_GROUPS, ++n_mine) {
-      const int key0 = j * AU_PT, s = j % AU_STAGES, i = n_mine;
+      const int key0 = (first_page + j) * AU_PT, s = j % AU_STAGES, i = n_mine;
       if (key0 + AU_PT > k_last + 1) {
         // rows past the last key hold whatever the page held before: zero the V rows, so that 0 * V is 0
         ok = au_wait(full0 + 8 * s, (j / AU_STAGES) & 1, fail, a.status, 315);
@@ -332,9 +347,25 @@ attention_prefill_umma_kernel(const __grid_constant__ CUtensorMap k_map, const _
       au_tmem_ld32_issue(t_row + AU_COL_S + (2 * grp + (i & 1)) * AU_PT, sc);
       au_tmem_ld32_issue(t_row + AU_COL_S + (2 * grp + (i & 1)) * AU_PT + 32, sc + 32);
       au_tmem_ld_wait();
+      if (capped) {
+        float am = 0.f;
+#pragma unroll
+        for (int c = 0; c < AU_PT; ++c) { sc[c] *= cap_in; am = fmaxf(am, fabsf(sc[c])); }
+        if (__all_sync(0xffffffffu, am <= SOFT_CAP_SERIES_TO)) {
+#pragma unroll
+          for (int c = 0; c < AU_PT; ++c) sc[c] = a.cap_log2 * tanh_series(sc[c]);
+        } else {
+#pragma unroll
+          for (int c = 0; c < AU_PT; ++c) sc[c] = a.cap_log2 * tanh_any(sc[c]);
+        }
+      }
       if (key0 + AU_PT - 1 > pos) {
 #pragma unroll
         for (int c = 0; c < AU_PT; ++c) sc[c] = (key0 + c <= pos) ? sc[c] : -INFINITY;
+      }
+      if (AU_EXTENDED && key0 < lo) {
+#pragma unroll
+        for (int c = 0; c < AU_PT; ++c) sc[c] = (key0 + c >= lo) ? sc[c] : -INFINITY;
       }
       float r4[4] = {sc[0], sc[1], sc[2], sc[3]};               // four chains, not one of 63 dependent steps
 #pragma unroll
@@ -420,7 +451,7 @@ attention_prefill_umma_kernel(const __grid_constant__ CUtensorMap k_map, const _
     }
     asm volatile("bar.sync 1, %0;\n" ::"n"(128 * AU_GROUPS) : "memory");
     if (grp == 0 && ok && !*fail && valid) {
-      float mm = m;                                            // group 0 has page 0: m is finite
+      float mm = m;                    // (-inf where the row sees none of group 0's pages: a window; the row's own page is somebody's)
 #pragma unroll
       for (int q = 0; q < AU_GROUPS - 1; ++q) mm = fmaxf(mm, merge[((size_t)q * AU_ROWS + row) * AU_MERGE_STRIDE + AU_VD]);
       const float sk = a.sinks ? a.sinks[g * R + head] * 1.4426950408889634f : -INFINITY;
@@ -439,6 +470,19 @@ attention_prefill_umma_kernel(const __grid_constant__ CUtensorMap k_map, const _
         for (int d = 0; d < AU_VD; ++d) o[d] = fmaf(rec[d], cq, o[d]);
       }
       const float inv = 1.0f / lt;
+      if (AU_EXTENDED && a.og) {
+        const uint4* gate = (const uint4*)(a.og + (size_t)(row_begin + tok0 + tok) * a.ldog + (size_t)(g * R + head) * AU_VD);
+#pragma unroll
+        for (int ch = 0; ch < AU_VD / 8; ++ch) {
+          const uint4 raw = gate[ch];
+          const __nv_bfloat162* h2 = (const __nv_bfloat162*)&raw;
+#pragma unroll
+          for (int e = 0; e < 4; ++e) {
+            const float2 z = __bfloat1622float2(h2[e]);
+            o[8 * ch + 2 * e] *= __fdividef(1.0f, 1.0f + __expf(-z.x)); o[8 * ch + 2 * e + 1] *= __fdividef(1.0f, 1.0f + __expf(-z.y));
+          }
+        }
+      }
       uint4* dst = (uint4*)(a.out + out_row);
 #pragma unroll
       for (int ch = 0; ch < AU_VD / 8; ++ch) {
@@ -497,23 +541,26 @@ static int au_pool_map(const bf16* base, int size, long long records, int G, CUt
 FELLM_API int fellm_attn_prefill_umma_takes(int H, int G, int hd, int vd, int page_tokens, int window) {
   if (G < 1 || H % G) return 0;
   const int R = H / G;
-  return (hd == AU_KD && vd == AU_VD && page_tokens == AU_PT && window <= 0 && R <= AU_ROWS && AU_ROWS % R == 0) ? 1 : 0;
+  return (hd == AU_KD && vd == AU_VD && page_tokens == AU_PT && (AU_EXTENDED || window <= 0) && R <= AU_ROWS && AU_ROWS % R == 0) ? 1 : 0;
 }
 
 // q [T, ldq] bfloat16, head h at column h hd (rotated; normed where the layer norms), out [T, H*vd]; pool [n_pages,
 // layers_in_group, record], a record being the keys [G][64][hd] and then the values [G][64][vd]; rows of item i are
 // item_start[i]..item_start[i+1], its positions are consecutive from positions[item_start[i]]; max_item_rows: the longest
 // item of the step.  sinks: float32 [H] or null.  status: device int32 that a role sets (311..317) if a wait ran out.
+// With -DAU_EXT also window (0: none), softcap (0: none) and og [T, ldog] bfloat16 (null: none), the outputs times its sigmoid.
 // FELLM_ERR_SIZE for sizes it does not take.
 FELLM_API int fellm_attn_prefill_umma(const void* q, int ldq, const void* pool, long long n_pages, const int* block_table,
                                       int max_pages, const int* positions, const int* row_slot, const int* item_start,
                                       int n_items, int max_item_rows, void* out, int T, int H, int G, int hd, int vd,
                                       int page_tokens, int layer, int layers_in_group, float scale, int window,
-                                      const float* sinks, int* status, cudaStream_t stream) {
+                                      const float* sinks, int* status, float softcap, const void* og, int ldog, cudaStream_t stream) {
   if (T <= 0 || n_items <= 0) return 0;
   if (!q || !pool || !block_table || !positions || !row_slot || !item_start || !out) return FELLM_ERR_ARG;
   if (!fellm_attn_prefill_umma_takes(H, G, hd, vd, page_tokens, window)) return FELLM_ERR_SIZE;
   if (!(scale > 0.f)) return FELLM_ERR_ARG;                    // a row's maximum is taken of the unscaled scores
+  if (!AU_EXTENDED && (softcap > 0.f || og)) return FELLM_ERR_SIZE;
+  if (softcap < 0.f || (og && (ldog < H * vd || (ldog & 7) || ((uintptr_t)og & 15)))) return FELLM_ERR_ARG;
   const long long records = n_pages * layers_in_group;
   if (records >= (1ll << 31) || ldq < H * hd || (ldq % 8) || ((uintptr_t)pool & 15) || ((uintptr_t)q & 15) || ((uintptr_t)out & 15))
     return FELLM_ERR_SIZE;
@@ -521,6 +568,7 @@ FELLM_API int fellm_attn_prefill_umma(const void* q, int ldq, const void* pool, 
   a.q = (const bf16*)q; a.ldq = ldq; a.block_table = block_table; a.positions = positions; a.row_slot = row_slot; a.item_start = item_start;
   a.out = (bf16*)out; a.status = status; a.sinks = sinks; a.max_pages = max_pages; a.H = H; a.G = G; a.layer = layer;
   a.layers_in_group = layers_in_group; a.scale_log2 = scale * 1.4426950408889634f;
+  a.og = (const bf16*)og; a.ldog = ldog; a.window = window > 0 ? window : 0; a.cap_log2 = softcap * 1.4426950408889634f;
   CUtensorMap k_map, v_map;
   int e = au_pool_map((const bf16*)pool, AU_KD, records, G, &k_map);
   if (!e) e = au_pool_map((const bf16*)pool + (size_t)G * AU_PT * AU_KD, AU_VD, records, G, &v_map);

@@ -40,6 +40,26 @@ __device__ __forceinline__ float glu_act(float g, float u, float limit, float al
   return g / (1.0f + expf(-g)) * u;
 }
 
+// A soft cap on attention scores, cap * tanh(s / cap).  tanh by two forms of it: up to 1/2 the Taylor series x - x^3/3 + 2 x^5/15
+// - 17 x^7/315 + 62 x^9/2835 - 1382 x^11/155925 + 21844 x^13/6081075 (the next term is below 1e-7 of x), beyond it (1 - e) / (1 +
+// e) with e = exp(-2 |x|).  The first costs no exponential and no division: a caller with many scores asks once whether all
+// of them are that small.
+#define SOFT_CAP_SERIES_TO 0.5f
+__device__ __forceinline__ float tanh_series(float x) {
+  const float y = x * x;
+  float p = 21844.0f / 6081075.0f;
+  p = fmaf(p, y, -1382.0f / 155925.0f);
+  p = fmaf(p, y, 62.0f / 2835.0f);
+  p = fmaf(p, y, -17.0f / 315.0f);
+  p = fmaf(p, y, 2.0f / 15.0f);
+  p = fmaf(p, y, -1.0f / 3.0f);
+  return fmaf(x * y, p, x);
+}
+__device__ __forceinline__ float tanh_any(float x) {
+  const float ax = fabsf(x), e = exp2f(ax * -2.885390081777927f);        // exp(-2 |x|)
+  return ax <= SOFT_CAP_SERIES_TO ? tanh_series(x) : copysignf(__fdividef(1.0f - e, 1.0f + e), x);
+}
+
 // ---- programmatic dependent launch: a kernel launched with launch_k() may start while its
 // predecessor in the stream is still running.  What does not depend on the predecessor (weight
 // prefetch, index set-up) goes before pdl_wait(); everything that reads or writes data another

@@ -1897,10 +1897,10 @@ def attention_decode(q, pool, block_table, positions, row_slot, layer, scale, wi
         return out
     f = _fn("attention_mma", "fellm_attn_decode_mma",
             [_c_p, _c_int, _c_p, _c_p, _c_int, _c_p, _c_p, _c_p, _c_p, _c_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int,
-             _c_int, _c_f, _c_int, _c_int, _c_int, _c_p, _c_p], defines={"HD": hd})
+             _c_int, _c_f, _c_int, _c_int, _c_int, _c_p, _c_f, _c_p, _c_int, _c_p], defines={"HD": hd})
     _check(f(_p(q), H * hd, _p(pool), _p(block_table), block_table.shape[1], _p(positions), _p(row_slot), _p(out),
              _p(scratch), _p(counters), T, H, G, hd, page_tokens, layer, pool.shape[1], float(scale),
-             int(window or 0), split_len, max_splits, None, _stream()), "attention_decode")
+             int(window or 0), split_len, max_splits, None, 0.0, None, 0, _stream()), "attention_decode")
     return out
 
 
@@ -1938,15 +1938,18 @@ def attention_prefill(q, pool, block_table, positions, row_slot, item_start, n_i
     return out
 
 
-def _umma_defines(hd: int, vd: int):
-    return None if hd == vd == 64 else {"AU_KD": hd, "AU_VD": vd}
+def _umma_defines(hd: int, vd: int, ext: bool = False):
+    d = {} if hd == vd == 64 else {"AU_KD": hd, "AU_VD": vd}
+    if ext:
+        d["AU_EXT"] = 1                 # with a window, a soft cap and a gate on the outputs
+    return d or None
 
 
-def umma_prefill_takes(H: int, G: int, hd: int, vd: int, page_tokens: int, window, scale: float) -> bool:
-    """Whether the tcgen05 attention of prompt portions takes a layer of these sizes: pages of 64 tokens, no window, a
-    positive scale, 128 rows a whole number of tokens' heads, key and value sizes of a multiple of 16 whose query, score
+def umma_prefill_takes(H: int, G: int, hd: int, vd: int, page_tokens: int, window, scale: float, ext: bool = False) -> bool:
+    """Whether the tcgen05 attention of prompt portions takes a layer of these sizes: pages of 64 tokens, no window (ext: the
+    library that takes one), a positive scale, 128 rows a whole number of tokens' heads, key and value sizes of a multiple of 16 whose query, score
     weight and page tiles (two atoms of 64 elements at most each, so four pages fit) and accumulators fit an SM."""
-    if not USE_UMMA_PREFILL or page_tokens != 64 or window or not scale > 0 or G < 1 or H % G or 128 % (H // G):
+    if not USE_UMMA_PREFILL or page_tokens != 64 or (window and not ext) or not scale > 0 or G < 1 or H % G or 128 % (H // G):
         return False
     if hd % 16 or vd % 16 or min(hd, vd) < 16:
         return False
@@ -1956,19 +1959,23 @@ def umma_prefill_takes(H: int, G: int, hd: int, vd: int, page_tokens: int, windo
 
 
 def _prefill_umma(q, ldq, H, G, hd, vd, pool, block_table, positions, row_slot, item_start, n_items, max_item_rows, layer,
-                  page_tokens, scale, sinks, out):
+                  page_tokens, scale, sinks, out, *, window=None, softcap=None, gate=None, ext=False):
     T = q.shape[0]
     f = _fn("attention_umma", "fellm_attn_prefill_umma",
             [_c_p, _c_int, _c_p, ctypes.c_longlong, _c_p, _c_int, _c_p, _c_p, _c_p, _c_int, _c_int, _c_p, _c_int, _c_int, _c_int,
-             _c_int, _c_int, _c_int, _c_int, _c_int, _c_f, _c_int, _c_p, _c_p, _c_p], defines=_umma_defines(hd, vd))
+             _c_int, _c_int, _c_int, _c_int, _c_int, _c_f, _c_int, _c_p, _c_p, _c_f, _c_p, _c_int, _c_p],
+            defines=_umma_defines(hd, vd, ext))
     _check(f(_p(q), int(ldq), _p(pool), pool.shape[0], _p(block_table), block_table.shape[1], _p(positions), _p(row_slot),
              _p(item_start), n_items, max_item_rows, _p(out), T, H, G, hd, vd, page_tokens, layer, pool.shape[1],
-             float(scale), 0, _p(sinks), _p(umma_status(q.device)), _stream()), "attention_prefill (tcgen05)")
+             float(scale), int(window or 0), _p(sinks), _p(umma_status(q.device)), float(softcap or 0.0), _p(gate),
+             gate.stride(0) if gate is not None else 0, _stream()), "attention_prefill (tcgen05)")
     return out
 
 
-def _mma_defines(hd: int, vd: int, wide: bool = False):
+def _mma_defines(hd: int, vd: int, wide: bool = False, ext: bool = False):
     d = {"HD": hd} if hd == vd else {"HD": hd, "VD": vd}
+    if ext:
+        d["EXT"] = 1                    # single tokens with a soft cap, a gate on the outputs and norms over whole projections
     if wide and _wide_stage_bytes(hd, vd) * 8 <= 216 * 1024:
         d["WIDE"] = 1                   # with the decode kernel that takes the input product's rows as they are
     return d
@@ -1992,10 +1999,12 @@ def decode_wide_takes(qkv, H: int, G: int, hd: int, vd: int, page_tokens: int, p
             and pool.data_ptr() % 16 == 0)
 
 
-def decode_wide_plan(max_len: int, rows: int, kv_heads: int, hd: int, vd: int):
+def decode_wide_plan(max_len: int, rows: int, kv_heads: int, hd: int, vd: int, window=None):
     """(split_len, ranges, stages, cluster): the key ranges of a row and kv head, how many half pages a warp keeps in flight,
     and whether the ranges merge as one cluster.  Chosen for contexts up to the next multiple of 1,024."""
     bucket = -(-max(max_len, 1) // 1024) * 1024
+    if window:
+        bucket = min(bucket, -(-(window + 63) // 64) * 64)       # the ranges start at the page of the window's first key
     items = max(rows * kv_heads, 1)
     stage = _wide_stage_bytes(hd, vd)
     per_sm = max(1, 227 * 1024 // (8 * stage + 9 * 1024 + 32 * hd))
@@ -2013,25 +2022,35 @@ def decode_wide_plan(max_len: int, rows: int, kv_heads: int, hd: int, vd: int):
     return split_len, ranges, stages, cluster
 
 
-def decode_wide_scratch_need(max_rows: int, heads: int, kv_heads: int, hd: int, vd: int, n_ctx: int):
+def decode_wide_scratch_need(max_rows: int, heads: int, kv_heads: int, hd: int, vd: int, n_ctx: int, window=None):
     """(floats, counters) attention_decode_wide can ask for with up to max_rows rows and contexts up to n_ctx."""
     floats = 0
     for rows in range(1, max(max_rows, 1) + 1):
         for bucket in range(1024, max(n_ctx, 1) + 1024, 1024):
-            floats = max(floats, rows * heads * decode_wide_plan(bucket, rows, kv_heads, hd, vd)[1] * (vd + 2))
+            floats = max(floats, rows * heads * decode_wide_plan(bucket, rows, kv_heads, hd, vd, window)[1] * (vd + 2))
     return floats, max(max_rows, 1) * kv_heads
 
 
 def attention_decode_wide(qkv, H, G, hd, vd, cache, ctx, scale, *, rot_dim=0, inv_freq=None, pairing="split_half", mag=1.0, v_first=None,
-                          lam=None, window=None, sinks=None, out=None):
+                          lam=None, window=None, sinks=None, softcap=None, gate=None, q_w=None, k_w=None, eps=0.0,
+                          reads_only=False, ext=False, out=None):
     """A decode step (every row its request's only one) straight from the input product's rows [q (H hd) | k (G hd) | v (G
     vd)]: what qkv_rotate_write and attention_written do, in one kernel (see decode_wide_takes); q stays as it was in
-    qkv.  Returns [T, H * vd]."""
+    qkv.  With ext (the library compiled for these) also what qkv_norm_rotate_write does (q_w, k_w, eps), softcap and gate
+    as attention_written, and reads_only: the rows hold no k and v, the pages are another layer's and nothing is written.
+    Returns [T, H * vd]."""
     pool, bt = cache.pool, cache.block_table
-    _dev(qkv, inv_freq, ctx.positions, ctx.row_slot, pool, bt, v_first, lam, sinks)
+    _dev(qkv, inv_freq, ctx.positions, ctx.row_slot, pool, bt, v_first, lam, sinks, gate, q_w, k_w)
     T = qkv.shape[0]
+    if not ext and (softcap or gate is not None or q_w is not None or reads_only):
+        raise KernelError("attention_decode_wide: a soft cap, a gate, norms or another layer's pages need the extended library")
+    if q_w is not None:
+        assert q_w.dtype == torch.float32 and q_w.numel() == H * hd and q_w.is_contiguous()
+        assert reads_only or (k_w.dtype == torch.float32 and k_w.numel() == G * hd and k_w.is_contiguous())
+    if gate is not None:
+        assert gate.shape == (T, H * vd) and gate.dtype == qkv.dtype and gate.stride(1) == 1
     assert decode_wide_takes(qkv, H, G, hd, vd, cache.page_tokens, pool)
-    assert qkv.stride(1) == 1 and qkv.shape[1] >= H * hd + G * (hd + vd) and pool.is_contiguous()
+    assert qkv.stride(1) == 1 and qkv.shape[1] >= H * hd + (0 if reads_only else G * (hd + vd)) and pool.is_contiguous()
     assert pool[0, 0].numel() == G * cache.page_tokens * (hd + vd)
     rot_dim = 0 if inv_freq is None else int(rot_dim)
     if rot_dim % 2 or not 0 <= rot_dim <= hd:
@@ -2044,29 +2063,31 @@ def attention_decode_wide(qkv, H, G, hd, vd, cache, ctx, scale, *, rot_dim=0, in
     if sinks is not None:
         assert sinks.dtype == torch.float32 and sinks.numel() == H and sinks.is_contiguous()
     _i32(ctx.positions, "positions"), _i32(ctx.row_slot, "row_slot"), _i32(bt, "block_table")
-    split_len, ranges, stages, cluster = decode_wide_plan(ctx.max_len, T, G, hd, vd)
+    split_len, ranges, stages, cluster = decode_wide_plan(ctx.max_len, T, G, hd, vd, window)
     scratch, counters = reserve_decode_scratch(pool.device, T, H, G, vd, ranges)
     if out is None:
         out = torch.empty((T, H * vd), dtype=torch.bfloat16, device=qkv.device)
     f = _fn("attention_mma", "fellm_attn_decode_wide",
             [_c_p, _c_int, _c_p, _c_ll, _c_p, _c_int, _c_p, _c_p, _c_p, _c_p, _c_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int,
-             _c_int, _c_f, _c_int, _c_int, _c_int, _c_p, _c_int, _c_int, _c_f, _c_p, _c_int, _c_p, _c_p, _c_int, _c_int, _c_p, _c_p],
-            defines=_mma_defines(hd, vd, True))
+             _c_int, _c_f, _c_int, _c_int, _c_int, _c_p, _c_int, _c_int, _c_f, _c_p, _c_int, _c_p, _c_p, _c_int, _c_int, _c_p,
+             _c_f, _c_p, _c_int, _c_p, _c_p, _c_f, _c_int, _c_p],
+            defines=_mma_defines(hd, vd, True, ext))
     _check(f(_p(qkv), qkv.stride(0), _p(pool), pool.shape[0], _p(bt), bt.shape[1], _p(ctx.positions), _p(ctx.row_slot), _p(out),
              _p(scratch), _p(counters), T, H, G, hd, vd, cache.page_tokens, cache.layer, pool.shape[1], float(scale), int(window or 0),
              split_len, ranges, _p(inv_freq), rot_dim, PAIRINGS[pairing], float(mag), _p(v_first),
              v_first.stride(0) if v_first is not None else 0, _p(lam), _p(sinks), stages, int(cluster), _p(umma_status(pool.device)),
-             _stream()), "attention_decode_wide")
+             float(softcap or 0.0), _p(gate), gate.stride(0) if gate is not None else 0, _p(q_w), _p(k_w), float(eps),
+             int(bool(reads_only)), _stream()), "attention_decode_wide")
     return out
 
 
-def written_attention_modules(dtype: str, H: int, G: int, hd: int, vd: int, page_tokens: int, window, scale: float):
+def written_attention_modules(dtype: str, H: int, G: int, hd: int, vd: int, page_tokens: int, window, scale: float, ext: bool = False):
     """The modules attention_written launches for a layer of these sizes."""
     mods = [("attention_simt", None)]
     if dtype == "bfloat16" and _mma_takes(H, G, hd, vd):
-        mods.append(("attention_mma", _mma_defines(hd, vd, True)))
-        if umma_prefill_takes(H, G, hd, vd, page_tokens, window, scale):
-            mods.append(("attention_umma", _umma_defines(hd, vd)))
+        mods.append(("attention_mma", _mma_defines(hd, vd, True, ext)))
+        if umma_prefill_takes(H, G, hd, vd, page_tokens, window, scale, ext):
+            mods.append(("attention_umma", _umma_defines(hd, vd, ext)))
     return mods
 
 
@@ -2075,11 +2096,12 @@ def _mma_takes(H: int, G: int, hd: int, vd: int) -> bool:
             and H // G <= 64)
 
 
-def attention_written(qkv, H, G, hd, vd, cache, ctx, scale, *, window=None, softcap=None, sinks=None, gate=None, warps=8, out=None):
+def attention_written(qkv, H, G, hd, vd, cache, ctx, scale, *, window=None, softcap=None, sinks=None, gate=None, warps=8, ext=False,
+                      out=None):
     """Attention of a step's rows over pages that already hold the rows' own keys and values (qkv_rotate_write): query head
     h of row t is qkv[t, h hd : (h + 1) hd] as it lies; keys of hd, values of vd; sinks float32 [H]: exp(sinks[h]) joins
     head h's softmax denominator; softcap: scores c tanh(s / c); gate [T, H * vd] (qkv's dtype, rows of any stride): the result
-    times sigmoid(gate), element by element.  bfloat16 on tensor cores (portions: tcgen05 where the sizes allow, else mma.sync; single
+    times sigmoid(gate), element by element (both on tensor cores with ext, the libraries compiled for them).  bfloat16 on tensor cores (portions: tcgen05 where the sizes allow, else mma.sync; single
     tokens: the key walk split over CTAs), everything else on CUDA cores.  Returns [T, H * vd] in qkv's dtype."""
     pool, bt, positions, row_slot = cache.pool, cache.block_table, ctx.positions, ctx.row_slot
     if qkv.dtype != torch.bfloat16 or not _mma_takes(H, G, hd, vd) or qkv.stride(0) % 8 or qkv.data_ptr() % 16 or pool.data_ptr() % 16:
@@ -2097,41 +2119,43 @@ def attention_written(qkv, H, G, hd, vd, cache, ctx, scale, *, window=None, soft
     _i32(bt, "block_table"), _i32(positions, "positions"), _i32(row_slot, "row_slot")
     if out is None:
         out = torch.empty((T, H * vd), dtype=torch.bfloat16, device=qkv.device)
-    if ctx.all_single and softcap:
-        paged_attention_general(qkv, H, hd, vd, pool, bt, positions, row_slot, cache.layer, pt, G, scale, window=window,
-                                softcap=softcap, warps=warps, sinks=sinks, out=out)
-        return out if gate is None else gate_mul(out, gate)
+    if not ext and (softcap or gate is not None):
+        raise KernelError("attention_written: a soft cap or a gate needs the extended libraries (ext)")
+    if gate is not None:
+        assert gate.shape == (T, H * vd) and gate.dtype == qkv.dtype and gate.stride(1) == 1
+    ldg = gate.stride(0) if gate is not None else 0
     if ctx.all_single:
         split_len, max_splits = decode_split(ctx.max_len, T, G)
         scratch, counters = reserve_decode_scratch(pool.device, T, H, G, vd, max_splits)
         f = _fn("attention_mma", "fellm_attn_decode_mma",
                 [_c_p, _c_int, _c_p, _c_p, _c_int, _c_p, _c_p, _c_p, _c_p, _c_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int,
-                 _c_int, _c_f, _c_int, _c_int, _c_int, _c_p, _c_p], defines=_mma_defines(hd, vd, True))
+                 _c_int, _c_f, _c_int, _c_int, _c_int, _c_p, _c_f, _c_p, _c_int, _c_p], defines=_mma_defines(hd, vd, True, ext))
         _check(f(_p(qkv), qkv.stride(0), _p(pool), _p(bt), bt.shape[1], _p(positions), _p(row_slot), _p(out), _p(scratch),
                  _p(counters), T, H, G, hd, pt, cache.layer, pool.shape[1], float(scale), int(window or 0), split_len,
-                 max_splits, _p(sinks), _stream()), "attention_decode")
+                 max_splits, _p(sinks), float(softcap or 0.0), _p(gate), ldg, _stream()), "attention_decode")
         return out
     _i32(ctx.item_start, "item_start")
-    if umma_prefill_takes(H, G, hd, vd, pt, window, scale) and not softcap and gate is None:
+    if umma_prefill_takes(H, G, hd, vd, pt, window, scale, ext) and (gate is None or (ldg % 8 == 0 and gate.data_ptr() % 16 == 0)):
         return _prefill_umma(qkv, qkv.stride(0), H, G, hd, vd, pool, bt, positions, row_slot, ctx.item_start, ctx.n_items,
-                             ctx.max_item_rows, cache.layer, pt, scale, sinks, out)
+                             ctx.max_item_rows, cache.layer, pt, scale, sinks, out, window=window, softcap=softcap, gate=gate, ext=ext)
     _prefill_biased(qkv, pool, bt, positions, row_slot, ctx.item_start, ctx.n_items, ctx.max_item_rows, out, T, H, G, hd, vd, pt,
-                    cache.layer, scale, window, softcap=softcap, sinks=sinks, wide=True)
-    return out if gate is None else gate_mul(out, gate)
+                    cache.layer, scale, window, softcap=softcap, sinks=sinks, wide=True, out_gate=gate, ext=ext)
+    return out
 
 
 def _prefill_biased(qkv, pool, block_table, positions, row_slot, item_start, n_items, max_item_rows, out, T, H, G, hd, vd,
                     page_tokens, layer, scale, window, *, chunk=None, softcap=None, gate=None, slopes=None, q_temp=None,
-                    values_are_keys=False, sinks=None, wide=False):
+                    values_are_keys=False, sinks=None, wide=False, out_gate=None, ext=False):
     qt_coef, qt_every = q_temp if q_temp else (0.0, 0)
     f = _fn("attention_mma", "fellm_attn_prefill_mma_biased",
             [_c_p, _c_int, _c_p, _c_p, _c_int, _c_p, _c_p, _c_p, _c_int, _c_int, _c_p, _c_int, _c_int, _c_int, _c_int, _c_int,
-             _c_int, _c_int, _c_f, _c_int, _c_int, _c_f, _c_p, _c_int, _c_p, _c_f, _c_int, _c_int, _c_p, _c_p],
-            defines=_mma_defines(hd, vd, wide))
+             _c_int, _c_int, _c_f, _c_int, _c_int, _c_f, _c_p, _c_int, _c_p, _c_f, _c_int, _c_int, _c_p, _c_p, _c_int, _c_p],
+            defines=_mma_defines(hd, vd, wide, ext))
     _check(f(_p(qkv), qkv.stride(0), _p(pool), _p(block_table), block_table.shape[1], _p(positions), _p(row_slot),
              _p(item_start), n_items, max_item_rows, _p(out), T, H, G, hd, page_tokens, layer, pool.shape[1], float(scale),
              int(window or 0), int(chunk or 0), float(softcap or 0.0), _p(gate), gate.stride(0) if gate is not None else 0,
-             _p(slopes), float(qt_coef), int(qt_every), int(bool(values_are_keys)), _p(sinks), _stream()), "attention_prefill_general")
+             _p(slopes), float(qt_coef), int(qt_every), int(bool(values_are_keys)), _p(sinks), _p(out_gate),
+             out_gate.stride(0) if out_gate is not None else 0, _stream()), "attention_prefill_general")
 
 
 def attention_prefill_general(qkv, H, pool, block_table, positions, row_slot, item_start, n_items, max_item_rows, layer,

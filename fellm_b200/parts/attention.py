@@ -208,7 +208,7 @@ class Attention(Mixer):
             ops.reserve_decode_scratch(device, 1, self.H, self.G, self.hd, 1, floats=floats, counters=counters)
         elif self.w["qkv.weight"].dtype == torch.bfloat16 and self.written:
             floats, counters = ops.decode_scratch_need(max_rows, self.H, self.G, self.vd, n_ctx)
-            floats = max(floats, ops.decode_wide_scratch_need(max_rows, self.H, self.G, self.hd, self.vd, n_ctx)[0])
+            floats = max(floats, ops.decode_wide_scratch_need(max_rows, self.H, self.G, self.hd, self.vd, n_ctx, self.window)[0])
             ops.reserve_decode_scratch(device, 1, self.H, self.G, self.vd, 1, floats=floats, counters=counters)
 
     can_store = property(lambda self: self.general)        # (the general path's forward(store=True) writes its rows)
@@ -287,9 +287,12 @@ class Attention(Mixer):
             v_first = ctx.carried["v_first"]
         mag = getattr(self.position, "magnitude", 1.0)
         gate = qkv[:, self.gate_off:self.gate_off + H * vd] if self.out_gate else None
-        kw = dict(window=self.window, sinks=self.w.get("sink"))
-        if ctx.all_single and not self.whole_norm and ops.decode_wide_takes(qkv, H, G, hd, vd, cache.page_tokens, cache.pool):
-            # a decode step: rotation, mixing and the cache write happen inside the attention kernel
+        # (ext: the libraries that also take a soft cap, a gate and norms over whole projections)
+        kw = dict(window=self.window, sinks=self.w.get("sink"), softcap=self.softcap, gate=gate, ext=self.whole_norm)
+        if ctx.all_single and ops.decode_wide_takes(qkv, H, G, hd, vd, cache.page_tokens, cache.pool):
+            # a decode step: norm, rotation, mixing and the cache write happen inside the attention kernel
+            if self.whole_norm:
+                kw.update(q_w=self.w["q_norm.weight"], k_w=self.w.get("k_norm.weight"), eps=self.eps, reads_only=self.shares_cache)
             a = ops.attention_decode_wide(qkv, H, G, hd, vd, cache, ctx, self.scale, rot_dim=self.rot_dim, inv_freq=self.position.inv_freq,
                                           pairing=self.position.pairing, mag=mag, v_first=v_first, lam=self.w.get("vmix"), **kw)
             linear(a, self.w["out_proj.weight"], out=out, accumulate=not store)
@@ -301,7 +304,7 @@ class Attention(Mixer):
         else:
             ops.qkv_rotate_write(qkv, H, G, hd, vd, self.rot_dim, self.position.inv_freq, self.position.pairing, mag, ctx.positions,
                                  ctx.row_slot, cache, v_first=v_first, lam=self.w.get("vmix"), status=ctx.status)
-        a = ops.attention_written(qkv, H, G, hd, vd, cache, ctx, self.scale, softcap=self.softcap, gate=gate, warps=self.simt_warps, **kw)
+        a = ops.attention_written(qkv, H, G, hd, vd, cache, ctx, self.scale, warps=self.simt_warps, **kw)
         linear(a, self.w["out_proj.weight"], out=out, accumulate=not store)
         return out
 
@@ -342,7 +345,7 @@ class Attention(Mixer):
     def kernel_modules(self, dtype):
         if self.written:
             return linear_modules(dtype) + [("qk_rope_write", None)] + ([("sublayer", None)] if self.out_gate else []) + \
-                ops.written_attention_modules(dtype, self.H, self.G, self.hd, self.vd, 64, self.window, self.scale)
+                ops.written_attention_modules(dtype, self.H, self.G, self.hd, self.vd, 64, self.window, self.scale, self.whole_norm)
         if self.general:
             mma = dtype == "bfloat16" and self.vd == self.hd and self.hd % 16 == 0 and self.H // self.G <= 64
             extra = ([("qk_rope_write", None)] if self.in_place else []) + ([("sublayer", None)] if self.out_gate else [])
