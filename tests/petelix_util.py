@@ -113,8 +113,11 @@ def write_folder(folder, cfg, seed, scales=SCALES):
         for pat, s in scales:
             if pat in name and tensors[name].dim() == 2:
                 tensors[name] = (tensors[name].float() * s).bfloat16()
-        if name.endswith(".correction"):          # choice scores on both sides of zero
-            tensors[name] = (tensors[name].float() - 0.2).bfloat16()
+        if name.endswith(".correction"):
+            # choice scores on both sides of zero, and far apart where the scores are small: fewer choices that rounding decides
+            n = tensors[name].numel()
+            order = np.random.default_rng(seed + n).permutation(n)
+            tensors[name] = torch.from_numpy(0.2 - 0.9 * order / max(n, 10)).bfloat16()
     (folder / "config.json").write_text(json.dumps(typed.to_dict(), indent=1))
     write_safetensors(folder / "model.safetensors", tensors)
     return str(folder)
@@ -178,6 +181,7 @@ def row_distances(got, want) -> torch.Tensor:
 
 
 LIMIT = {"float32": 2e-5, "bfloat16": 5e-2}
+NOISE = {"M": 3.0, "W": 3.0}        # (sharp scores and experts on top of one another: rounding itself is that much larger)
 
 
 def assert_close(got, want, dtype: str, times: float = 1.0, note=None):
