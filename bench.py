@@ -406,11 +406,23 @@ def vofezen_config(width, ff, layers, vocab):
                              mlp=dict(ff=ff, kind="dense")) for i in range(layers)])
 
 
+def petelix_config(width, ff, layers, vocab):
+    """A Petelix model of real-looking layers at this width: attention with heads of 64 (one per 64 of width, four per key
+    head), queries and keys normed over their whole projections, half a head rotated, a soft cap of 50, a window of 1,024
+    positions, an output gate, every second layer reading the keys and values of the one before it; behind each 8 experts of
+    ff / 2 and 4 identity experts, in 4 groups of which 2 are kept, two a token."""
+    H = max(width // 64, 1)
+    att = dict(dim=64, heads=H, kv_heads=max(H // 4, 1), mask=dict(size=1024), rot=dict(base=10000.0, dims=32), scale=0.125, softcap=50.0, vdim=64)
+    moe = dict(expert=dict(ff=ff // 2), kind="moe", router=dict(experts=8, groups=dict(count=4, keep=2), identity=4, top=2))
+    return dict(architecture="Petelix", embedding=dict(scale=1.0), vocab=vocab, width=width, norm=dict(eps=1e-5),
+                layers=[dict(type="attention", mixer=dict(att, kv_from=i - 1) if i % 2 else att, mlp=moe) for i in range(layers)])
+
+
 DESIGNS = {"robazen": robazen_config, "samusun": samusun_config, "meresun": meresun_config, "nalizen": nalizen_config,
-           "vofezen": vofezen_config}
+           "vofezen": vofezen_config, "petelix": petelix_config}
 # the models a design is measured beside (default: LFM2 of the same width, depth, feed-forward and vocabulary);
 # "lfm2_attention": LFM2 with attention in every layer
-BESIDE = {"meresun": ("samusun",), "nalizen": ("samusun",), "vofezen": ("lfm2_attention", "meresun")}
+BESIDE = {"meresun": ("samusun",), "nalizen": ("samusun",), "vofezen": ("lfm2_attention", "meresun"), "petelix": ("nalizen", "meresun")}
 
 
 def run_design(design, shapes, layers, batches, steps, warmup):
@@ -606,7 +618,7 @@ def main():
     ap.add_argument("--context", type=int, default=PROMPT)
     ap.add_argument("--design", choices=sorted(DESIGNS), default=None,
                     help="prefill and decode throughput of this design at a few real-looking sizes beside the closest model of "
-                         "equal width, depth and feed-forward (LFM2; Samusun for meresun and nalizen; LFM2 with attention in every layer and Meresun for vofezen) (--layers layers, default 8; --steps decode steps, default 64); "
+                         "equal width, depth and feed-forward (LFM2; Samusun for meresun and nalizen; LFM2 with attention in every layer and Meresun for vofezen; Nalizen and Meresun for petelix) (--layers layers, default 8; --steps decode steps, default 64); "
                          "prints one line of its own and leaves the headline measurement alone")
     args = ap.parse_args()
 

@@ -98,16 +98,18 @@ __device__ __forceinline__ void cap_scores(float (&s)[N][4], float f0, float f1,
   }
   if (__all_sync(0xffffffffu, am <= SOFT_CAP_SERIES_TO)) {
 #pragma unroll
-    for (int n = 0; n < N; ++n) {
-#pragma unroll
-      for (int e = 0; e < 4; ++e) s[n][e] = cap_log2 * tanh_series(s[n][e]);
-    }
+    for (int n = 0; n < N; ++n) { tanh_series_f2<false>(s[n][0], s[n][1]); tanh_series_f2<false>(s[n][2], s[n][3]); }
   } else {
 #pragma unroll
     for (int n = 0; n < N; ++n) {
 #pragma unroll
-      for (int e = 0; e < 4; ++e) s[n][e] = cap_log2 * tanh_any(s[n][e]);
+      for (int e = 0; e < 4; ++e) s[n][e] = tanh_any(s[n][e]);
     }
+  }
+#pragma unroll
+  for (int n = 0; n < N; ++n) {
+#pragma unroll
+    for (int e = 0; e < 4; ++e) s[n][e] *= cap_log2;
   }
 }
 

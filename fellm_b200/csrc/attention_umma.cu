@@ -319,7 +319,7 @@ attention_prefill_umma_kernel(const __grid_constant__ CUtensorMap k_map, const _
     const unsigned t_acc = t_row + AU_COL_O + grp * AU_VC * 32;
     const unsigned s_full = s_full0 + 16 * grp, p_full = p_full0 + 16 * grp, o_full = o_full0 + 16 * grp;
     const bool capped = AU_EXTENDED && a.cap_log2 > 0.f;
-    const float scale = capped ? 1.0f : a.scale_log2;            // (capped scores are in the log2 domain already)
+    const float scale = capped ? a.cap_log2 : a.scale_log2;      // (capped: of tanh's values)
     const float cap_in = capped ? a.scale_log2 / a.cap_log2 : 0.f;
     const int lo = (AU_EXTENDED && a.window > 0) ? pos - a.window + 1 : 0;         // the first key the row sees
     // The accumulator of P V stays in tensor memory, scaled by 2^-m where m is the row's REFERENCE
@@ -348,15 +348,23 @@ attention_prefill_umma_kernel(const __grid_constant__ CUtensorMap k_map, const _
       au_tmem_ld32_issue(t_row + AU_COL_S + (2 * grp + (i & 1)) * AU_PT + 32, sc + 32);
       au_tmem_ld_wait();
       if (capped) {
-        float am = 0.f;
+        float a2[2] = {0.f, 0.f};
+        const unsigned long long f2 = pack_f2(cap_in, cap_in);
 #pragma unroll
-        for (int c = 0; c < AU_PT; ++c) { sc[c] *= cap_in; am = fmaxf(am, fabsf(sc[c])); }
-        if (__all_sync(0xffffffffu, am <= SOFT_CAP_SERIES_TO)) {
+        for (int c = 0; c < AU_PT; c += 2) {
+          unpack_f2(mul_f2(pack_f2(sc[c], sc[c + 1]), f2), sc[c], sc[c + 1]);
+          a2[0] = fmaxf(a2[0], fabsf(sc[c])); a2[1] = fmaxf(a2[1], fabsf(sc[c + 1]));
+        }
+        const float am = fmaxf(a2[0], a2[1]);
+        if (__all_sync(0xffffffffu, am <= SOFT_CAP_SHORT_TO)) {
 #pragma unroll
-          for (int c = 0; c < AU_PT; ++c) sc[c] = a.cap_log2 * tanh_series(sc[c]);
+          for (int c = 0; c < AU_PT; c += 2) tanh_series_f2<true>(sc[c], sc[c + 1]);
+        } else if (__all_sync(0xffffffffu, am <= SOFT_CAP_SERIES_TO)) {
+#pragma unroll
+          for (int c = 0; c < AU_PT; c += 2) tanh_series_f2<false>(sc[c], sc[c + 1]);
         } else {
 #pragma unroll
-          for (int c = 0; c < AU_PT; ++c) sc[c] = a.cap_log2 * tanh_any(sc[c]);
+          for (int c = 0; c < AU_PT; ++c) sc[c] = tanh_any(sc[c]);
         }
       }
       if (key0 + AU_PT - 1 > pos) {

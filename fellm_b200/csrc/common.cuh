@@ -41,23 +41,53 @@ __device__ __forceinline__ float glu_act(float g, float u, float limit, float al
 }
 
 // A soft cap on attention scores, cap * tanh(s / cap).  tanh by two forms of it: up to 1/2 the Taylor series x - x^3/3 + 2 x^5/15
-// - 17 x^7/315 + 62 x^9/2835 - 1382 x^11/155925 + 21844 x^13/6081075 (the next term is below 1e-7 of x), beyond it (1 - e) / (1 +
-// e) with e = exp(-2 |x|).  The first costs no exponential and no division: a caller with many scores asks once whether all
-// of them are that small.
+// - 17 x^7/315 + 62 x^9/2835 - 1382 x^11/155925 + 21844 x^13/6081075 (the next term is below 1e-7 of x; up to 1/4 the terms
+// to x^9 do), beyond it (1 - e) / (1 + e) with e = exp(-2 |x|).  The series costs no exponential and no division and runs on
+// pairs (two float32 operations an instruction): a caller with many scores asks once whether all of them are that small.
+#define SOFT_CAP_SHORT_TO 0.25f
 #define SOFT_CAP_SERIES_TO 0.5f
-__device__ __forceinline__ float tanh_series(float x) {
-  const float y = x * x;
-  float p = 21844.0f / 6081075.0f;
-  p = fmaf(p, y, -1382.0f / 155925.0f);
+__device__ __forceinline__ unsigned long long pack_f2(float a, float b) {
+  unsigned long long r;
+  asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(a), "f"(b));
+  return r;
+}
+__device__ __forceinline__ void unpack_f2(unsigned long long v, float& a, float& b) { asm("mov.b64 {%0, %1}, %2;" : "=f"(a), "=f"(b) : "l"(v)); }
+__device__ __forceinline__ unsigned long long mul_f2(unsigned long long a, unsigned long long b) {
+  unsigned long long r;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+  return r;
+}
+__device__ __forceinline__ unsigned long long fma_f2(unsigned long long a, unsigned long long b, unsigned long long c) {
+  unsigned long long r;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
+  return r;
+}
+// tanh of two numbers of at most 1/2 (SHORT: 1/4).
+template <bool SHORT>
+__device__ __forceinline__ void tanh_series_f2(float& a, float& b) {
+  auto two = [](float c) { return pack_f2(c, c); };
+  const unsigned long long x = pack_f2(a, b), y = mul_f2(x, x);
+  unsigned long long p = two(62.0f / 2835.0f);
+  if (!SHORT) {
+    p = fma_f2(two(21844.0f / 6081075.0f), y, two(-1382.0f / 155925.0f));
+    p = fma_f2(p, y, two(62.0f / 2835.0f));
+  }
+  p = fma_f2(p, y, two(-17.0f / 315.0f));
+  p = fma_f2(p, y, two(2.0f / 15.0f));
+  p = fma_f2(p, y, two(-1.0f / 3.0f));
+  unpack_f2(fma_f2(mul_f2(x, y), p, x), a, b);
+}
+__device__ __forceinline__ float tanh_any(float x) {
+  const float y = x * x;                  // (one at a time: pairs would hold twice the registers here)
+  float p = fmaf(21844.0f / 6081075.0f, y, -1382.0f / 155925.0f);
   p = fmaf(p, y, 62.0f / 2835.0f);
   p = fmaf(p, y, -17.0f / 315.0f);
   p = fmaf(p, y, 2.0f / 15.0f);
   p = fmaf(p, y, -1.0f / 3.0f);
-  return fmaf(x * y, p, x);
-}
-__device__ __forceinline__ float tanh_any(float x) {
-  const float ax = fabsf(x), e = exp2f(ax * -2.885390081777927f);        // exp(-2 |x|)
-  return ax <= SOFT_CAP_SERIES_TO ? tanh_series(x) : copysignf(__fdividef(1.0f - e, 1.0f + e), x);
+  const float s = fmaf(x * y, p, x), ax = fabsf(x);
+  float e;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(ax * -2.885390081777927f));        // exp(-2 |x|)
+  return ax <= SOFT_CAP_SERIES_TO ? s : copysignf(__fdividef(1.0f - e, 1.0f + e), x);
 }
 
 // ---- programmatic dependent launch: a kernel launched with launch_k() may start while its

@@ -18,6 +18,12 @@
 #define MOE_MAX_TOP 16
 #define PLAN_TILE 1024
 
+__device__ __forceinline__ void unpack8(const uint4& raw, float* f) {
+  const __nv_bfloat162* h = (const __nv_bfloat162*)&raw;
+#pragma unroll
+  for (int e = 0; e < 4; ++e) { float2 v = __bfloat1622float2(h[e]); f[2 * e] = v.x; f[2 * e + 1] = v.y; }
+}
+
 // ---------------------------------------------------------------- routing
 // One warp: softmax over z[0..E) in float32, the `top` largest (ties: the lower expert) into idx / w.
 __device__ __forceinline__ void route_warp(const float* z, int E, int top, int renorm, int* idx, float* w, int lane) {
@@ -170,9 +176,10 @@ FELLM_API int fellm_moe_route(const float* logits, int ld, int T, int E, int top
 
 // The router's product and the routing in one kernel: a block per token, its warps take the experts by turns
 // (z_e = sum_k h[k] Wr[e, k] in float32: a lane sums its share of k in order, the lanes are added by a butterfly: the
-// order depends on K alone), then the first warp routes.  h [T, ldh] and Wr [E, K] bfloat16 or float32.
-#define ROUTER_WARPS 4
-template <typename TA, typename TW>
+// order depends on K alone), then the first warp routes.  h [T, ldh] and Wr [E, K] bfloat16 or float32.  VEC (both
+// bfloat16, K a multiple of 8, rows on 16-byte boundaries): a lane takes eight k at a time.
+#define ROUTER_WARPS 8
+template <typename TA, typename TW, bool VEC>
 __global__ void __launch_bounds__(ROUTER_WARPS * 32)
 moe_router_kernel(const TA* __restrict__ h, int ldh, const TW* __restrict__ Wr, int K, int E, int top, int renorm,
                   int* __restrict__ idx, float* __restrict__ w, int form, const float* __restrict__ corr,
@@ -183,7 +190,17 @@ moe_router_kernel(const TA* __restrict__ h, int ldh, const TW* __restrict__ Wr, 
   for (int e = warp; e < E; e += ROUTER_WARPS) {
     const TW* wr = Wr + (size_t)e * K;
     float s = 0.f;
-    for (int k = lane; k < K; k += 32) s = fmaf(to_f(hr[k]), to_f(wr[k]), s);
+    if constexpr (VEC) {
+#pragma unroll 4
+      for (int k = lane * 8; k < K; k += 256) {
+        float a[8], b[8];
+        unpack8(*(const uint4*)(hr + k), a); unpack8(*(const uint4*)(wr + k), b);
+#pragma unroll
+        for (int j = 0; j < 8; ++j) s = fmaf(a[j], b[j], s);
+      }
+    } else {
+      for (int k = lane; k < K; k += 32) s = fmaf(to_f(hr[k]), to_f(wr[k]), s);
+    }
     s = warp_sum(s);
     if (lane == 0) zs[e] = bias ? s + bias[e] : s;
   }
@@ -192,6 +209,45 @@ moe_router_kernel(const TA* __restrict__ h, int ldh, const TW* __restrict__ Wr, 
     if (form) route_choice_warp(form == 2, zs, corr, E, top, renorm, n_groups, keep, gtop, zs + E, idx + (size_t)t * top, w + (size_t)t * top, lane);
     else route_warp(zs, E, top, renorm, idx + (size_t)t * top, w + (size_t)t * top, lane);
   }
+}
+
+// The same sums for many tokens (bfloat16, as VEC above): a warp a token, its experts four at a time against one reading
+// of h, so that no warp waits while another routes.
+__global__ void __launch_bounds__(ROUTER_WARPS * 32)
+moe_router_many_kernel(const bf16* __restrict__ h, int ldh, const bf16* __restrict__ Wr, int T, int K, int E, int top, int renorm,
+                       int* __restrict__ idx, float* __restrict__ w, int form, const float* __restrict__ corr,
+                       int n_groups, int keep, int gtop, const float* __restrict__ bias, int per_warp) {
+  extern __shared__ float zs_all[];             // per_warp floats a warp
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, t = blockIdx.x * ROUTER_WARPS + warp;
+  if (t >= T) return;
+  float* zs = zs_all + (size_t)warp * per_warp;
+  const bf16* hr = h + (size_t)t * ldh;
+  for (int e0 = 0; e0 < E; e0 += 4) {
+    const bf16* wr[4];
+    float s[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+    for (int i = 0; i < 4; ++i) wr[i] = Wr + (size_t)min(e0 + i, E - 1) * K;
+#pragma unroll 2
+    for (int k = lane * 8; k < K; k += 256) {
+      float a[8];
+      unpack8(*(const uint4*)(hr + k), a);
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        float b[8];
+        unpack8(*(const uint4*)(wr[i] + k), b);
+#pragma unroll
+        for (int j = 0; j < 8; ++j) s[i] = fmaf(a[j], b[j], s[i]);
+      }
+    }
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      s[i] = warp_sum(s[i]);
+      if (lane == 0 && e0 + i < E) zs[e0 + i] = bias ? s[i] + bias[e0 + i] : s[i];
+    }
+  }
+  __syncwarp();
+  if (form) route_choice_warp(form == 2, zs, corr, E, top, renorm, n_groups, keep, gtop, zs + E, idx + (size_t)t * top, w + (size_t)t * top, lane);
+  else route_warp(zs, E, top, renorm, idx + (size_t)t * top, w + (size_t)t * top, lane);
 }
 
 FELLM_API int fellm_moe_router(const void* h, int h_bf16, int ldh, const void* Wr, int w_bf16, int T, int K, int E, int top,
@@ -207,22 +263,48 @@ FELLM_API int fellm_moe_router(const void* h, int h_bf16, int ldh, const void* W
   if (form < 0 || form > 2 || (form && (E % n_groups || keep < 1 || keep > n_groups || gtop < 1 || top > (E / n_groups) * keep))) return FELLM_ERR_SIZE;
   if (!h || !Wr || !idx || !w) return FELLM_ERR_ARG;
   const size_t sh = (size_t)(form ? 2 * E + n_groups : E) * sizeof(float);
-#define ROUTER(TA_, TW_) moe_router_kernel<TA_, TW_><<<T, ROUTER_WARPS * 32, sh, stream>>>((const TA_*)h, ldh, (const TW_*)Wr, K, E, top, renorm, idx, w, form, corr, n_groups, keep, gtop, bias)
-  if (h_bf16) { if (w_bf16) ROUTER(bf16, bf16); else ROUTER(bf16, float); }
-  else { if (w_bf16) ROUTER(float, bf16); else ROUTER(float, float); }
+#define ROUTER(TA_, TW_, V_) moe_router_kernel<TA_, TW_, V_><<<T, ROUTER_WARPS * 32, sh, stream>>>((const TA_*)h, ldh, (const TW_*)Wr, K, E, top, renorm, idx, w, form, corr, n_groups, keep, gtop, bias)
+  const bool vec = h_bf16 && w_bf16 && K % 8 == 0 && ldh % 8 == 0 && (((uintptr_t)h | (uintptr_t)Wr) & 15) == 0;
+  if (vec && T >= 256 && sh * ROUTER_WARPS <= 48 * 1024) {
+    moe_router_many_kernel<<<(T + ROUTER_WARPS - 1) / ROUTER_WARPS, ROUTER_WARPS * 32, sh * ROUTER_WARPS, stream>>>(
+        (const bf16*)h, ldh, (const bf16*)Wr, T, K, E, top, renorm, idx, w, form, corr, n_groups, keep, gtop, bias, (int)(sh / sizeof(float)));
+    return launch_status();
+  }
+  if (vec) ROUTER(bf16, bf16, true);
+  else if (h_bf16) { if (w_bf16) ROUTER(bf16, bf16, false); else ROUTER(bf16, float, false); }
+  else { if (w_bf16) ROUTER(float, bf16, false); else ROUTER(float, float, false); }
 #undef ROUTER
   return launch_status();
 }
 
 // ---------------------------------------------------------------- the plan
 // Pairs p = t * top + c, P of them.  A choice beyond the E experts (an identity expert: the token's input handed on, no
-// product) is no row of the plan: its place is -1.  n_tiles[0]: row tiles, n_tiles[1]: sorted rows.  Tile i of PLAN_TILE pairs: counts[i][e] and each pair's rank among the pairs of
-// its tile that chose the same expert before it.
+// product) is no row of the plan: its place is -1.  n_tiles[0]: row tiles, n_tiles[1]: sorted rows.  Tile i of PLAN_TILE
+// pairs: counts[i][e] and each pair's rank among the pairs of its tile that chose the same expert before it.
 __global__ void __launch_bounds__(PLAN_TILE)
-moe_count_kernel(const int* __restrict__ idx, int P, int E, int* __restrict__ counts, int* __restrict__ rank) {
-  __shared__ int ex[PLAN_TILE];
+moe_count_kernel(const int* __restrict__ idx, int P, int E, int* __restrict__ counts, int* __restrict__ rank, int per_warp) {
+  extern __shared__ int sh[];
   const int p = blockIdx.x * PLAN_TILE + threadIdx.x;
   const int e = p < P && idx[p] < E ? idx[p] : -1;
+  if (per_warp) {
+    // [32 warps][E]: a warp's pairs of each expert; then, down the warps, those in front of it
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    for (int i = threadIdx.x; i < 32 * E; i += PLAN_TILE) sh[i] = 0;
+    __syncthreads();
+    const unsigned same = __match_any_sync(0xffffffffu, e);
+    const int before = __popc(same & ((1u << lane) - 1));
+    if (e >= 0 && before == 0) sh[warp * E + e] = __popc(same);
+    __syncthreads();
+    for (int i = threadIdx.x; i < E; i += PLAN_TILE) {
+      int n = 0;
+      for (int w = 0; w < 32; ++w) { const int c = sh[w * E + i]; sh[w * E + i] = n; n += c; }
+      counts[(size_t)blockIdx.x * E + i] = n;
+    }
+    __syncthreads();
+    if (e >= 0) rank[p] = sh[warp * E + e] + before;
+    return;
+  }
+  int* ex = sh;                          // [PLAN_TILE]
   ex[threadIdx.x] = e;
   for (int i = threadIdx.x; i < E; i += PLAN_TILE) counts[(size_t)blockIdx.x * E + i] = 0;
   __syncthreads();
@@ -328,7 +410,8 @@ FELLM_API int fellm_moe_plan(const int* idx, int P, int E, int BM, int* scratch,
   }
   const int tiles = (P + PLAN_TILE - 1) / PLAN_TILE;
   int* counts = scratch; int* base = counts + (size_t)tiles * E; int* rank = base + (size_t)tiles * E;
-  moe_count_kernel<<<tiles, PLAN_TILE, 0, stream>>>(idx, P, E, counts, rank);
+  const bool per_warp = E <= 320;        // 40 KB of counts; more experts: every pair looks at the tile's others
+  moe_count_kernel<<<tiles, PLAN_TILE, (per_warp ? (size_t)32 * E : PLAN_TILE) * sizeof(int), stream>>>(idx, P, E, counts, rank, per_warp);
   const size_t sh = (size_t)3 * E * sizeof(int);
   if (sh > 48 * 1024) return FELLM_ERR_SIZE;
   moe_scan_kernel<<<1, 1024, sh, stream>>>(counts, tiles, E, BM, base, table, n_tiles);
@@ -517,11 +600,6 @@ moe_gemm_mma_kernel(const bf16* __restrict__ A, int lda, const int* __restrict__
 // sums are added by a butterfly.  bfloat16 only; K a multiple of 8.
 #define VW 8            // warps a block
 #define VR 4            // rows at once
-__device__ __forceinline__ void unpack8(const uint4& raw, float* f) {
-  const __nv_bfloat162* h = (const __nv_bfloat162*)&raw;
-#pragma unroll
-  for (int e = 0; e < 4; ++e) { float2 v = __bfloat1622float2(h[e]); f[2 * e] = v.x; f[2 * e + 1] = v.y; }
-}
 // A warp's columns: n and, GATED, its up partner; not gated: n and n + 1 (two weight rows against the same rows of A).
 template <typename TO, bool GATED>
 __global__ void __launch_bounds__(VW * 32)
@@ -667,11 +745,45 @@ __global__ void moe_combine_kernel(float* __restrict__ x, const float* __restric
   }
 }
 
+// The same, d a multiple of 4 and everything on 16-byte boundaries (h on 8): four elements a thread.
+__device__ __forceinline__ float4 load4(const float* p) { return *(const float4*)p; }
+__device__ __forceinline__ float4 load4(const bf16* p) {
+  const uint2 raw = *(const uint2*)p;
+  const __nv_bfloat162* h2 = (const __nv_bfloat162*)&raw;
+  const float2 a = __bfloat1622float2(h2[0]), b = __bfloat1622float2(h2[1]);
+  return make_float4(a.x, a.y, b.x, b.y);
+}
+template <typename TH>
+__global__ void moe_combine_vec_kernel(float* __restrict__ x, const float* __restrict__ y, const int* __restrict__ place_of,
+                                       const float* __restrict__ w, const TH* __restrict__ h, int ldh, int T, int top, int d4, int store) {
+  const long long u = (long long)blockIdx.x * blockDim.x + threadIdx.x;
+  if (u >= (long long)T * d4) return;
+  const int t = (int)(u / d4), i = 4 * (int)(u - (long long)t * d4), d = 4 * d4;
+  float4* dst = (float4*)(x + (size_t)t * d + i);
+  const float4 old = store ? make_float4(0.f, 0.f, 0.f, 0.f) : *dst;
+  float4 s = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 4
+  for (int c = 0; c < top; ++c) {
+    const int place = place_of[(size_t)t * top + c];
+    const float f = w[(size_t)t * top + c];
+    const float4 v = place < 0 ? load4(h + (size_t)t * ldh + i) : load4(y + (size_t)place * d + i);
+    s.x = fmaf(f, v.x, s.x); s.y = fmaf(f, v.y, s.y); s.z = fmaf(f, v.z, s.z); s.w = fmaf(f, v.w, s.w);
+  }
+  *dst = store ? s : make_float4(old.x + s.x, old.y + s.y, old.z + s.z, old.w + s.w);
+}
+
 // h [T, ldh] (bfloat16 or float32): needed where a plan has identity experts, else null.
 FELLM_API int fellm_moe_combine(float* x, const float* y, const int* place_of, const float* w, const void* h, int h_bf16, int ldh,
                                 int T, int top, int d, int store, cudaStream_t stream) {
   if (T <= 0) return 0;
   if (!x || !y || !place_of || !w) return FELLM_ERR_ARG;
+  if (d % 4 == 0 && (((uintptr_t)x | (uintptr_t)y | (uintptr_t)h) & 15) == 0 && ldh % 4 == 0) {
+    const int d4 = d / 4;
+    const unsigned blocks = (unsigned)(((long long)T * d4 + 127) / 128);
+    if (h_bf16) moe_combine_vec_kernel<bf16><<<blocks, 128, 0, stream>>>(x, y, place_of, w, (const bf16*)h, ldh, T, top, d4, store);
+    else moe_combine_vec_kernel<float><<<blocks, 128, 0, stream>>>(x, y, place_of, w, (const float*)h, ldh, T, top, d4, store);
+    return launch_status();
+  }
   const int threads = d >= 256 ? 256 : 128;
   if (h_bf16) moe_combine_kernel<bf16><<<T, threads, 0, stream>>>(x, y, place_of, w, (const bf16*)h, ldh, top, d, store);
   else moe_combine_kernel<float><<<T, threads, 0, stream>>>(x, y, place_of, w, (const float*)h, ldh, top, d, store);

@@ -258,14 +258,15 @@ def test_decode_from_the_input_products_rows(monkeypatch, H, G, hd, vd, rot, pai
 
 
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+@pytest.mark.parametrize("T", [37, 301])                 # (a block a token, a warp a token)
 @pytest.mark.parametrize("K,E,ident,top,count,keep", [(96, 6, 9, 4, 5, 2), (71, 7, 2, 3, 3, 2), (128, 1, 1, 1, 1, 1), (64, 2, 14, 1, 8, 3),
                                                       (256, 40, 24, 16, 16, 5), (40, 3, 0, 3, 3, 3), (1024, 96, 160, 8, 8, 4)])
-def test_router_choice(dtype, K, E, ident, top, count, keep):
+def test_router_choice(dtype, T, K, E, ident, top, count, keep):
     """Softmax scores over experts and identity experts, the choice by score + correction (all choice scores negative; in every
     second case the correction outweighs the scores) inside the best groups, the weights the plain scores."""
     from fellm_b200 import ops
     g = torch.Generator().manual_seed(K + E)
-    n, T = E + ident, 37
+    n = E + ident
     h = torch.randn(T, K, generator=g).to(dtype)
     wr = (torch.randn(n, K, generator=g) * (2.0 / math.sqrt(K))).to(dtype)
     corr = -1.0 - torch.rand(n, generator=g) * (0.7 if K % 3 else 0.02)
