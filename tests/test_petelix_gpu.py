@@ -141,7 +141,7 @@ def _attention_case(H, G, hd, vd, page, T, window, seed):
 @pytest.mark.parametrize("H,G,hd,vd,page,T,window", [
     (8, 1, 128, 80, 64, 300, 70), (16, 4, 128, 64, 64, 270, 128), (4, 4, 48, 96, 64, 150, 1), (8, 2, 80, 16, 64, 200, None),
     (2, 1, 128, 80, 64, 330, 65), (32, 1, 64, 48, 64, 100, 31), (6, 2, 64, 48, 64, 200, 64), (4, 2, 64, 32, 16, 130, 33),
-    (3, 1, 256, 32, 64, 100, 50), (4, 1, 24, 40, 16, 90, 17), (2, 2, 7, 5, 16, 70, 16), (4, 2, 64, 32, 64, 400, 136)])
+    (3, 1, 256, 32, 64, 100, 50), (4, 1, 24, 40, 16, 90, 17), (2, 2, 7, 5, 16, 70, 16), (12, 3, 64, 32, 64, 400, 150)])
 def test_attention_with_window_cap_sink_and_gate_over_written_pages(H, G, hd, vd, page, T, window, cap):
     """Portions that start and end in front of, on and behind the edges of pages, of windows and of the kernels' blocks,
     single tokens alone (the key walk split over CTAs) and beside portions, of two requests in one step: tcgen05 where the
@@ -199,7 +199,7 @@ def test_attention_with_window_cap_sink_and_gate_over_written_pages(H, G, hd, vd
 @pytest.mark.parametrize("H,G,hd,vd,rot,pairing,window,cap,own", [
     (8, 1, 128, 80, 64, "adjacent", 100, 5.0, True), (16, 4, 128, 64, 32, "adjacent", 1000, 30.0, True), (4, 4, 48, 96, 0, "adjacent", 64, 2.0, True),
     (16, 1, 80, 16, 2, "adjacent", None, 9.0, True), (12, 1, 128, 80, 128, "split_half", 1, 20.0, True), (4, 2, 80, 16, 48, "adjacent", 65, None, True),
-    (6, 2, 48, 96, 16, "split_half", 600, 1.0, True), (4, 2, 64, 32, 16, "adjacent", 136, 50.0, False), (10, 1, 64, 48, 64, "adjacent", 31, 4.0, False),
+    (6, 2, 48, 96, 16, "split_half", 600, 1.0, True), (12, 3, 64, 32, 24, "adjacent", 150, 40.0, False), (10, 1, 64, 48, 64, "adjacent", 31, 4.0, False),
     (8, 2, 128, 64, 32, "adjacent", None, 7.0, False)])
 @pytest.mark.parametrize("ranges,stages,cluster", [(8, 0, True), (8, 2, False), (40, 4, False), (1, 0, True)])
 def test_decode_from_the_input_products_rows(monkeypatch, H, G, hd, vd, rot, pairing, window, cap, own, ranges, stages, cluster):
